@@ -90,6 +90,11 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
     return __float2bfloat16_rn(x);
 }
 
+// xIELU with its two constants: z > 0: p z^2 + z/2;  z <= 0: n (exp(z) - 1 - z) + z/2
+__device__ __forceinline__ float lia_xielu(float z, float p, float n) {
+    return fmaf(0.5f, z, z > 0.f ? p * z * z : n * (expm1f(z) - z));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -38,6 +38,54 @@ LIA_EXPORT int lia_embedding(const int* tokens, const void* table, int table_dty
 }
 
 // ---------------------------------------------------------------------------------------
+// Embedding with a sinusoidal vector of the position: h[t, c] = table[token_t, c] * scale + sin(p f_i) for even c, the
+// cosine for odd c, i = c / 2, p the token's position; angles, sines and cosines 32-bit.  `copy` (optional): the same
+// rows in the compute element type (the input of a first layer that reads the stream itself).
+template <typename TW, typename TC>
+__global__ void embedding_sinusoidal_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
+                                            const TW* __restrict__ table, const float* __restrict__ freq,
+                                            float* __restrict__ out, TC* __restrict__ copy, int n_tokens, int hidden,
+                                            int vocab, float scale, int* __restrict__ error_flag) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    if (t >= n_tokens) return;
+    const int token = tokens[t];
+    const float position = (float)positions[t];
+    const bool ok = token >= 0 && token < vocab;
+    if (!ok && threadIdx.x == 0 && blockIdx.y == 0 && error_flag) atomicExch(error_flag, 1);
+    const TW* row = table + (size_t)(ok ? token : 0) * hidden;
+    float* dst = out + (size_t)t * hidden;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; 2 * i < hidden; i += gridDim.y * blockDim.x) {
+        float sn, cs;
+        sincosf(position * freq[i], &sn, &cs);
+        for (int c = 2 * i; c < min(hidden, 2 * i + 2); ++c) {
+            const float v = ok ? fmaf(to_float(row[c]), scale, (c & 1) ? cs : sn) : 0.f;
+            dst[c] = v;
+            if (copy) copy[(size_t)t * hidden + c] = from_float<TC>(v);
+        }
+    }
+}
+
+// freq [(hidden + 1) / 2] 32-bit, positions [n]; copy [n, hidden] of copy_dtype or null.
+LIA_EXPORT int lia_embedding_sinusoidal(const int* tokens, const int* positions, const void* table, int table_dtype,
+                                        const float* freq, float* out, void* copy, int copy_dtype, int n_tokens, int hidden,
+                                        int vocab, float scale, int* error_flag, cudaStream_t stream) {
+    if (n_tokens <= 0) return LIA_OK;
+    if (hidden <= 0 || vocab <= 0 || !freq) return LIA_ERR_SIZE;
+    const int threads = 128;
+    const dim3 grid(n_tokens, n_tokens >= 256 ? 1 : (hidden / 2 + threads) / threads);
+#define LIA_SINUSOIDAL(TW, TC)                                                                                          \
+    return lia_launch(embedding_sinusoidal_kernel<TW, TC>, grid, dim3(threads), 0, stream, tokens, positions,          \
+                      (const TW*)table, freq, out, (TC*)copy, n_tokens, hidden, vocab, scale, error_flag)
+    if (table_dtype == LIA_BF16 && copy_dtype == LIA_BF16) LIA_SINUSOIDAL(__nv_bfloat16, __nv_bfloat16);
+    if (table_dtype == LIA_BF16 && copy_dtype == LIA_F32) LIA_SINUSOIDAL(__nv_bfloat16, float);
+    if (table_dtype == LIA_F32 && copy_dtype == LIA_F32) LIA_SINUSOIDAL(float, float);
+#undef LIA_SINUSOIDAL
+    return LIA_ERR_DTYPE;
+}
+
+// ---------------------------------------------------------------------------------------
 // RMSNorm of 32-bit rows: y = x * rsqrt(mean(x^2) + eps) * w * out_scale.
 // Sum of squares, mean, eps and the reciprocal root are 32-bit; the order of the additions
 // depends on `hidden` alone, not on the number of rows.  `rows_index` (optional) gathers:

@@ -46,8 +46,9 @@
 // gate, out = up * relu(gate), and the storing form with out = relu(alpha * sum)^2.
 #define GEMM_REGLU 3
 #define GEMM_STORE_RELU2 4
+#define GEMM_STORE_XIELU 5
 #define GATED(MODE) ((MODE) == GEMM_SWIGLU || (MODE) == GEMM_REGLU)
-#define STORES(MODE) ((MODE) == GEMM_STORE || (MODE) == GEMM_STORE_RELU2)
+#define STORES(MODE) ((MODE) == GEMM_STORE || (MODE) == GEMM_STORE_RELU2 || (MODE) == GEMM_STORE_XIELU)
 
 namespace {
 constexpr int ROWS = 16;                 // rows of W per block: the MMA's M
@@ -124,6 +125,7 @@ struct Args {
     int stages, early, chunks, ck;   // ring; stages asked for before the tokens' rows; K chunks per block; elements of K per chunk (a multiple of 64)
     int blocks, x_pitch, stage_bytes, half_bytes;
     int norm, out_bf16;              // norm: 0 none, 1 weight bf16, 2 weight f32
+    float act_p, act_n;              // xIELU's two constants
     int activation;                  // STORE only: 0 none, 1 GELU (tanh form), 2 SiLU, applied to alpha * sum before the store
     float alpha, eps;
     int* error_flag;
@@ -385,6 +387,8 @@ gemm_stream_kernel(Args a) {
                         } else if (MODE == GEMM_STORE_RELU2) {
                             value = fmaxf(value, 0.f);
                             value *= value;
+                        } else if (MODE == GEMM_STORE_XIELU) {
+                            value = lia_xielu(value, a.act_p, a.act_n);
                         }
                         if (a.out_bf16) reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)token * a.ldo + f] = __float2bfloat16_rn(value);
                         else reinterpret_cast<float*>(a.out)[(size_t)token * a.ldo + f] = value;
@@ -731,16 +735,17 @@ LIA_EXPORT int lia_gemm_stream_stages(int mode, int M, int N, int K, int with_no
 // pointers that are not 16-byte aligned (bulk copies and 16-byte loads need both), and sizes whose rows do not
 // fit in shared memory beside a ring (ask lia_gemm_stream_stages first).  `stages_cap` > 0 limits the ring;
 // `early_stages` > 0 sets how many stages the producer asks for before the tokens' rows have been asked for (default 2).
-// `activation`: STORE: 1 the tanh form of GELU, 2 SiLU, 3 the square of ReLU; SWIGLU: 4 makes the gate a ReLU; applied to the 32-bit result before it is stored.
+// `activation`: STORE: 1 the tanh form of GELU, 2 SiLU, 3 the square of ReLU, 5 xIELU with the constants act_p, act_n; SWIGLU: 4 makes the gate a ReLU; applied to the 32-bit result before it is stored.
 LIA_EXPORT int lia_gemm_stream(int mode, const void* X, int ldx, const void* W, int ldw, void* out, int out_dtype,
                                int ldo, int M, int N, int K, float alpha, const float* norm_src, int ld_norm,
                                const void* norm_weight, int norm_weight_dtype, float eps, int sms, int stages_cap,
-                               int early_stages, int activation, int* error_flag, cudaStream_t stream) {
+                               int early_stages, int activation, float act_p, float act_n, int* error_flag, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return LIA_OK;
-    // the kernel's form: the mode, or one of the two forms that an activation selects
+    // the kernel's form: the mode, or one of the forms that an activation selects
     int form = mode;
     if (mode == GEMM_SWIGLU && activation == 4) form = GEMM_REGLU, activation = 0;
     else if (mode == GEMM_STORE && activation == 3) form = GEMM_STORE_RELU2, activation = 0;
+    else if (mode == GEMM_STORE && activation == 5) form = GEMM_STORE_XIELU, activation = 0;
     if (activation < 0 || activation > 2 || (activation && mode != GEMM_STORE)) return LIA_ERR_SIZE;
     if (M > TOKENS || K <= 0 || K % 64 || ldw % 8 || ldw < K || ldo < N || sms <= 0) return LIA_ERR_SIZE;
     if ((uintptr_t)W & 15u) return LIA_ERR_ALIGN;
@@ -761,6 +766,7 @@ LIA_EXPORT int lia_gemm_stream(int mode, const void* X, int ldx, const void* W, 
     a.norm = !norm_src ? 0 : (norm_weight_dtype == LIA_BF16 ? 1 : 2);
     a.out_bf16 = out_dtype == LIA_BF16;
     a.activation = activation;
+    a.act_p = act_p; a.act_n = act_n;
     a.ldw = ldw; a.ldx = ldx; a.ldo = ldo; a.M = M; a.N = N; a.K = K; a.alpha = alpha; a.error_flag = error_flag;
     chunking(K, &a.chunks, &a.ck);
     const long long blocks = mode == GEMM_SWIGLU ? (N + HALF_ROWS - 1) / HALF_ROWS : (N + ROWS - 1) / ROWS;
@@ -779,5 +785,6 @@ LIA_EXPORT int lia_gemm_stream(int mode, const void* X, int ldx, const void* W, 
     if (form == GEMM_ACCUM) return launch_form<GEMM_ACCUM>(a, form_chunks, form_pw, ctas, stream);
     if (form == GEMM_REGLU) return launch_form<GEMM_REGLU>(a, form_chunks, form_pw, ctas, stream);
     if (form == GEMM_STORE_RELU2) return launch_form<GEMM_STORE_RELU2>(a, form_chunks, form_pw, ctas, stream);
+    if (form == GEMM_STORE_XIELU) return launch_form<GEMM_STORE_XIELU>(a, form_chunks, form_pw, ctas, stream);
     return launch_form<GEMM_SWIGLU>(a, form_chunks, form_pw, ctas, stream);
 }

@@ -47,10 +47,11 @@ using namespace tc5;
 #define GEMM_STORE 0
 #define GEMM_ACCUM 1
 #define GEMM_SWIGLU 2
-// Two more forms of the kernel, instantiations of their own so that the three above are what they were: the gated form
-// with a ReLU gate, out = up * relu(gate), and the storing form with out = relu(alpha * sum)^2.
+// More forms of the kernel, instantiations of their own so that the three above are what they were: the gated form
+// with a ReLU gate, out = up * relu(gate), and the storing forms with out = relu(alpha * sum)^2 and out = xIELU(alpha * sum).
 #define GEMM_REGLU 3
 #define GEMM_STORE_RELU2 4
+#define GEMM_STORE_XIELU 5
 #define GATED(MODE) ((MODE) == GEMM_SWIGLU || (MODE) == GEMM_REGLU)
 
 namespace {
@@ -75,6 +76,7 @@ struct Shape {
     int via_tma;              // 1: the epilogue leaves through shared memory and TMA
     int ldo;
     float alpha;
+    float act_p, act_n;       // xIELU's two constants
     float* partial;           // [splits][M][n_total]
     int* counters;            // [f_tiles * t_tiles], zero between launches
     int* error_flag;
@@ -121,9 +123,11 @@ __device__ __forceinline__ float relu_squared(float z) {
 }
 
 template <int MODE, typename TO>
-__device__ __forceinline__ void apply_epilogue(TO* dst, float acc, float up, float alpha) {
+__device__ __forceinline__ void apply_epilogue(TO* dst, float acc, float up, const Shape& s) {
+    const float alpha = s.alpha;
     if (MODE == GEMM_STORE) *dst = from_float<TO>(alpha * acc);
     else if (MODE == GEMM_STORE_RELU2) *dst = from_float<TO>(relu_squared(alpha * acc));
+    else if (MODE == GEMM_STORE_XIELU) *dst = from_float<TO>(lia_xielu(alpha * acc, s.act_p, s.act_n));
     else if (MODE == GEMM_REGLU) *dst = from_float<TO>(up * fmaxf(acc, 0.f));
     else if (MODE == GEMM_ACCUM) *dst = from_float<TO>(to_float(*dst) + alpha * acc);
     else *dst = from_float<TO>(up * (acc / (1.0f + __expf(-acc))));
@@ -356,7 +360,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                             for (int c = 0; c < 8; ++c)
                                 if (c0 + c < rows)
-                                    apply_epilogue<MODE, TO>(out + (size_t)(u.t0 + c0 + c) * s.ldo + f, acc[c], up[c], s.alpha);
+                                    apply_epilogue<MODE, TO>(out + (size_t)(u.t0 + c0 + c) * s.ldo + f, acc[c], up[c], s);
                         }
                     }
                 }
@@ -382,6 +386,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         if (MODE == GEMM_SWIGLU) v = up[c] * __fdividef(acc[c], 1.0f + __expf(-acc[c]));
                         else if (MODE == GEMM_REGLU) v = up[c] * fmaxf(acc[c], 0.f);
                         else if (MODE == GEMM_STORE_RELU2) v = relu_squared(s.alpha * acc[c]);
+                        else if (MODE == GEMM_STORE_XIELU) v = lia_xielu(s.alpha * acc[c], s.act_p, s.act_n);
                         else v = s.alpha * acc[c];
                         stage[c * TILE_F + group * 32 + lane] = from_float<TO>(v);
                     }
@@ -408,7 +413,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         for (int c = 0; c < 16; ++c) {
                             const int t = u.t0 + c0 + c;
                             if (t >= u.t_end) break;
-                            apply_epilogue<MODE, TO>(out + (size_t)t * s.ldo + f, acc[c], up[c], s.alpha);
+                            apply_epilogue<MODE, TO>(out + (size_t)t * s.ldo + f, acc[c], up[c], s);
                         }
                     }
                 }
@@ -515,10 +520,10 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const CUtensorMap& mo, 
 // of 8 elements, pointers that are not 16-byte aligned.
 LIA_EXPORT int lia_gemm_tc(int mode, const void* X, int ldx, const void* W, int ldw, void* out, int out_dtype,
                            int ldo, int M, int N, int K, float alpha, float* scratch, long long scratch_floats,
-                           int sm_count, int* error_flag, cudaStream_t stream) {
-    const int act = mode >> 8;           // the epilogue's variant rides above the mode's byte
+                           int sm_count, float act_p, float act_n, int* error_flag, cudaStream_t stream) {
+    const int act = mode >> 8;           // the epilogue's variant rides above the mode's byte (5: xIELU with act_p, act_n)
     mode &= 0xff;
-    if (act != 0 && !(mode == GEMM_SWIGLU && act == 4) && !(mode == GEMM_STORE && act == 3)) return LIA_ERR_SIZE;
+    if (act != 0 && !(mode == GEMM_SWIGLU && act == 4) && !(mode == GEMM_STORE && (act == 3 || act == 5))) return LIA_ERR_SIZE;
     if (M <= 0 || N <= 0) return LIA_OK;
     if (K <= 0 || K % 8 || ldx < K || ldw < K || ldo < N || sm_count <= 0) return LIA_ERR_SIZE;
     if (mode != GEMM_STORE && mode != GEMM_ACCUM && mode != GEMM_SWIGLU) return LIA_ERR_SIZE;
@@ -536,6 +541,7 @@ LIA_EXPORT int lia_gemm_tc(int mode, const void* X, int ldx, const void* W, int 
     s.acc_buffers = 2 * s.acc_cols <= 512 ? 2 : 1;
     s.tmem_cols = pow2_at_least(s.acc_buffers * s.acc_cols);
     s.ldo = ldo; s.alpha = alpha; s.error_flag = error_flag;
+    s.act_p = act_p; s.act_n = act_n;
     s.group_tiles = nullptr; s.group_count = nullptr; s.group_rows = 0;
     s.counters = reinterpret_cast<int*>(scratch);
     s.partial = scratch ? scratch + COUNTER_WORDS : nullptr;
@@ -557,6 +563,10 @@ LIA_EXPORT int lia_gemm_tc(int mode, const void* X, int ldx, const void* W, int 
     }
     const long long units = (long long)plan.f_tiles * plan.t_tiles * plan.splits;
     const int grid = (int)min((long long)sm_count, units);
+    if (mode == GEMM_STORE && act == 5) {
+        if (out_dtype == LIA_F32) return launch<GEMM_STORE_XIELU, float>(mw, mx, mo, (float*)out, s, grid, stream);
+        return launch<GEMM_STORE_XIELU, __nv_bfloat16>(mw, mx, mo, (__nv_bfloat16*)out, s, grid, stream);
+    }
     if (mode == GEMM_STORE && act == 3) {
         if (out_dtype == LIA_F32) return launch<GEMM_STORE_RELU2, float>(mw, mx, mo, (float*)out, s, grid, stream);
         return launch<GEMM_STORE_RELU2, __nv_bfloat16>(mw, mx, mo, (__nv_bfloat16*)out, s, grid, stream);
@@ -679,12 +689,13 @@ LIA_EXPORT long long lia_gemm_tc_noalloc_scratch_floats(int mode, int M, int N, 
 LIA_EXPORT int lia_gemm_tc_noalloc(int mode, const void* X, int ldx, const void* W, int ldw, void* out,
                                    int out_dtype, int ldo, int M, int N, int K, float alpha, int sm_count,
                                    int* error_flag, cudaStream_t stream) {
+    if ((mode >> 8) == 5) return LIA_ERR_SIZE;                 // xIELU's constants have no way in here
     if (lia_gemm_tc_noalloc_scratch_floats(mode & 0xff, M, N, K, sm_count) > NOALLOC_FLOATS) return LIA_ERR_SCRATCH;
     float* scratch = nullptr;
     const int rc = noalloc_scratch_address(&scratch);
     if (rc != LIA_OK) return rc;
     return lia_gemm_tc(mode, X, ldx, W, ldw, out, out_dtype, ldo, M, N, K, alpha, scratch, NOALLOC_FLOATS,
-                       sm_count, error_flag, stream);
+                       sm_count, 0.f, 0.f, error_flag, stream);
 }
 
 // Puts the tile counters at the head of the array back to zero, in stream order.  For use after a call whose

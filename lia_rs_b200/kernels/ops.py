@@ -56,14 +56,15 @@ class _Signatures:
     lia_attention_decode_cluster_splits = [c_int, c_int, c_int, c_int]
     lia_attention_decode_ctas_per_sm = [c_int, c_int]
     lia_gemm_tc = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                   c_void_p, ctypes.c_longlong, c_int, c_void_p, c_void_p]
+                   c_void_p, ctypes.c_longlong, c_int, c_float, c_float, c_void_p, c_void_p]
     lia_gemm_cluster = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                         c_int, c_void_p, c_void_p]
     lia_gemm_cluster_splits = [c_int, c_int, c_int, c_int, c_int]
     lia_gemm_skinny = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                        c_void_p, c_void_p]
     lia_gemm_stream = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                       c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+                       c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p,
+                       c_void_p]
     lia_gemm_stream_stages = [c_int, c_int, c_int, c_int, c_int, c_int]
     lia_attention_prefill = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
@@ -96,7 +97,8 @@ class _Signatures:
 
     lia_norm_residual = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float,
                          c_void_p]
-    lia_activation_rows = [c_void_p, ctypes.c_longlong, c_void_p, c_int, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p]
+    lia_activation_rows = [c_void_p, ctypes.c_longlong, c_void_p, c_int, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_float, c_float,
+                           c_void_p]
     lia_attention_general = [c_void_p, ctypes.c_longlong, ctypes.c_longlong, c_void_p, ctypes.c_longlong, ctypes.c_longlong,
                              c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                              c_int, c_void_p, c_void_p, ctypes.c_longlong, ctypes.c_longlong, c_int, c_int, c_int, c_int,
@@ -143,6 +145,24 @@ class _Signatures:
     lia_gla = [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, c_int,
                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, ctypes.c_longlong, c_void_p, c_int,
                c_void_p, c_int, c_float, c_float, c_void_p]
+    lia_embedding_sinusoidal = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                c_float, c_void_p, c_void_p]
+    lia_norm_terms_residual = [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_void_p, c_float, c_float,
+                               c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p]
+    lia_ring_conv = [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p,
+                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
+    lia_ring_store = [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_int, c_int,
+                      c_void_p]
+    lia_rglru_gates = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                       c_void_p]
+    lia_rglru_scan = [c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                      ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                      c_void_p]
+    lia_ssd = [c_void_p, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong,
+               c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+               ctypes.c_longlong, c_void_p]
+    lia_gated_group_norm = [c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                            c_void_p]
     lia_retention_chunks = [c_int, c_int]
     lia_retention_encode = [c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                             c_void_p]
@@ -277,6 +297,20 @@ def embedding(tokens, table, out, scale: float, error_flag=None):
                                    table.shape[0], scale, _p(error_flag), _stream()), "embedding")
 
 
+def embedding_sinusoidal(tokens, positions, table, freq, out, scale: float, copy=None, error_flag=None):
+    """out[t] = table[tokens[t]] * scale + the position's vector (sine of position * freq[i] in column 2i, cosine in 2i + 1);
+    `copy`: the same rows in the compute element type; see csrc/elementwise.cu."""
+    _cuda(tokens, positions, table, freq, out, copy, error_flag)
+    n, hidden = out.shape
+    if freq.dtype != torch.float32 or freq.numel() < (hidden + 1) // 2 or table.shape[1] != hidden or \
+            (copy is not None and tuple(copy.shape) != (n, hidden)):
+        raise KernelError("embedding_sinusoidal: one 32-bit frequency per pair of columns, rows of the table's width")
+    with _timed("embedding"):
+        _check(lib().lia_embedding_sinusoidal(_p(tokens), _p(positions), _p(table), dtype_code(table.dtype), _p(freq), _p(out),
+                                              _p(copy), F32 if copy is None else dtype_code(copy.dtype), n, hidden,
+                                              table.shape[0], float(scale), _p(error_flag), _stream()), "embedding_sinusoidal")
+
+
 def rmsnorm(x, weight, out, eps: float, out_scale: float = 1.0, rows_index=None):
     _cuda(x, weight, out, rows_index)
     rows, hidden = out.shape
@@ -391,10 +425,11 @@ def gemm_tc_tiles_fill_the_sms(a, out) -> bool:
     return 4 * ((out.shape[1] + 127) // 128) >= 3 * sms
 
 
-def gemm_tc(mode, a, w, out, alpha: float = 1.0, error_flag=None, label=None, act: int = 0):
+def gemm_tc(mode, a, w, out, alpha: float = 1.0, error_flag=None, label=None, act: int = 0, act_constants=(0.0, 0.0)):
     """out[M, N] (op)= alpha * a[M, K] @ w[N, K]^T on the tensor cores; see csrc/gemm_tc.cu.  Products
     with few tiles split K and use this device's scratch, so calls on one device must not overlap.
-    `act`: with GEMM_SWIGLU, ACT_RELU makes the gate a ReLU; with GEMM_STORE, ACT_RELU_SQUARED squares the result's ReLU."""
+    `act`: with GEMM_SWIGLU, ACT_RELU makes the gate a ReLU; with GEMM_STORE, ACT_RELU_SQUARED squares the result's ReLU
+    and ACT_XIELU applies xIELU with `act_constants`."""
     M, K = a.shape
     N = out.shape[1]
     if w.shape[1] != K or out.shape[0] != M or w.shape[0] != (2 * N if mode == GEMM_SWIGLU else N):
@@ -402,8 +437,8 @@ def gemm_tc(mode, a, w, out, alpha: float = 1.0, error_flag=None, label=None, ac
     scratch, sms = _device_scratch(a.device)
     with _timed("gemm_tc", label, work=lambda: _gemm_work(a, w, out)):
         _check(lib().lia_gemm_tc(mode | (int(act) << 8), _p(a), a.stride(0), _p(w), w.stride(0), _p(out), dtype_code(out.dtype),
-                                 out.stride(0), M, N, K, alpha, _p(scratch), scratch.numel(), sms, _p(error_flag),
-                                 _stream()), "gemm_tc")
+                                 out.stride(0), M, N, K, alpha, _p(scratch), scratch.numel(), sms, float(act_constants[0]),
+                                 float(act_constants[1]), _p(error_flag), _stream()), "gemm_tc")
 
 
 def gemm_cluster_accepts(mode, a, w, out) -> bool:
@@ -474,11 +509,11 @@ def gemm_stream_accepts(mode, a, w, out, norm=False) -> bool:
 
 
 def gemm_stream(mode, a, w, out, alpha: float = 1.0, error_flag=None, label=None, norm_weight=None, eps: float = 0.0,
-                stages_cap: int = 0, early_stages: int = 0, activation: int = 0):
+                stages_cap: int = 0, early_stages: int = 0, activation: int = 0, act_constants=(0.0, 0.0)):
     """out[M, N] (op)= alpha * x[M, K] @ w[N, K]^T for M <= 16 tokens, one persistent CTA per SM with the
     tokens' rows resident in shared memory; see csrc/gemm_stream.cu.  Without `norm_weight`, x = a (bfloat16);
     with it, a is 32-bit and x = RMSNorm(a; norm_weight, eps) rounded to bfloat16, computed inside the kernel.
-    `activation` (STORE: ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED or ACT_RELU, applied to the 32-bit result before it is
+    `activation` (STORE: ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED or ACT_XIELU with `act_constants`, applied to the 32-bit result before it is
     stored; SWIGLU: ACT_RELU makes the gate a ReLU)."""
     M, K = a.shape
     N = out.shape[1]
@@ -494,8 +529,7 @@ def gemm_stream(mode, a, w, out, alpha: float = 1.0, error_flag=None, label=None
     with _timed("gemm_stream", label, work=lambda: _gemm_work(a, w, out)):
         _check(lib().lia_gemm_stream(mode, x, ldx, _p(w), w.stride(0), _p(out), dtype_code(out.dtype), out.stride(0),
                                      M, N, K, alpha, src, ld_src, nw, nw_code, eps, sms, stages_cap, early_stages, int(activation),
-                                     _p(error_flag),
-                                     _stream()), "gemm_stream")
+                                     float(act_constants[0]), float(act_constants[1]), _p(error_flag), _stream()), "gemm_stream")
 
 
 ATTENTION_HEAD_DIM_STEP, ATTENTION_HEAD_DIM_MAX = 16, 256      # what csrc/attention_generic.cu takes
@@ -849,7 +883,7 @@ def sigmoid_attention_tc(q, k_pages, v_pages, segments, n_segments, portion_tile
 # ---- parts of decoders with a norm on both sides of a sublayer, attention through a latent, attention with a sink,
 # ---- and a recurrent mixer with input-dependent decay
 
-ACT_NONE, ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED, ACT_RELU = 0, 1, 2, 3, 4
+ACT_NONE, ACT_GELU_TANH, ACT_SILU, ACT_RELU_SQUARED, ACT_RELU, ACT_XIELU = 0, 1, 2, 3, 4, 5
 
 
 def _f32(*tensors):
@@ -873,17 +907,52 @@ def norm_residual(y, weight, residual, eps: float, bias=None, next_weight=None, 
                                        next_eps, _stream()), "norm_residual")
 
 
-def activation_rows(source, out, act: int = ACT_NONE, gated: bool = False):
+class NormTerm:
+    """One of the rows that `norm_terms_residual` adds up: scale * rms(rows + bias) * weight, or scale * (rows + bias) without a
+    weight (rows, bias and weight 32-bit)."""
+    __slots__ = ("rows", "bias", "weight", "scale", "eps")
+
+    def __init__(self, rows, bias=None, weight=None, scale: float = 1.0, eps: float = 0.0):
+        self.rows, self.bias, self.weight, self.scale, self.eps = rows, bias, weight, float(scale), float(eps)
+
+
+def norm_terms_residual(terms, weight, residual, eps: float, next_out=None):
+    """residual += rms(sum of one or two `NormTerm`s) * weight; with `next_out` also next_out = the new residual in its element
+    type, in one pass over the rows; see csrc/norm_residual.cu."""
+    rows, hidden = residual.shape
+    if not 1 <= len(terms) <= 2:
+        raise KernelError("norm_terms_residual takes one or two terms")
+    _cuda(weight, residual, next_out)
+    _f32(weight, residual)
+    for term in terms:
+        _cuda(term.rows, term.bias, term.weight)
+        _f32(term.rows, term.bias, term.weight)
+        if tuple(term.rows.shape) != (rows, hidden) or any(v is not None and v.numel() != hidden for v in (term.bias, term.weight)):
+            raise KernelError("norm_terms_residual: rows of one width, weights and biases of that width")
+    if weight.numel() != hidden or (next_out is not None and tuple(next_out.shape) != (rows, hidden)):
+        raise KernelError("norm_terms_residual: rows of one width, weights and biases of that width")
+    args = []
+    for i in range(2):
+        t = terms[i] if i < len(terms) else None
+        args += [_p(t.rows), _p(t.bias), _p(t.weight), t.scale, t.eps] if t is not None else [None, None, None, 0.0, 0.0]
+    nbytes = rows * hidden * (4 * (len(terms) + 2) + (next_out.element_size() if next_out is not None else 0))
+    with _timed("norm_terms_residual", nbytes=nbytes):
+        _check(lib().lia_norm_terms_residual(*args, _p(weight), _p(residual), _p(next_out),
+                                             dtype_code(next_out.dtype) if next_out is not None else F32, rows, hidden,
+                                             float(eps), _stream()), "norm_terms_residual")
+
+
+def activation_rows(source, out, act: int = ACT_NONE, gated: bool = False, constants=(0.0, 0.0)):
     """out[r, :] = act(source[r, :]) for 32-bit rows `source` (any row stride); with `gated` the rows hold a gate half and
-    then another half of out's width, out = act(gate) * the other half; see csrc/norm_residual.cu."""
+    then another half of out's width, out = act(gate) * the other half; `constants`: ACT_XIELU's; see csrc/norm_residual.cu."""
     if not (source.is_cuda and out.is_cuda) or source.dtype != torch.float32 or source.dim() != 2 or out.dim() != 2 or \
             source.shape[0] != out.shape[0] or source.shape[1] != (2 if gated else 1) * out.shape[1] or \
             source.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("activation_rows: 32-bit rows in, rows of the same shape (gated: of half the width) out")
     with _timed("activation_rows", nbytes=source.numel() * 4 + out.numel() * out.element_size()):
         _check(lib().lia_activation_rows(_p(source), source.stride(0), _p(out), dtype_code(out.dtype), out.stride(0),
-                                         out.shape[0], out.shape[1], int(act), 1 if gated else 0, _stream()),
-               "activation_rows")
+                                         out.shape[0], out.shape[1], int(act), 1 if gated else 0, float(constants[0]), float(constants[1]),
+                                         _stream()), "activation_rows")
 
 
 def attention_general(q1, q1_strides, q2, q2_strides, k1_pages, k2_pages, v_pages, v_stride, dv, positions, slots,
@@ -1384,3 +1453,120 @@ def gla(rows, log_decay, state, segments, n_segments: int, max_chunks: int, sing
                              dtype_code(out.dtype), heads, d, dv, float(eps), _p(scratch),
                              0 if scratch is None else scratch.numel(), _p(w_a2), F32 if w_a2 is None else dtype_code(w_a2.dtype),
                              _p(bias), 0 if w_a2 is None else w_a2.shape[1], float(q_scale), float(tau), _stream()), "gla")
+
+
+# ---- short convolutions over a ring, the real-gated linear recurrent unit and the state-space recurrence with one decay a
+# ---- head: csrc/ring_conv.cu, csrc/rglru.cu, csrc/state_space.cu
+RING_MAX_TAPS = 8
+SSD_MAX_HEAD = 256
+RGLRU_MAX_BLOCK = 6400
+
+
+def _slots_of(t, shape, what):
+    """`t` [slots, *shape], 32-bit, each slot's part contiguous: its slot stride."""
+    if t.dtype != torch.float32 or tuple(t.shape[1:]) != tuple(shape) or not t[0].is_contiguous():
+        raise KernelError(f"{what}: the state is 32-bit [slots, {', '.join(map(str, shape))}], contiguous per slot")
+    return t.stride(0)
+
+
+def ring_conv(x, in_bias, weight, bias, ring, positions, slots, out, act: int = 0):
+    """out[t, c] = act(bias[c] + sum_j weight[j, c] (x[t - taps + 1 + j, c] + in_bias[c])) along each request's run, earlier
+    inputs from `ring` [slots, taps, channels] (position p's input in row p % taps, in_bias included), zero before the start;
+    x 32-bit rows (the first `channels` columns); act 1: SiLU.  The ring is read, not changed."""
+    _cuda(in_bias, weight, bias, positions, slots, out)
+    _f32(x, in_bias, weight, bias)
+    n, channels = out.shape
+    taps = weight.shape[0]
+    if x.stride(1) != 1 or x.shape[0] != n or x.shape[1] < channels or weight.shape[1] != channels:
+        raise KernelError("ring_conv: rows of at least `channels` columns, weight [taps, channels]")
+    stride = _slots_of(ring, (taps, channels), "ring_conv") if taps > 1 else 0
+    with _timed("ring_conv", nbytes=n * channels * (4 + out.element_size())):
+        _check(lib().lia_ring_conv(_p(x), x.stride(0), _p(in_bias), _p(weight), _p(bias), _p(ring) if taps > 1 else None, stride,
+                                   _p(positions), _p(slots), _p(out), dtype_code(out.dtype), n, channels, taps, int(act),
+                                   _stream()), "ring_conv")
+
+
+def ring_store(x, in_bias, ring, positions, slots):
+    """The inputs x[t, c] + in_bias[c] of every run's last tokens into the slots' rings."""
+    _cuda(in_bias, positions, slots)
+    _f32(x, in_bias)
+    taps, channels = ring.shape[1], ring.shape[2]
+    if x.stride(1) != 1 or x.shape[1] < channels:
+        raise KernelError("ring_store: rows of at least `channels` columns")
+    with _timed("ring_store"):
+        _check(lib().lia_ring_store(_p(x), x.stride(0), _p(in_bias), _p(ring), _slots_of(ring, (taps, channels), "ring_store"),
+                                    _p(positions), _p(slots), x.shape[0], channels, taps, _stream()), "ring_store")
+
+
+def rglru_gates(u, weight, bias, rate, slots, a_out, inflow, blocks: int):
+    """r, i = sigmoid of u's parts through weight [blocks, size, 2 size] ([in][r's outputs | i's outputs]) plus bias
+    [2, width]; a_out = exp(-rate r), inflow = sqrt(1 - a_out^2) i u (32-bit), on the 32-bit pipes; see csrc/rglru.cu."""
+    _cuda(u, weight, bias, rate, slots, a_out, inflow)
+    _f32(bias, rate, a_out, inflow)
+    n, width = u.shape
+    size = width // blocks
+    if tuple(weight.shape) != (blocks, size, 2 * size) or tuple(a_out.shape) != (n, width) or tuple(inflow.shape) != (n, width) \
+            or bias.numel() != 2 * width or rate.numel() != width or u.dtype != weight.dtype:
+        raise KernelError("rglru_gates: shapes or element types do not agree")
+    with _timed("rglru_gates", nbytes=n * width * (u.element_size() + 8) + weight.numel() * weight.element_size(),
+                flops=4 * n * width * size):
+        _check(lib().lia_rglru_gates(_p(u), dtype_code(u.dtype), _p(weight), dtype_code(weight.dtype), _p(bias), _p(rate),
+                                     _p(slots), _p(a_out), _p(inflow), n, width, int(blocks), _stream()), "rglru_gates")
+
+
+def rglru_scan(a, inflow, y, x, y_bias, x_bias, ring, state, segments, n_segments: int, single_rows, positions, slots, out,
+               taps: int):
+    """S <- a S + inflow per channel along the step's runs, out = S * gelu(y + y_bias); state [slots, width] 32-bit; the
+    convolution's last inputs x + x_bias go to ring [slots, taps, width]; see csrc/rglru.cu."""
+    _cuda(a, inflow, y_bias, x_bias, segments, single_rows, positions, slots, out)
+    _f32(a, inflow, y, x, y_bias, x_bias)
+    n, width = out.shape
+    n_single = 0 if single_rows is None else single_rows.numel()
+    if y.stride(1) != 1 or x.stride(1) != 1 or y.stride(0) != x.stride(0) or tuple(a.shape) != (n, width) or \
+            tuple(inflow.shape) != (n, width):
+        raise KernelError("rglru_scan: shapes do not agree")
+    stride = _slots_of(state, (width,), "rglru_scan")
+    if taps > 1 and _slots_of(ring, (taps, width), "rglru_scan") != stride:
+        raise KernelError("rglru_scan: ring and state must have one slot stride")
+    with _timed("rglru_scan", nbytes=n * width * (12 + out.element_size())):
+        _check(lib().lia_rglru_scan(_p(a), _p(inflow), _p(y), _p(x), y.stride(0), _p(y_bias), _p(x_bias),
+                                    _p(ring) if taps > 1 else None, _p(state), stride, _p(segments), int(n_segments),
+                                    _p(single_rows), n_single, _p(positions), _p(slots), _p(out), dtype_code(out.dtype), width,
+                                    int(taps), _stream()), "rglru_scan")
+
+
+def ssd_scratch_floats(chunks: int, heads: int, states: int, size: int) -> int:
+    return chunks * heads * (states * size + 1)
+
+
+def ssd(xbc, dt, dt_bias, rate, skip, state, segments, n_segments: int, max_chunks: int, single_rows, slots, y, heads: int,
+        groups: int, states: int, size: int, scratch=None):
+    """S <- exp(-rate dt) S + dt B x^T, y = S^T C + skip x per head with dt = softplus(dt + dt_bias), along the step's runs;
+    xbc [n, heads size + 2 groups states] = [x | B | C], dt [n, heads] columns of wider rows, state [slots, heads, states,
+    size], y [n, heads size]: all 32-bit; see csrc/state_space.cu."""
+    _cuda(dt_bias, rate, skip, segments, single_rows, slots, y, scratch)
+    _f32(xbc, dt, dt_bias, rate, skip, y, scratch)
+    n = y.shape[0]
+    n_single = 0 if single_rows is None else single_rows.numel()
+    if xbc.stride(1) != 1 or dt.stride(1) != 1 or xbc.shape[1] != heads * size + 2 * groups * states or dt.shape[1] != heads or \
+            xbc.shape[0] != n or dt.shape[0] != n or y.shape[1] != heads * size:
+        raise KernelError("ssd: shapes do not agree")
+    stride = _slots_of(state, (heads, states, size), "ssd")
+    with _timed("ssd", nbytes=n * heads * size * 8 + 2 * n_single * heads * states * size * 4,
+                flops=4 * n * heads * states * size):
+        _check(lib().lia_ssd(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(rate), _p(skip), _p(state), stride,
+                             _p(segments), int(n_segments), int(max_chunks), _p(single_rows), n_single, _p(slots), _p(y), heads,
+                             groups, states, size, _p(scratch), 0 if scratch is None else scratch.numel(), _stream()), "ssd")
+
+
+def gated_group_norm(y, z, weight, slots, out, groups: int, eps: float):
+    """out = rms(y * silu(z)) * weight over each of `groups` equal parts of a row; y, z (columns of wider rows) and weight
+    32-bit; see csrc/state_space.cu."""
+    _cuda(y, weight, slots, out)
+    _f32(y, z, weight)
+    n, width = out.shape
+    if tuple(y.shape) != (n, width) or tuple(z.shape) != (n, width) or z.stride(1) != 1 or weight.numel() != width or width % groups:
+        raise KernelError("gated_group_norm: shapes do not agree")
+    with _timed("gated_group_norm", nbytes=n * width * (8 + out.element_size())):
+        _check(lib().lia_gated_group_norm(_p(y), _p(z), z.stride(0), _p(weight), _p(slots), _p(out), dtype_code(out.dtype), n,
+                                          int(groups), width // groups, float(eps), _stream()), "gated_group_norm")

@@ -42,6 +42,7 @@ class ModelSpec:
     final_norm_prefix: str = "model.norm."
     eos_token_ids: tuple = ()
     position_table_name: Optional[str] = None       # a learned vector per position [max_positions, hidden], added to the embedding
+    sinusoidal_base: Optional[float] = None         # a sinusoidal vector of the position is added to the embedding: sine of p * base^(-2i/hidden) in column 2i, cosine in 2i + 1
     junctions: dict = field(default_factory=dict)   # schedule position -> PartSpec of a junction that runs ahead of that entry
     streams: int = 1                                # copies of the residual stream in a token's row (hyper-connections); all start as the embedding output, their sum goes to the final norm
     logit_softcap: Optional[float] = None           # logits <- cap * tanh(logits / cap)
@@ -60,6 +61,9 @@ class ModelSpec:
                 raise ValueError(f"the model keeps {self.streams} residual streams; a layer's arrangement keeps another number")
         if self.streams != 1 and self.junctions:
             raise ValueError("junctions act on a single residual stream")
+        if self.sinusoidal_base is not None and (not float(self.sinusoidal_base) > 0 or self.position_table_name is not None or
+                                                 self.streams != 1):
+            raise ValueError("sinusoidal_base must be positive, without a position table and with a single residual stream")
         if self.logit_softcap is not None and not float(self.logit_softcap) > 0:
             raise ValueError("logit_softcap must be positive")
         for position, junction in self.junctions.items():
@@ -141,6 +145,10 @@ class DecoderModel:
         self.position_table = None
         if spec.position_table_name is not None:
             self.position_table = prepare_weight(tensors[spec.position_table_name].to(device), runtime)
+        self.position_frequencies = None
+        if spec.sinusoidal_base is not None:
+            exponents = -2.0 * torch.arange((spec.hidden_size + 1) // 2, dtype=torch.float64) / spec.hidden_size
+            self.position_frequencies = (float(spec.sinusoidal_base) ** exponents).to(torch.float32).to(device)
         self.junctions = {}
         for position, junction in spec.junctions.items():
             cls = lookup(JUNCTIONS, junction.kind, "junction")
@@ -194,10 +202,19 @@ class DecoderModel:
         streams = spec.streams
         h = ctx.buffer("model.h", (n, streams * spec.hidden_size), torch.float32)
         first = ctx.buffer("model.h0", (n, spec.hidden_size), torch.float32) if self._keeps_first else None
+        rounded = None
         if streams > 1:
             if self.position_table is not None:
                 raise ValueError("a position table with several residual streams is not built")
             rt.ops.embedding_streams(ctx.tokens, self.embedding, h, streams, spec.embedding_scale, ctx.error_flag)
+        elif self.position_frequencies is not None:
+            # (a first layer that reads the stream itself gets it in the compute element type from the same kernel)
+            if rt.compute_dtype != torch.float32 and self.layers[spec.schedule[0].layer].reads_stream:
+                rounded = ctx.buffer("block.x", (n, spec.hidden_size), rt.compute_dtype)
+            rt.ops.embedding_sinusoidal(ctx.tokens, ctx.positions, self.embedding, self.position_frequencies, h,
+                                        spec.embedding_scale, copy=rounded, error_flag=ctx.error_flag)
+            if first is not None:
+                first.copy_(h)
         elif self.position_table is not None:
             rt.ops.embedding_positions(ctx.tokens, ctx.positions, self.embedding, self.position_table, h,
                                        spec.embedding_scale, copy=first, error_flag=ctx.error_flag)
@@ -205,6 +222,7 @@ class DecoderModel:
             rt.ops.embedding(ctx.tokens, self.embedding, h, spec.embedding_scale, ctx.error_flag)
             if first is not None:
                 first.copy_(h)
+        ctx.rounded_stream = rounded
         picked = None
         last = len(spec.schedule) - 1
         for position, entry in enumerate(spec.schedule):
@@ -214,6 +232,7 @@ class DecoderModel:
                 owed[0].settle(ctx, h)
             if junction is not None:
                 junction.forward(ctx, h, first)
+                ctx.rounded_stream = None
             kv = ctx.kv_view(entry.cache, entry.writes) if entry.cache is not None else None
             layer = self.layers[entry.layer]
             more = {"own_state": ctx.state(("layer", position))} if self._own_state[position] else {}
@@ -221,6 +240,8 @@ class DecoderModel:
                 picked = layer.forward(ctx, h, kv=kv, state=ctx.state(position), rows=ctx.out_rows, n_rows=ctx.n_out, **more)
             else:
                 layer.forward(ctx, h, kv=kv, state=ctx.state(position), **more)
+            if not getattr(layer, "reads_stream", False):
+                ctx.rounded_stream = None
         owed = getattr(ctx, "owed", None)
         if owed is not None:
             if ctx.n_out > 0:

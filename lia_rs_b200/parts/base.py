@@ -175,6 +175,9 @@ class Mixer(Part):
     # True: `forward` takes `store=True` and then WRITES scale * mixer(x) into `residual` instead of adding to it (its
     # last product stores); an arrangement that gives the part a buffer of its own then need not clear it first.
     can_store = False
+    # True: the mixer's result is a sum that it leaves to the arrangement: `output_terms` stands in for `forward` (an
+    # arrangement that norms the mixer's output takes both; the others refuse such a mixer).
+    gives_terms = False
 
     @staticmethod
     def cache_request(params: dict) -> Optional[KVCacheRequest]:
@@ -187,6 +190,10 @@ class Mixer(Part):
     def forward(self, ctx, x: torch.Tensor, residual: torch.Tensor, scale: float, kv=None, state=None):
         """residual += scale * mixer(x).  `kv` is the layer's `cache.KVView` (or None), `state`
         the tensor [slots, *shape] of its per-request state (or None)."""
+        raise NotImplementedError
+
+    def output_terms(self, ctx, x, kv=None, state=None) -> list:
+        """One or two `ops.NormTerm`s whose sum is mixer(x) (their rows lie in step buffers)."""
         raise NotImplementedError
 
 
@@ -238,6 +245,10 @@ class Arrangement:
 
     # True: `forward` takes `rows` / `n_rows` and then returns the residual rows of those tokens alone.
     supports_rows = False
+    # True: the layer reads the stream itself and not a norm of it, and leaves `ctx.rounded_stream`: the stream's rows in the
+    # compute element type (bfloat16) as they are behind the layer, or None.  The model offers the embedding output's to a
+    # first layer that says so and drops what a layer of another kind has made stale.
+    reads_stream = False
 
     def forward(self, ctx, residual: torch.Tensor, kv=None, state=None, rows=None, n_rows=None):
         """Run the layer on the residual stream in place.  With `rows` (device int32 batch indices, `n_rows` of

@@ -1,6 +1,6 @@
 """Arrangements of a layer's parts.
 
-`sandwich` (a norm before and after each sublayer) and `parallel` are described at their classes.
+`sandwich` (a norm before and after each sublayer), `postnorm` (a norm after each sublayer alone) and `parallel` are described at their classes.
 
 `prenorm`: r = h + s * mixer(norm1(h)); h' = r + s * ffn(norm2(r))
 (src/inference/llama_fusion.rs:41-117; s is MiniCPM's scale_depth / sqrt(layers), 1 for plain
@@ -70,6 +70,8 @@ class PreNormBlock(Arrangement):
         self.graph_safe = all(part.graph_safe for part in (self.norm1, self.mixer, self.norm2, self.feed_forward))
         if self.mixer.output_bias is not None:
             raise ValueError("the pre-norm arrangement does not add a mixer's output bias")
+        if self.mixer.gives_terms:
+            raise ValueError("the pre-norm arrangement does not add up a mixer's terms")
 
     def graph_key(self, ctx) -> tuple:
         return (self.norm1.graph_key(ctx) + self.mixer.graph_key(ctx) + self.norm2.graph_key(ctx) +
@@ -158,6 +160,8 @@ class SandwichBlock(Arrangement):
                 if record is None:
                     raise ValueError("the sandwich arrangement needs RMS norms")
                 self.post[place] = (record[0].to(torch.float32).contiguous(), float(record[1]))
+        if self.mixer.gives_terms:
+            raise ValueError("the sandwich arrangement does not add up a mixer's terms")
         self.graph_safe = all(part.graph_safe for part in parts.values())
         self._parts = list(parts.values())
 
@@ -196,6 +200,125 @@ class SandwichBlock(Arrangement):
             self.feed_forward.forward(ctx, x, y, 1.0)
         weight, eps = self.post["norm2b"]
         ops.norm_residual(y, weight, residual, eps)
+        return None
+
+
+@register_arrangement("postnorm")
+class PostNormBlock(Arrangement):
+    """A norm on each sublayer's output, none on its input:
+
+        x <- x + norm1(mixer(x));   x <- x + norm2(feed_forward(x))
+
+    The sublayer's output goes to 32-bit rows of its own (or stays the terms of a sum, `Mixer.output_terms`); one kernel
+    norms it, adds it to the stream and leaves the new stream in the compute element type for the product that reads it
+    next, in this layer or the one behind it (`ctx.rounded_stream`; csrc/norm_residual.cu).  The norms must be RMS norms
+    (`rms_record`).  The feed-forward may be absent.  A mixer's `output_bias` is added ahead of its norm.  `residual_scale`
+    has no meaning here (a norm follows the sublayer) and must be 1.  Checkpoint names: `names["norm1"]`, `["mixer"]`,
+    `["norm2"]`, `["feed_forward"]`."""
+    supports_rows = True
+    reads_stream = True
+
+    @staticmethod
+    def _classes(spec: LayerSpec):
+        """[(class, params, place)] of the norms that exist, the mixer and the feed-forward."""
+        places = ("norm1", "norm2") if spec.feed_forward is not None else ("norm1",)
+        out = [(lookup(NORMS, spec.norm_at(p).kind, "norm"), spec.norm_at(p).params, p) for p in places]
+        out.append((lookup(MIXERS, spec.mixer.kind, "mixer"), spec.mixer.params, "mixer"))
+        if spec.feed_forward is not None:
+            out.append((lookup(FEED_FORWARDS, spec.feed_forward.kind, "feed-forward"), spec.feed_forward.params, "feed_forward"))
+        return out
+
+    @staticmethod
+    def check(spec: LayerSpec) -> None:
+        for cls, params, _ in PostNormBlock._classes(spec):
+            cls.check_params(params)
+        if float(spec.residual_scale) != 1.0:
+            raise ValueError("the post-norm arrangement takes no residual scale")
+
+    @staticmethod
+    def tensor_specs(spec: LayerSpec, prefix: str) -> list:
+        specs = [t for cls, params, place in PostNormBlock._classes(spec) for t in cls.tensor_specs(params, prefix + spec.names[place])]
+        if spec.feed_forward is None:
+            # a checkpoint may carry the norm of the absent sublayer all the same: taken if there, never used
+            norm = spec.norm_at("norm2")
+            specs += [TensorSpec(t.name, t.shape, t.kind, optional=True)
+                      for t in lookup(NORMS, norm.kind, "norm").tensor_specs(norm.params, prefix + spec.names["norm2"])]
+        return specs
+
+    def __init__(self, spec: LayerSpec, tensors: dict, prefix: str, runtime):
+        self.runtime = runtime
+        parts = {place: cls(params, tensors, prefix + spec.names[place], runtime) for cls, params, place in self._classes(spec)}
+        self.mixer, self.feed_forward = parts["mixer"], parts.get("feed_forward")
+        self.post = {}
+        for place in ("norm1", "norm2"):
+            if place in parts:
+                record = parts[place].rms_record()
+                if record is None:
+                    raise ValueError("the post-norm arrangement needs RMS norms")
+                self.post[place] = (record[0].to(torch.float32).contiguous(), float(record[1]))
+        self.graph_safe = all(part.graph_safe for part in parts.values())
+        self._parts = list(parts.values())
+
+    def graph_key(self, ctx) -> tuple:
+        key = ()
+        for part in self._parts:
+            key += part.graph_key(ctx)
+        return key
+
+    def _join(self, ctx, terms, place, residual, last: bool):
+        """residual += norm(sum of the terms); returns the new stream in the compute element type (None where `last` and
+        nobody reads it)."""
+        weight, eps = self.post[place]
+        if self.runtime.compute_dtype == torch.float32:
+            self.runtime.ops.norm_terms_residual(terms, weight, residual, eps)
+            return residual
+        rounded = None if last else ctx.buffer("block.x", tuple(residual.shape), self.runtime.compute_dtype)
+        self.runtime.ops.norm_terms_residual(terms, weight, residual, eps, next_out=rounded)
+        return rounded
+
+    def forward(self, ctx, residual, kv=None, state=None, rows=None, n_rows=None):
+        ops = self.runtime.ops
+        x = getattr(ctx, "rounded_stream", None)
+        if self.runtime.compute_dtype == torch.float32:
+            x = residual
+        elif x is None:
+            x = ctx.buffer("block.x", tuple(residual.shape), self.runtime.compute_dtype)
+            ops.activation_rows(residual, x, ops.ACT_NONE)
+        ctx.rounded_stream = None
+        if self.mixer.gives_terms:
+            terms = self.mixer.output_terms(ctx, x, kv=kv, state=state)
+        else:
+            y = ctx.buffer("block.sublayer", tuple(residual.shape), torch.float32)
+            if self.mixer.can_store:
+                self.mixer.forward(ctx, x, y, 1.0, kv=kv, state=state, store=True)
+            else:
+                y.zero_()
+                self.mixer.forward(ctx, x, y, 1.0, kv=kv, state=state)
+            terms = [ops.NormTerm(y, bias=self.mixer.output_bias)]
+        if rows is not None:
+            # only `rows` matter after this layer: cache and state are up to date for every token, the rest runs on the
+            # picked rows alone
+            picked = ctx.buffer("block.picked", (n_rows, residual.shape[1]), residual.dtype)
+            if not n_rows:
+                return picked
+            ops.gather_rows(residual, rows, picked)
+            for i, term in enumerate(terms):
+                chosen = ctx.buffer(f"block.picked_term{i}", tuple(picked.shape), torch.float32)
+                ops.gather_rows(term.rows, rows, chosen)
+                term.rows = chosen
+            residual = picked
+        x = self._join(ctx, terms, "norm1", residual, last=self.feed_forward is None and rows is not None)
+        if self.feed_forward is not None:
+            y = ctx.buffer("block.sublayer", tuple(residual.shape), torch.float32)
+            if self.feed_forward.can_store:
+                self.feed_forward.forward(ctx, x, y, 1.0, store=True)
+            else:
+                y.zero_()
+                self.feed_forward.forward(ctx, x, y, 1.0)
+            x = self._join(ctx, [ops.NormTerm(y)], "norm2", residual, last=rows is not None)
+        if rows is not None:
+            return residual
+        ctx.rounded_stream = x if self.runtime.compute_dtype != torch.float32 else None
         return None
 
 
@@ -275,6 +398,8 @@ class ParallelBlock(Arrangement):
         self.graph_safe = all(part.graph_safe for part in parts)
         if self.mixer.output_bias is not None:
             raise ValueError("the parallel arrangement does not add a mixer's output bias")
+        if self.mixer.gives_terms:
+            raise ValueError("the parallel arrangement does not add up a mixer's terms")
 
     def graph_key(self, ctx) -> tuple:
         key = self.norm.graph_key(ctx) + self.mixer.graph_key(ctx)

@@ -60,7 +60,9 @@ class SwiGLU(FeedForward):
 @register_feed_forward("dense_act")
 class DenseActivation(FeedForward):
     """Dense feed-forward without a gate: f = Wd act(Wu x), no biases.  `activation`: "gelu_tanh"
-    (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), "silu", "relu_squared" (relu(z)^2), "relu" or "none".  The activation is taken of the up product's
+    (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), "silu", "relu_squared" (relu(z)^2), "relu", "xielu" or "none".
+    xIELU has two stored numbers p, q (tensor `names["act"]` [2]): softplus(p) z^2 + z/2 for z > 0, else (1/2 + softplus(q))
+    (exp(z) - 1 - z) + z/2; the two constants are formed once, at load, in 32-bit.  The activation is taken of the up product's
     32-bit result and rounded once to the compute element type: in the product's epilogue where the kernel can (the
     few-token persistent product), else by a kernel of its own on the product's 32-bit rows; the down product adds into
     the residual stream.  Parameters: hidden, intermediate, activation, and optionally `names`: the checkpoint names of the up and
@@ -68,8 +70,8 @@ class DenseActivation(FeedForward):
     graph_safe = True
     takes_deferred_norm = True
     can_store = True
-    NAMES = {"up": "up_proj.weight", "down": "down_proj.weight"}
-    ACTIVATIONS = {"none": 0, "gelu_tanh": 1, "silu": 2, "relu_squared": 3, "relu": 4}
+    NAMES = {"up": "up_proj.weight", "down": "down_proj.weight", "act": "act"}
+    ACTIVATIONS = {"none": 0, "gelu_tanh": 1, "silu": 2, "relu_squared": 3, "relu": 4, "xielu": 5}
 
     def graph_key(self, ctx) -> tuple:
         return ()
@@ -77,7 +79,7 @@ class DenseActivation(FeedForward):
     @staticmethod
     def _names(params, prefix):
         names = {**DenseActivation.NAMES, **params.get("names", {})}
-        return prefix + names["up"], prefix + names["down"]
+        return prefix + names["up"], prefix + names["down"], prefix + names["act"]
 
     @staticmethod
     def check_params(params):
@@ -88,15 +90,20 @@ class DenseActivation(FeedForward):
     @staticmethod
     def tensor_specs(params, prefix):
         h, i = params["hidden"], params["intermediate"]
-        up, down = DenseActivation._names(params, prefix)
-        return [TensorSpec(up, (i, h)), TensorSpec(down, (h, i))]
+        up, down, act = DenseActivation._names(params, prefix)
+        constants = [TensorSpec(act, (2,))] if params.get("activation") == "xielu" else []
+        return [TensorSpec(up, (i, h)), TensorSpec(down, (h, i))] + constants
 
     def __init__(self, params, tensors, prefix, runtime):
         super().__init__(params, tensors, prefix, runtime)
         self.check_params(params)
         self.hidden, self.intermediate = int(params["hidden"]), int(params["intermediate"])
         self.activation = self.ACTIVATIONS[params.get("activation", "gelu_tanh")]
-        up, down = self._names(params, prefix)
+        up, down, act = self._names(params, prefix)
+        self.constants = (0.0, 0.0)
+        if self.activation == self.ACTIVATIONS["xielu"]:
+            raised = torch.nn.functional.softplus(tensors[act].to("cpu", torch.float32))
+            self.constants = (float(raised[0]), 0.5 + float(raised[1]))
         self.w_up = prepare_weight(tensors[up], runtime)
         self.w_down = prepare_weight(tensors[down], runtime)
 
@@ -107,6 +114,6 @@ class DenseActivation(FeedForward):
         if self.activation == 0:
             linear(rt, STORE, x, self.w_up, act, error_flag=ctx.error_flag, name="up")
         elif not linear(rt, STORE, x, self.w_up, act, error_flag=ctx.error_flag, name="up", activation=self.activation,
-                        unactivated=up):
-            rt.ops.activation_rows(up, act, self.activation)
+                        unactivated=up, activation_constants=self.constants):
+            rt.ops.activation_rows(up, act, self.activation, constants=self.constants)
         linear(rt, STORE if store else ACCUM, act, self.w_down, residual, scale, error_flag=ctx.error_flag, name="down")

@@ -58,7 +58,8 @@ def _choose(mode, a, w, out) -> int:
 
 
 def linear(runtime, mode: int, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float = 1.0,
-           error_flag=None, name=None, activation: int = 0, unactivated: torch.Tensor = None, gate_activation: int = 0):
+           error_flag=None, name=None, activation: int = 0, unactivated: torch.Tensor = None, gate_activation: int = 0,
+           activation_constants=(0.0, 0.0)):
     """`name`: what the product is to its caller ("qkv", "down", ...), for the per-kernel-class profile.
     `error_flag` (int32[1] on the device, a step's `ctx.error_flag`): a tensor-core kernel that gives up on one
     of its bounded waits raises it to 3, and the step's caller then learns that the result is not to be used.
@@ -66,7 +67,7 @@ def linear(runtime, mode: int, a: torch.Tensor, w: torch.Tensor, out: torch.Tens
     kernel applies it in its epilogue and the call returns True; where another kernel serves the product, the plain
     product goes to `unactivated` (32-bit rows of out's shape) instead of `out`, the call returns False and the
     activation is the caller's (`ops.activation_rows`): nothing is rounded ahead of the activation either way (the squared
-    ReLU is also applied by the persistent tcgen05 kernel).
+    ReLU and xIELU, with its two `activation_constants`, are also applied by the persistent tcgen05 kernel).
     `gate_activation` (SWIGLU only; `ops.ACT_RELU`): out = up * relu(gate) instead of up * silu(gate), in the epilogue of
     the persistent few-token kernel, of the persistent tcgen05 kernel and of the product on the 32-bit pipes."""
     if gate_activation and (mode != SWIGLU or gate_activation != ops.ACT_RELU):
@@ -87,7 +88,7 @@ def linear(runtime, mode: int, a: torch.Tensor, w: torch.Tensor, out: torch.Tens
                                          and ops.gemm_stream_accepts(mode, source, w, out, norm=True))
             if fused:
                 ops.gemm_stream(mode, source, w, out, alpha, error_flag, label=name, norm_weight=norm_weight, eps=eps,
-                                activation=activation or gate_activation)
+                                activation=activation or gate_activation, act_constants=activation_constants)
                 return bool(activation)
         a = a.tensor()
     if a.dtype != torch.bfloat16:
@@ -100,11 +101,12 @@ def linear(runtime, mode: int, a: torch.Tensor, w: torch.Tensor, out: torch.Tens
     if choice is None:
         choice = _choices[key] = _choose(mode, a, w, out)
     if activation:
-        if choice == _STREAM and activation in (ops.ACT_GELU_TANH, ops.ACT_SILU, ops.ACT_RELU_SQUARED):
-            ops.gemm_stream(mode, a, w, out, alpha, error_flag, label=name, activation=activation)
+        if choice == _STREAM and activation in (ops.ACT_GELU_TANH, ops.ACT_SILU, ops.ACT_RELU_SQUARED, ops.ACT_XIELU):
+            ops.gemm_stream(mode, a, w, out, alpha, error_flag, label=name, activation=activation,
+                            act_constants=activation_constants)
             return True
-        if choice == _TC and activation == ops.ACT_RELU_SQUARED:
-            ops.gemm_tc(mode, a, w, out, alpha, error_flag, label=name, act=activation)
+        if choice == _TC and activation in (ops.ACT_RELU_SQUARED, ops.ACT_XIELU):
+            ops.gemm_tc(mode, a, w, out, alpha, error_flag, label=name, act=activation, act_constants=activation_constants)
             return True
         linear(runtime, mode, a, w, unactivated, alpha, error_flag=error_flag, name=name)
         return False

@@ -14,6 +14,8 @@
     a key of score 0 that has no value;
   * a cap on the scores (optional, `softcap`): s <- cap * tanh(s / cap) ahead of the softmax;
   * all keys j <= i, or the last `window` of them;
+  * an output gate (optional, `gate` "sigmoid"): the heads side by side are multiplied by sigmoid(W_g x) ahead of the output
+    projection;
   * an output projection whose bias (optional; `biases` "qkv": the three input projections have biases and the output
     projection none) is the mixer's `output_bias`.
 
@@ -72,7 +74,7 @@ class SinkAttention(Mixer):
     takes_deferred_norm = True
     can_store = True
     NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "o_bias": "o.b",
-             "q_norm": "q.norm", "k_norm": "k.norm", "mix": "vmix"}
+             "q_norm": "q.norm", "k_norm": "k.norm", "mix": "vmix", "gate": "g"}
 
     @staticmethod
     def _names(params, prefix):
@@ -94,6 +96,8 @@ class SinkAttention(Mixer):
             raise ValueError("attention: softcap must be positive or None")
         if params.get("biases") not in (None, False, True, "qkv") or params.get("qk_norm") not in (None, False, True, "whole"):
             raise ValueError("attention: biases is absent, True or 'qkv'; qk_norm is absent, True or 'whole'")
+        if params.get("gate") not in (None, "sigmoid"):
+            raise ValueError("attention: gate is None or 'sigmoid'")
         if params.get("softcap") is not None and params.get("sink"):
             raise ValueError("attention: a sink and a cap on the scores together are not built")
 
@@ -103,6 +107,8 @@ class SinkAttention(Mixer):
         n = SinkAttention._names(params, prefix)
         specs = [TensorSpec(n["q"], (nq * d, h)), TensorSpec(n["k"], (nkv * d, h)), TensorSpec(n["v"], (nkv * dv, h)),
                  TensorSpec(n["o"], (h, nq * dv))]
+        if params.get("gate"):
+            specs.append(TensorSpec(n["gate"], (nq * dv, h)))
         if params.get("biases"):
             specs += [TensorSpec(n["q_bias"], (nq * d,)), TensorSpec(n["k_bias"], (nkv * d,)),
                       TensorSpec(n["v_bias"], (nkv * dv,))]
@@ -132,8 +138,16 @@ class SinkAttention(Mixer):
         n = self._names(params, prefix)
         device = runtime.device
         used = (self.nq + self.nkv) * self.d + self.nkv * self.dv
-        self.width = (used + 7) // 8 * 8
         parts = [tensors[n["q"]], tensors[n["k"]], tensors[n["v"]]]
+        self.gate_at = None
+        if params.get("gate"):                        # the gate's rows behind q, k and v in the same product
+            pad = -used % 8
+            if pad:
+                parts.append(torch.zeros((pad, self.hidden), dtype=parts[0].dtype, device=parts[0].device))
+            parts.append(tensors[n["gate"]])
+            self.gate_at = used + pad
+            used = self.gate_at + self.nq * self.dv
+        self.width = (used + 7) // 8 * 8
         if self.width > used:
             parts.append(torch.zeros((self.width - used, self.hidden), dtype=parts[0].dtype, device=parts[0].device))
         self.w_in = prepare_weight(torch.cat(parts, dim=0), runtime)
@@ -179,6 +193,8 @@ class SinkAttention(Mixer):
             ops.attention_general(q, (nq * d, d), None, None, kv.k_pages, None, kv.v_pages, dv, dv, ctx.positions, ctx.slots,
                                   kv.block_table, o, (nq * dv, dv), n, nq, nkv, self.window, self.scale, sink=self.sink,
                                   error_flag=flag, softcap=self.softcap)
+        if self.gate_at is not None:
+            ops.gate_rows(o, projected[:, self.gate_at:self.gate_at + nq * dv], ops.GATE_SIGMOID)
         linear(rt, STORE if store else ACCUM, o, self.w_o, residual, scale, error_flag=flag, name="o")
 
 
