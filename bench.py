@@ -588,6 +588,42 @@ def pilutar_workload(steps, warmup) -> int:
                          ZIPELIX_SIZES, pilutar_pair, steps, warmup)
 
 
+# The Foduzen decoder beside the Pilutar, Vatunex and Llama decoders at equal sizes (--workload foduzen): four layers each.
+# Foduzen: two gated linear recurrent units (parts of 256 and 128 channels) and two layers of windowed, gated grouped-query
+# attention (window of 1,024; key and value heads of equal size at 2B-widths, of 64 and 128 at 0.5B-widths) beside a
+# state-space recurrence (inner size twice the width), each with a dense xIELU feed-forward.  Pilutar (mixers side by side:
+# windowed attention and a linear recurrence) and Vatunex (a short convolution, a scan, an ungated feed-forward) are the
+# closest models.
+FODUZEN_SIZES = {
+    "2B-widths": dict(ZIPELIX_SIZES["2B-widths"], key_dim=128, value_dim=128, rnn=2560, blocks=10, ssd_heads=64, ssd_size=64,
+                      ssd_state=128, ssd_groups=1),
+    "0.5B-widths": dict(ZIPELIX_SIZES["0.5B-widths"], key_dim=64, value_dim=128, rnn=1280, blocks=10, ssd_heads=32, ssd_size=64,
+                        ssd_state=64, ssd_groups=2),
+}
+FODUZEN_WINDOW = 1024
+
+
+def foduzen_pair(size: dict):
+    from lia_rs_b200.config import FoduzenConfig
+    dense = {"kind": "dense", "ff": size["ff"]}
+    unit = {"type": "rglru", "mlp": dense, "mixer": {"width": size["rnn"], "blocks": size["blocks"], "conv": 4}}
+    parallel = {"type": "parallel", "mlp": dense, "mixer": {
+        "left": {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": size["key_dim"], "vdim": size["value_dim"],
+                 "scale": size["key_dim"] ** -0.5, "mask": {"size": FODUZEN_WINDOW}},
+        "right": {"heads": size["ssd_heads"], "vdim": size["ssd_size"], "state": size["ssd_state"],
+                  "groups": size["ssd_groups"], "norm_groups": 1, "conv": 4}}}
+    foduzen = FoduzenConfig.from_dict({
+        "architecture": "Foduzen", "vocab": 8192, "width": size["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 16.0},
+        "layers": [unit, parallel, unit, parallel]})
+    others = pilutar_pair(size)
+    return {"foduzen": foduzen, "pilutar": others["pilutar"], "vatunex": vatunex_pair(size)["vatunex"], "llama": others["llama"]}
+
+
+def foduzen_workload(steps, warmup) -> int:
+    return pair_workload("foduzen", "Foduzen beside the Pilutar, Vatunex and Llama decoders at equal sizes, four layers, bf16",
+                         FODUZEN_SIZES, foduzen_pair, steps, warmup)
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -598,7 +634,7 @@ def main() -> int:
                         help="run fewer layers than the configuration's 40 (both numbers are reported)")
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--no-points", action="store_true", help="skip batch 1 and batch 64")
-    parser.add_argument("--workload", default=None, choices=["8b-decode", "8b-prefill", "0.5b-mixed", "nafevik", "vatunex", "zipelix", "pilutar"],
+    parser.add_argument("--workload", default=None, choices=["8b-decode", "8b-prefill", "0.5b-mixed", "nafevik", "vatunex", "zipelix", "pilutar", "foduzen"],
                         help="one of the family's other sizes on the workload it is quoted on (prints its own line)")
     parser.add_argument("--device-trace", action="store_true",
                         help="with --workload 0.5b-mixed: one more pass under a trace of the device's kernels; adds "
@@ -625,6 +661,8 @@ def main() -> int:
         return zipelix_workload(args.steps, args.warmup)
     if args.workload == "pilutar":
         return pilutar_workload(args.steps, args.warmup)
+    if args.workload == "foduzen":
+        return foduzen_workload(args.steps, args.warmup)
     if args.workload:
         return other_workload(args.workload, args.steps, args.warmup, trace=args.device_trace)
 

@@ -28,13 +28,13 @@ namespace {
 struct Params {
     const __nv_bfloat16* q;          // [tokens, nq, D]
     const __nv_bfloat16* k_pages;    // [pages, page_size, nkv, D]
-    const __nv_bfloat16* v_pages;
+    const __nv_bfloat16* v_pages;    // [pages, page_size, nkv, DV]
     const int* rows;                 // [n_rows] batch index of each decoded token (negative: skip)
     const int* positions;            // [tokens]
     const int* slots;                // [tokens]
     const int* block_table;          // [slots, table_stride]
-    __nv_bfloat16* out;              // [tokens, nq, D]
-    float* partial;                  // [tokens, nq, n_splits, D] normalised outputs, then [tokens, nq, n_splits] log2-sum-exps
+    __nv_bfloat16* out;              // [tokens, nq, DV]
+    float* partial;                  // [tokens, nq, n_splits, DV] normalised outputs, then [tokens, nq, n_splits] log2-sum-exps
     int* counters;                   // [n_rows, gridDim.y], zero between launches; null: ranges are merged by a second kernel
     int n_tokens, table_stride, nq, nkv, page_size, page_shift, window, split_len, n_splits;
     float scale_log2;                // softmax scale * log2(e); with a cap on the scores: cap * log2(e)
@@ -163,10 +163,13 @@ __device__ __forceinline__ void cluster_merge(const Params& p, uint8_t* smem, in
 
 // NH: groups of 8 query heads per kv head that the CTA serves (1 or 2); CAP: the scores pass a tanh cap (an instantiation
 // of its own, so that the kernel without a cap is what it was)
-template <int D, int NH, bool CAP = false>
+// D: the keys' head size, DV: the values' (the encoding and append inside the kernel take equal sizes only)
+template <int D, int DV, int NH, bool CAP = false>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_decode_kernel(Params p) {
     using T = Tile<D>;
+    using TV = Tile<DV>;
+    constexpr int STAGE_BYTES = T::BYTES + TV::BYTES;
     constexpr int CHUNKS = T::CHUNKS;                 // 16-byte pieces per key row = lanes that share a row
     constexpr int ROWS_PER_PASS = WARPS * 32 / CHUNKS; // rows that one cp.async of every thread covers
     constexpr int PASSES = TILE_KEYS / ROWS_PER_PASS;
@@ -194,9 +197,9 @@ attention_decode_kernel(Params p) {
     const int key_end = min(pos + 1, key_begin + split_len);
     if (key_begin >= key_end) {
         if (!p.cluster) return;
-        float* exchange = exchange_of<D>(smem);       // a range without keys: it says so and stays for the cluster's merge
-        if (tid < 16) exchange[16 * D + tid] = -INFINITY;
-        cluster_merge<D>(p, smem, t, h0, heads);
+        float* exchange = exchange_of<DV>(smem);       // a range without keys: it says so and stays for the cluster's merge
+        if (tid < 16) exchange[16 * DV + tid] = -INFINITY;
+        cluster_merge<DV>(p, smem, t, h0, heads);
         return;
     }
     const int* table = p.block_table + (size_t)slot * p.table_stride;
@@ -209,7 +212,7 @@ attention_decode_kernel(Params p) {
     static_assert(ROWS_PER_PASS % 8 == 0 && PASSES <= CHUNKS, "the swizzle repeats every 8 rows; one lane per pass");
     // `left_out`: a key whose row of the tile no copy touches (this CTA writes it into the tile itself)
     auto load_tile = [&](int stage, int key0, int left_out) {
-        const uint32_t ks = smem_base + (uint32_t)stage * 2 * T::BYTES + piece_offset, vs = ks + T::BYTES;
+        const uint32_t ks = smem_base + (uint32_t)stage * STAGE_BYTES + piece_offset, vs = ks + T::BYTES;
         constexpr int LEFT_OUT = -2147483647 - 1;         // no row of the cache: cache_row_of gives -1 or a row >= 0
         int my_row = -1;
         if (piece < PASSES) {
@@ -224,7 +227,29 @@ attention_decode_kernel(Params p) {
             const bool valid = row >= 0;
             const size_t src = ((size_t)(valid ? row : 0) * p.nkv + kvh) * D + piece * 8;
             cp_async_16(ks + (uint32_t)(i * ROWS_PER_PASS * CHUNKS * 16), p.k_pages + src, valid);
-            cp_async_16(vs + (uint32_t)(i * ROWS_PER_PASS * CHUNKS * 16), p.v_pages + src, valid);
+            if constexpr (D == DV) cp_async_16(vs + (uint32_t)(i * ROWS_PER_PASS * CHUNKS * 16), p.v_pages + src, valid);
+        }
+        if constexpr (D != DV) {
+            // values of another size than the keys: their pieces and passes are their own
+            constexpr int V_CHUNKS = TV::CHUNKS, V_ROWS = WARPS * 32 / V_CHUNKS, V_PASSES = TILE_KEYS / V_ROWS;
+            static_assert(V_ROWS % 8 == 0, "the swizzle repeats every 8 rows");
+            const int v_sub = lane / V_CHUNKS, v_piece = lane % V_CHUNKS, v_base = warp * (32 / V_CHUNKS) + v_sub;
+            const uint32_t v_at = smem_base + (uint32_t)stage * STAGE_BYTES + T::BYTES + TV::offset(v_base, v_piece);
+            constexpr int LOOKUPS = (V_PASSES + V_CHUNKS - 1) / V_CHUNKS;      // passes whose row this lane looks up
+            int my_v_row[LOOKUPS];
+#pragma unroll
+            for (int l = 0; l < LOOKUPS; ++l) {
+                my_v_row[l] = -1;
+                const int pass = v_piece + l * V_CHUNKS;
+                const int key = key0 + v_base + pass * V_ROWS;
+                if (pass < V_PASSES && key < key_end) my_v_row[l] = cache_row_of(table, key, p.page_size, p.page_shift, p.num_pages, p.error_flag);
+            }
+#pragma unroll
+            for (int i = 0; i < V_PASSES; ++i) {
+                const int row = __shfl_sync(0xffffffffu, my_v_row[i / V_CHUNKS], v_sub * V_CHUNKS + i % V_CHUNKS);
+                const bool valid = row >= 0;
+                cp_async_16(v_at + (uint32_t)(i * V_ROWS * V_CHUNKS * 16), p.v_pages + ((size_t)(valid ? row : 0) * p.nkv + kvh) * DV + v_piece * 8, valid);
+            }
         }
     };
 
@@ -254,8 +279,8 @@ attention_decode_kernel(Params p) {
 
     // ---- Q fragments: rows = heads (row r -> head h0 + r), zero beyond `heads` ----
     uint32_t qb[D / 16][NH][2];          // Q^T as the MMA's second operand: lane (g, t) holds head g (+ 8), d = 2t, 2t + 1 (+ 8)
-    if (p.qkv) {
-        __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + STAGES * 2 * T::BYTES);       // [16][D]
+    if constexpr (D == DV) if (p.qkv) {
+        __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + STAGES * STAGE_BYTES);       // [16][D]
         const int width = (p.nq + 2 * p.nkv) * D;
         const float* row = p.qkv + (size_t)t * width;
         const int half = p.rotary_dim / 2;
@@ -330,7 +355,7 @@ attention_decode_kernel(Params p) {
                 const float* v = raw + 17 * D;
                 // the row of the tile that the copies left out, if this CTA fills it itself
                 const int tile_row = pos - key_begin - (n_tiles - 1) * TILE_KEYS;
-                uint8_t* k_tile = smem + (size_t)(n_tiles - 1) * 2 * T::BYTES;
+                uint8_t* k_tile = smem + (size_t)(n_tiles - 1) * STAGE_BYTES;
                 uint8_t* v_tile = k_tile + T::BYTES;
                 auto put = [&](__nv_bfloat16* cache, uint8_t* tile, int i, float value) {
                     const __nv_bfloat16 x = __float2bfloat16_rn(value);
@@ -362,7 +387,8 @@ attention_decode_kernel(Params p) {
                 qb[kk][h][0] = *reinterpret_cast<const uint32_t*>(src);
                 qb[kk][h][1] = *reinterpret_cast<const uint32_t*>(src + 8);
             }
-    } else {
+    }
+    if (D != DV || !p.qkv) {
         pdl_wait();
         const int r0 = lane >> 2, c = (lane & 3) * 2;
         const __nv_bfloat16* base = p.q + ((size_t)t * p.nq + h0) * D;
@@ -378,9 +404,9 @@ attention_decode_kernel(Params p) {
     }
 
     // O^T: d = 16 mt + g (+ 8) down the rows, head 8 h + 2 t (+ 1) across; lane (g, t) holds [mt][h][0..3]
-    float o[D / 16][NH][4];
+    float o[DV / 16][NH][4];
 #pragma unroll
-    for (int mt = 0; mt < D / 16; ++mt)
+    for (int mt = 0; mt < DV / 16; ++mt)
 #pragma unroll
         for (int h = 0; h < NH; ++h) o[mt][h][0] = o[mt][h][1] = o[mt][h][2] = o[mt][h][3] = 0.f;
     // per head 8 h + 2 t + j: the running maximum (the same in the 8 lanes that share t) and THIS lane's part of the sum
@@ -402,7 +428,7 @@ attention_decode_kernel(Params p) {
             cp_async_commit();
         }
         const int stage = tile % STAGES;
-        const uint32_t ks = smem_base + (uint32_t)stage * 2 * T::BYTES, vs = ks + T::BYTES;
+        const uint32_t ks = smem_base + (uint32_t)stage * STAGE_BYTES, vs = ks + T::BYTES;
         const int key0 = key_begin + tile * TILE_KEYS + warp * 16;       // this warp's 16 keys
         if (key0 < key_end) {
             // ---- S^T = K Q^T for 16 keys.  All fragments are asked for before the first product (one warp per
@@ -422,10 +448,10 @@ attention_decode_kernel(Params p) {
 #pragma unroll
                 for (int h = 0; h < NH; ++h) mma_bf16(kk & 1 ? st_odd[h] : st[h], kf[kk], qb[kk][h][0], qb[kk][h][1]);
             // the values' fragments travel while the probabilities are made: V^T as the first operand
-            uint32_t vf[D / 16][4];
+            uint32_t vf[DV / 16][4];
 #pragma unroll
-            for (int mt = 0; mt < D / 16; ++mt)
-                ldmatrix_x4_trans(vs + T::offset(v_row, mt * 2 + (lm & 1)), vf[mt][0], vf[mt][1], vf[mt][2], vf[mt][3]);
+            for (int mt = 0; mt < DV / 16; ++mt)
+                ldmatrix_x4_trans(vs + TV::offset(v_row, mt * 2 + (lm & 1)), vf[mt][0], vf[mt][1], vf[mt][2], vf[mt][3]);
             // st[h][0], [1]: key g, heads 2t, 2t + 1; [2], [3]: key g + 8
             const bool low_hidden = key0 + (lane >> 2) >= key_end, high_hidden = key0 + (lane >> 2) + 8 >= key_end;
             uint32_t pb[NH][2];
@@ -462,14 +488,14 @@ attention_decode_kernel(Params p) {
                 // ---- O^T = O^T * correction + V^T P^T (the maximum is a whole number and seldom moves) ----
                 if (__any_sync(0xffffffffu, correction[0] != 1.f || correction[1] != 1.f)) {
 #pragma unroll
-                    for (int mt = 0; mt < D / 16; ++mt) {
+                    for (int mt = 0; mt < DV / 16; ++mt) {
                         o[mt][h][0] *= correction[0]; o[mt][h][1] *= correction[1];
                         o[mt][h][2] *= correction[0]; o[mt][h][3] *= correction[1];
                     }
                 }
             }
 #pragma unroll
-            for (int mt = 0; mt < D / 16; ++mt)
+            for (int mt = 0; mt < DV / 16; ++mt)
 #pragma unroll
                 for (int h = 0; h < NH; ++h) mma_bf16(o[mt][h], vf[mt], pb[h][0], pb[h][1]);
         }
@@ -486,7 +512,7 @@ attention_decode_kernel(Params p) {
             head_sum[h][j] += __shfl_xor_sync(0xffffffffu, head_sum[h][j], 8);
             head_sum[h][j] += __shfl_xor_sync(0xffffffffu, head_sum[h][j], 16);
         }
-    constexpr int MERGE_STRIDE = D + 4;                               // heads 4 words apart: a warp's 32 stores meet 32 banks
+    constexpr int MERGE_STRIDE = DV + 4;                               // heads 4 words apart: a warp's 32 stores meet 32 banks
     float* merge_o = reinterpret_cast<float*>(smem);                  // [WARPS][16][MERGE_STRIDE]
     float* merge_m = merge_o + WARPS * 16 * MERGE_STRIDE;             // [WARPS][16]
     float* merge_l = merge_m + WARPS * 16;
@@ -494,7 +520,7 @@ attention_decode_kernel(Params p) {
     {
         const int g = lane >> 2, t2 = (lane & 3) * 2;
 #pragma unroll
-        for (int mt = 0; mt < D / 16; ++mt)
+        for (int mt = 0; mt < DV / 16; ++mt)
 #pragma unroll
             for (int h = 0; h < NH; ++h) {
                 float* dst = merge_o + ((size_t)warp * 16 + h * 8 + t2) * MERGE_STRIDE + mt * 16 + g;
@@ -529,19 +555,19 @@ attention_decode_kernel(Params p) {
         const float inv = 1.0f / total;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) merge_f[w * 16 + r] = f[w] * inv;
-        if (p.cluster) exchange_of<D>(smem)[16 * D + r] = top + log2f(total);
+        if (p.cluster) exchange_of<DV>(smem)[16 * DV + r] = top + log2f(total);
         else if (p.n_splits > 1)
-            p.partial[(size_t)p.n_tokens * p.nq * p.n_splits * D + ((size_t)t * p.nq + h0 + r) * p.n_splits + blockIdx.z] =
+            p.partial[(size_t)p.n_tokens * p.nq * p.n_splits * DV + ((size_t)t * p.nq + h0 + r) * p.n_splits + blockIdx.z] =
                 top + log2f(total);
     }
     __syncthreads();
     {
-        constexpr int PER_THREAD = (16 * (D / 4) + WARPS * 32 - 1) / (WARPS * 32);
+        constexpr int PER_THREAD = (16 * (DV / 4) + WARPS * 32 - 1) / (WARPS * 32);
 #pragma unroll
         for (int j = 0; j < PER_THREAD; ++j) {
             const int idx = tid + j * WARPS * 32;
-            if (idx >= heads * (D / 4)) break;
-            const int r = idx / (D / 4), c4 = idx % (D / 4);
+            if (idx >= heads * (DV / 4)) break;
+            const int r = idx / (DV / 4), c4 = idx % (DV / 4);
             float4 value = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
             for (int w = 0; w < WARPS; ++w) {
@@ -551,20 +577,20 @@ attention_decode_kernel(Params p) {
             }
             const int h = h0 + r;
             if (p.cluster) {
-                *reinterpret_cast<float4*>(exchange_of<D>(smem) + r * D + c4 * 4) = value;
+                *reinterpret_cast<float4*>(exchange_of<DV>(smem) + r * DV + c4 * 4) = value;
             } else if (p.n_splits == 1) {
                 uint2 packed;
                 packed.x = pack_bf16(value.x, value.y);
                 packed.y = pack_bf16(value.z, value.w);
-                *reinterpret_cast<uint2*>(p.out + ((size_t)t * p.nq + h) * D + c4 * 4) = packed;
+                *reinterpret_cast<uint2*>(p.out + ((size_t)t * p.nq + h) * DV + c4 * 4) = packed;
             } else {
                 const size_t at = ((size_t)t * p.nq + h) * p.n_splits + blockIdx.z;
-                *reinterpret_cast<float4*>(p.partial + at * D + c4 * 4) = value;
+                *reinterpret_cast<float4*>(p.partial + at * DV + c4 * 4) = value;
             }
         }
     }
     if (p.cluster) {
-        cluster_merge<D>(p, smem, t, h0, heads);
+        cluster_merge<DV>(p, smem, t, h0, heads);
         return;
     }
     if (p.n_splits == 1 || !p.counters) return;
@@ -585,22 +611,22 @@ attention_decode_kernel(Params p) {
     }
     __syncthreads();
     if (!last_flag) return;
-    const float* lse = p.partial + (size_t)p.n_tokens * p.nq * p.n_splits * D;
+    const float* lse = p.partial + (size_t)p.n_tokens * p.nq * p.n_splits * DV;
     if (used <= 16) {
         // Few ranges: a thread owns eight elements of a head and has every load it needs (the ranges'
         // log-sum-exps and their eight elements) in flight at once, so the token's tail is one trip to L2.
-        for (int idx = tid; idx < heads * (D / 8); idx += WARPS * 32) {
-            const int r = idx / (D / 8), c8 = idx % (D / 8);
+        for (int idx = tid; idx < heads * (DV / 8); idx += WARPS * 32) {
+            const int r = idx / (DV / 8), c8 = idx % (DV / 8);
             const float* lrow = lse + ((size_t)t * p.nq + h0 + r) * p.n_splits;
-            const float4* base = reinterpret_cast<const float4*>(p.partial + ((size_t)t * p.nq + h0 + r) * p.n_splits * D) + c8 * 2;
+            const float4* base = reinterpret_cast<const float4*>(p.partial + ((size_t)t * p.nq + h0 + r) * p.n_splits * DV) + c8 * 2;
             float l[16];
             float4 v[16][2];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
                 const bool there = j < used;
                 l[j] = there ? __ldcg(lrow + j) : -INFINITY;
-                v[j][0] = there ? __ldcg(base + (size_t)j * (D / 4)) : make_float4(0.f, 0.f, 0.f, 0.f);
-                v[j][1] = there ? __ldcg(base + (size_t)j * (D / 4) + 1) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[j][0] = there ? __ldcg(base + (size_t)j * (DV / 4)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[j][1] = there ? __ldcg(base + (size_t)j * (DV / 4) + 1) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
             float top = l[0];
 #pragma unroll
@@ -620,7 +646,7 @@ attention_decode_kernel(Params p) {
             packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
             packed.z = pack_bf16(acc[4] * inv, acc[5] * inv);
             packed.w = pack_bf16(acc[6] * inv, acc[7] * inv);
-            *reinterpret_cast<uint4*>(p.out + ((size_t)t * p.nq + h0 + r) * D + c8 * 8) = packed;
+            *reinterpret_cast<uint4*>(p.out + ((size_t)t * p.nq + h0 + r) * DV + c8 * 8) = packed;
         }
         return;
     }
@@ -643,15 +669,15 @@ attention_decode_kernel(Params p) {
     }
     __syncthreads();
     // 16 bytes per load, eight ranges in flight per thread: the last CTA's reads are the tail of the step
-    for (int idx = tid; idx < heads * (D / 4); idx += WARPS * 32) {
-        const int r = idx / (D / 4), c4 = idx % (D / 4);
-        const float4* base = reinterpret_cast<const float4*>(p.partial + ((size_t)t * p.nq + h0 + r) * p.n_splits * D) + c4;
+    for (int idx = tid; idx < heads * (DV / 4); idx += WARPS * 32) {
+        const int r = idx / (DV / 4), c4 = idx % (DV / 4);
+        const float4* base = reinterpret_cast<const float4*>(p.partial + ((size_t)t * p.nq + h0 + r) * p.n_splits * DV) + c4;
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         for (int s0 = 0; s0 < used; s0 += 8) {
             float4 v[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-                v[j] = s0 + j < used ? __ldcg(base + (size_t)(s0 + j) * (D / 4)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[j] = s0 + j < used ? __ldcg(base + (size_t)(s0 + j) * (DV / 4)) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 const float w = s0 + j < used ? weight[r * used + s0 + j] : 0.f;
@@ -662,7 +688,7 @@ attention_decode_kernel(Params p) {
         uint2 packed;
         packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
         packed.y = pack_bf16(acc[2] * inv, acc[3] * inv);
-        *reinterpret_cast<uint2*>(p.out + ((size_t)t * p.nq + h0 + r) * D + c4 * 4) = packed;
+        *reinterpret_cast<uint2*>(p.out + ((size_t)t * p.nq + h0 + r) * DV + c4 * 4) = packed;
     }
 }
 
@@ -695,21 +721,21 @@ __global__ void attention_merge_kernel(Params p) {
     }
 }
 
-template <int D>
+template <int D, int DV>
 size_t decode_smem_bytes() {
-    const size_t ring = (size_t)STAGES * 2 * Tile<D>::BYTES + 16 * D * 2 + D * 4 + 18 * D * 4;   // the tiles, the rotated queries, the angles' cosines and sines, the step's 32-bit rows
-    const size_t merge = (size_t)WARPS * 16 * (D + 4 + 3) * sizeof(float) + (size_t)(16 * D + 16) * sizeof(float);   // the warps' merge, then the cluster's exchange
+    const size_t ring = (size_t)STAGES * (Tile<D>::BYTES + Tile<DV>::BYTES) + 16 * D * 2 + D * 4 + 18 * D * 4;   // the tiles, the rotated queries, the angles' cosines and sines, the step's 32-bit rows
+    const size_t merge = (size_t)WARPS * 16 * (DV + 4 + 3) * sizeof(float) + (size_t)(16 * DV + 16) * sizeof(float);   // the warps' merge, then the cluster's exchange
     const size_t weights = (size_t)16 * (MAX_FUSED_SPLITS + 1) * sizeof(float);
     return ring > merge ? (ring > weights ? ring : weights) : (merge > weights ? merge : weights);
 }
 
-template <int D, int NH, bool CAP = false>
+template <int D, int DV, int NH, bool CAP = false>
 int configure_decode() {
     static int state = 0;                  // 1: done, -1: failed
     if (state == 0) {
         state = 1;
-        if (cudaFuncSetAttribute(attention_decode_kernel<D, NH, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<D>()) != cudaSuccess ||
-            cudaFuncSetAttribute(attention_decode_kernel<D, NH, CAP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
+        if (cudaFuncSetAttribute(attention_decode_kernel<D, DV, NH, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<D, DV>()) != cudaSuccess ||
+            cudaFuncSetAttribute(attention_decode_kernel<D, DV, NH, CAP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
             cudaGetLastError();
             state = -1;
         }
@@ -718,17 +744,17 @@ int configure_decode() {
 }
 
 // Clusters of `size` CTAs of the kernel that the device holds at once (asked of the driver once per size; 0: none).
-template <int D, int NH>
+template <int D, int DV, int NH>
 int max_active_clusters(int size) {
     static int cached[MAX_CLUSTER + 1] = {};
     if (size < 2 || size > MAX_CLUSTER) return 0;
     if (cached[size] == 0) {
         cached[size] = -1;
-        if (configure_decode<D, NH>() == LIA_OK) {
+        if (configure_decode<D, DV, NH>() == LIA_OK) {
             cudaLaunchConfig_t config = {};
             config.gridDim = dim3(1, 1, (unsigned)size);
             config.blockDim = dim3(WARPS * 32);
-            config.dynamicSmemBytes = decode_smem_bytes<D>();
+            config.dynamicSmemBytes = decode_smem_bytes<D, DV>();
             cudaLaunchAttribute attribute[1];
             attribute[0].id = cudaLaunchAttributeClusterDimension;
             attribute[0].val.clusterDim.x = 1;
@@ -737,7 +763,7 @@ int max_active_clusters(int size) {
             config.attrs = attribute;
             config.numAttrs = 1;
             int clusters = 0;
-            if (cudaOccupancyMaxActiveClusters(&clusters, attention_decode_kernel<D, NH>, &config) == cudaSuccess && clusters > 0)
+            if (cudaOccupancyMaxActiveClusters(&clusters, attention_decode_kernel<D, DV, NH>, &config) == cudaSuccess && clusters > 0)
                 cached[size] = clusters;
             else
                 cudaGetLastError();
@@ -746,11 +772,11 @@ int max_active_clusters(int size) {
     return cached[size] > 0 ? cached[size] : 0;
 }
 
-template <int D, int NH, bool CAP = false>
+template <int D, int DV, int NH, bool CAP = false>
 int launch_decode(const Params& p, int n_rows, cudaStream_t stream) {
-    int rc = configure_decode<D, NH, CAP>();
+    int rc = configure_decode<D, DV, NH, CAP>();
     if (rc != LIA_OK) return rc;
-    const size_t smem = decode_smem_bytes<D>();
+    const size_t smem = decode_smem_bytes<D, DV>();
     const int group = p.nq / p.nkv;
     dim3 grid(n_rows, p.nkv * ((group + 15) / 16), p.n_splits);
     if (p.cluster) {
@@ -769,28 +795,28 @@ int launch_decode(const Params& p, int n_rows, cudaStream_t stream) {
         config.attrs = attributes;
         config.numAttrs = lia_pdl_enabled.load(std::memory_order_relaxed) ? 2 : 1;
         lia_launch_counter.fetch_add(1, std::memory_order_relaxed);
-        if (cudaLaunchKernelEx(&config, attention_decode_kernel<D, NH, CAP>, p) != cudaSuccess) {
+        if (cudaLaunchKernelEx(&config, attention_decode_kernel<D, DV, NH, CAP>, p) != cudaSuccess) {
             cudaGetLastError();
             return LIA_ERR_LAUNCH;
         }
         return cudaGetLastError() == cudaSuccess ? LIA_OK : LIA_ERR_LAUNCH;
     }
-    rc = lia_launch(attention_decode_kernel<D, NH, CAP>, grid, dim3(WARPS * 32), smem, stream, p);
+    rc = lia_launch(attention_decode_kernel<D, DV, NH, CAP>, grid, dim3(WARPS * 32), smem, stream, p);
     if (rc != LIA_OK) return rc;
     if (p.n_splits > 1 && !p.counters)
-        rc = lia_launch(attention_merge_kernel<D>, dim3(n_rows, p.nq), dim3(D < 128 ? D : 128), 0, stream, p);
+        rc = lia_launch(attention_merge_kernel<DV>, dim3(n_rows, p.nq), dim3(DV < 128 ? DV : 128), 0, stream, p);
     return rc;
 }
 
 // CTAs of the kernel that one SM holds at once (asked of the driver once; 0: unknown).
-template <int D, int NH>
+template <int D, int DV, int NH>
 int ctas_per_sm() {
     static int cached = 0;
     if (cached == 0) {
         cached = -1;
         int blocks = 0;
-        if (configure_decode<D, NH>() == LIA_OK &&
-            cudaOccupancyMaxActiveBlocksPerMultiprocessor(&blocks, attention_decode_kernel<D, NH>, WARPS * 32, decode_smem_bytes<D>()) == cudaSuccess &&
+        if (configure_decode<D, DV, NH>() == LIA_OK &&
+            cudaOccupancyMaxActiveBlocksPerMultiprocessor(&blocks, attention_decode_kernel<D, DV, NH>, WARPS * 32, decode_smem_bytes<D, DV>()) == cudaSuccess &&
             blocks > 0)
             cached = blocks;
         else
@@ -799,11 +825,11 @@ int ctas_per_sm() {
     return cached > 0 ? cached : 0;
 }
 
-template <int D>
+template <int D, int DV>
 int cluster_splits_for(bool wide, int clusters, int wanted) {
     for (int size = MAX_CLUSTER; size >= 2; size /= 2) {
         if (size > wanted) continue;
-        const int fit = wide ? max_active_clusters<D, 2>(size) : max_active_clusters<D, 1>(size);
+        const int fit = wide ? max_active_clusters<D, DV, 2>(size) : max_active_clusters<D, DV, 1>(size);
         if (clusters <= fit) return size;
     }
     return 1;
@@ -813,35 +839,52 @@ int cluster_splits_for(bool wide, int clusters, int wanted) {
 // Into how many ranges (2, 4, 8 or 16, at most `wanted`) the kernel can cut the keys of `clusters` (token, head group)
 // pairs with the ranges of a pair as one thread-block cluster, all clusters on the device at once; 1: none, the
 // ranges then meet through scratch memory (or there is one range).
-LIA_EXPORT int lia_attention_decode_cluster_splits(int d, int heads_per_kv_head, int clusters, int wanted) {
+#define LIA_DECODE_SIZES(CASE)                                                                       \
+    if (d == 128 && dv == 128) CASE(128, 128);                                                       \
+    if (d == 64 && dv == 64) CASE(64, 64);                                                           \
+    if (d == 32 && dv == 32) CASE(32, 32);                                                           \
+    if (d == 64 && dv == 128) CASE(64, 128);                                                         \
+    if (d == 128 && dv == 64) CASE(128, 64);                                                         \
+    if (d == 32 && dv == 64) CASE(32, 64);                                                           \
+    if (d == 64 && dv == 32) CASE(64, 32);
+
+LIA_EXPORT int lia_attention_decode_cluster_splits(int d, int dv, int heads_per_kv_head, int clusters, int wanted) {
     if (clusters <= 0 || wanted < 2) return 1;
     const bool wide = heads_per_kv_head > 8;
-    if (d == 128) return cluster_splits_for<128>(wide, clusters, wanted);
-    if (d == 64) return cluster_splits_for<64>(wide, clusters, wanted);
-    if (d == 32) return cluster_splits_for<32>(wide, clusters, wanted);
+#define LIA_CASE(D, DV) return cluster_splits_for<D, DV>(wide, clusters, wanted)
+    LIA_DECODE_SIZES(LIA_CASE)
+#undef LIA_CASE
     return 1;
+}
+
+// Whether the kernel takes keys and values of these head sizes.
+LIA_EXPORT int lia_attention_decode_accepts(int d, int dv) {
+#define LIA_CASE(D, DV) return 1
+    LIA_DECODE_SIZES(LIA_CASE)
+#undef LIA_CASE
+    return 0;
 }
 
 // CTAs of the kernel that an SM holds at once for this head size (registers and shared memory decide: 2 at head
 // size 128, more below); 0: the kernel does not take the head size, or the driver did not say.
-LIA_EXPORT int lia_attention_decode_ctas_per_sm(int d, int heads_per_kv_head) {
+LIA_EXPORT int lia_attention_decode_ctas_per_sm(int d, int dv, int heads_per_kv_head) {
     const bool wide = heads_per_kv_head > 8;
-    if (d == 128) return wide ? ctas_per_sm<128, 2>() : ctas_per_sm<128, 1>();
-    if (d == 64) return wide ? ctas_per_sm<64, 2>() : ctas_per_sm<64, 1>();
-    if (d == 32) return wide ? ctas_per_sm<32, 2>() : ctas_per_sm<32, 1>();
+#define LIA_CASE(D, DV) return wide ? ctas_per_sm<D, DV, 2>() : ctas_per_sm<D, DV, 1>()
+    LIA_DECODE_SIZES(LIA_CASE)
+#undef LIA_CASE
     return 0;
 }
 
 // Floats of scratch that n_rows tokens with n_splits ranges need.
-LIA_EXPORT long long lia_attention_decode_scratch_floats(int n_tokens, int nq, int d, int n_splits) {
-    return n_splits > 1 ? (long long)n_tokens * nq * n_splits * (d + 1) : 0;
+LIA_EXPORT long long lia_attention_decode_scratch_floats(int n_tokens, int nq, int dv, int n_splits) {
+    return n_splits > 1 ? (long long)n_tokens * nq * n_splits * (dv + 1) : 0;
 }
 
 // `qkv` non-null: q is ignored; the kernel takes the queries from the 32-bit q|k|v rows, applies the rotary
 // encoding (rotary_dim leading elements of each head; 0: none) and, when `write_kv`, the CTA of each token's last
 // range rotates the token's key and appends key and value to the page of its position before reading them.
 // Decode attention for the tokens listed in `rows` (indices into the step's batch), bfloat16 only,
-// head_dim 32, 64 or 128 (other sizes: LIA_ERR_SIZE; the caller falls back to the generic kernel).
+// keys of head size d and values of head size dv, 32, 64 or 128 and equal or neighbours (other sizes: LIA_ERR_SIZE; the caller falls back to the generic kernel).
 // `cluster` non-zero: `n_splits` is what lia_attention_decode_cluster_splits gave; `partial` and `counters` are not used.
 // `all_new` non-zero: the rows may be tokens of prompt portions of this step, whose earlier keys the kernels ahead
 // have written too; zero: only a row's own key is of this step (decoded tokens), and older tiles are fetched early.
@@ -850,7 +893,7 @@ LIA_EXPORT long long lia_attention_decode_scratch_floats(int n_tokens, int nq, i
 LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const void* v_pages, const int* rows,
                                     int n_rows, const int* positions, const int* slots, const int* block_table,
                                     int table_stride, void* out, float* partial, long long partial_floats,
-                                    int* counters, int n_tokens, int nq, int nkv, int d, int page_size, int window, float scale,
+                                    int* counters, int n_tokens, int nq, int nkv, int d, int dv, int page_size, int window, float scale,
                                     int split_len, int n_splits, const float* qkv, const float* inv_freq, int rotary_dim,
                                     int write_kv, int num_pages, int cluster, int all_new, int sink, float softcap,
                                     int* error_flag, cudaStream_t stream) {
@@ -859,7 +902,7 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
         n_splits > 65535)
         return LIA_ERR_SIZE;
     if (cluster && (n_splits < 2 || n_splits > MAX_CLUSTER || (n_splits & (n_splits - 1)))) return LIA_ERR_SIZE;
-    if (!cluster && n_splits > 1 && (!partial || partial_floats < lia_attention_decode_scratch_floats(n_tokens, nq, d, n_splits)))
+    if (!cluster && n_splits > 1 && (!partial || partial_floats < lia_attention_decode_scratch_floats(n_tokens, nq, dv, n_splits)))
         return LIA_ERR_SIZE;
     if (!cluster && n_splits > 1 && ((uintptr_t)partial & 15u)) return LIA_ERR_ALIGN;
     Params p;
@@ -867,7 +910,7 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
     p.rows = rows; p.positions = positions; p.slots = slots; p.block_table = block_table;
     p.out = (__nv_bfloat16*)out; p.partial = partial;
     p.counters = n_splits <= MAX_FUSED_SPLITS ? counters : nullptr;
-    if (qkv && (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim > 0 && !inv_freq) || nq / nkv > 16))
+    if (qkv && (d != dv || rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim > 0 && !inv_freq) || nq / nkv > 16))
         return LIA_ERR_SIZE;             // with more than 16 heads per kv head two CTAs would share the appended key
     p.qkv = qkv; p.inv_freq = inv_freq; p.rotary_dim = rotary_dim; p.write_kv = write_kv; p.num_pages = num_pages;
     p.k_write = (__nv_bfloat16*)const_cast<void*>(k_pages); p.v_write = (__nv_bfloat16*)const_cast<void*>(v_pages);
@@ -887,13 +930,14 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
     }
     const bool wide = nq / nkv > 8;             // more than 8 query heads per kv head: two groups of 8 per CTA
     if (p.cap_in != 0.f) {
-        if (d == 128) return wide ? launch_decode<128, 2, true>(p, n_rows, stream) : launch_decode<128, 1, true>(p, n_rows, stream);
-        if (d == 64) return wide ? launch_decode<64, 2, true>(p, n_rows, stream) : launch_decode<64, 1, true>(p, n_rows, stream);
-        if (d == 32) return wide ? launch_decode<32, 2, true>(p, n_rows, stream) : launch_decode<32, 1, true>(p, n_rows, stream);
+        if (d != dv) return LIA_ERR_SIZE;       // (a cap with unequal sizes: the caller's other kernel)
+        if (d == 128) return wide ? launch_decode<128, 128, 2, true>(p, n_rows, stream) : launch_decode<128, 128, 1, true>(p, n_rows, stream);
+        if (d == 64) return wide ? launch_decode<64, 64, 2, true>(p, n_rows, stream) : launch_decode<64, 64, 1, true>(p, n_rows, stream);
+        if (d == 32) return wide ? launch_decode<32, 32, 2, true>(p, n_rows, stream) : launch_decode<32, 32, 1, true>(p, n_rows, stream);
         return LIA_ERR_SIZE;
     }
-    if (d == 128) return wide ? launch_decode<128, 2>(p, n_rows, stream) : launch_decode<128, 1>(p, n_rows, stream);
-    if (d == 64) return wide ? launch_decode<64, 2>(p, n_rows, stream) : launch_decode<64, 1>(p, n_rows, stream);
-    if (d == 32) return wide ? launch_decode<32, 2>(p, n_rows, stream) : launch_decode<32, 1>(p, n_rows, stream);
+#define LIA_CASE(D, DV) return wide ? launch_decode<D, DV, 2>(p, n_rows, stream) : launch_decode<D, DV, 1>(p, n_rows, stream)
+    LIA_DECODE_SIZES(LIA_CASE)
+#undef LIA_CASE
     return LIA_ERR_SIZE;
 }

@@ -33,8 +33,8 @@
 // point and its sum in scratch memory, and attention_prefill_merge_kernel puts a row's ranges together.
 //
 // Rows are (token, head) pairs: row r is token r / g, head r % g of the CTA's tokens, so the keys of a kv
-// head are read once for all its query heads.  Head sizes 64 and 128, g a divisor of 128; the caller uses
-// the mma.sync kernel (attention_prefill.cu) for everything else.
+// head are read once for all its query heads.  Head sizes 64 and 128, the keys' and the values' apart, g a divisor of
+// 128; the caller uses other kernels (attention_prefill.cu, attention_generic.cu) for everything else.
 #include "attention_tmem.cuh"
 
 using namespace tc5;
@@ -52,11 +52,11 @@ constexpr float LAZY = 8.f;              // see the softmax
 struct Params {
     const __nv_bfloat16* q;          // [tokens, nq, D]
     const __nv_bfloat16* k_pages;    // [pages, page_size, nkv, D]
-    const __nv_bfloat16* v_pages;
+    const __nv_bfloat16* v_pages;    // [pages, page_size, nkv, DV]
     const int* segments;             // [n_segments][3]: first token's batch index, its position, count
     const int* slots;                // [tokens]
     const int* block_table;          // [slots, table_stride]
-    __nv_bfloat16* out;              // [tokens, nq, D]
+    __nv_bfloat16* out;              // [tokens, nq, DV]
     int n_segments, table_stride, nq, nkv, page_size, page_shift, window, tokens_per_tile;
     float scale_log2;                // softmax scale * log2(e); with a cap on the scores: cap * log2(e)
     float cap_in;                    // 0: no cap; else scale / cap: the score is cap * tanh(q.k * cap_in)
@@ -65,14 +65,14 @@ struct Params {
     // With `splits` > 1 the keys of every CTA's rows are cut into that many ranges (blockIdx.z; whole tiles): each
     // range leaves its output unnormalised and the row's reference point and sum, and the merge kernel puts them together.
     int splits;
-    float* partial_o;                // [splits][tokens * nq][D]
+    float* partial_o;                // [splits][tokens * nq][DV]
     float* partial_ms;               // [splits][tokens * nq][2]: reference point (a whole number, or -infinity), sum
     long long n_rows_total;          // tokens * nq
     int sink;                        // 1: one is added to the softmax's denominator (a key of score 0 without a value)
 };
 
 // CAP: the scores pass a tanh cap (an instantiation of its own, so that the kernel without a cap is what it was)
-template <int D, bool CAP = false>
+template <int D, int DV, bool CAP = false>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(Params p) {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -80,7 +80,7 @@ attention_prefill_tc_kernel(Params p) {
     __shared__ uint32_t tmem_base_slot;
     __shared__ short pair_ref[2][2][ROWS];         // what the two threads of a row tell each other (16 bits: shared memory is full to the last KB)
     constexpr int PIECES = D / 8;                      // 16-byte pieces per row
-    constexpr uint32_t Q_BYTES = ROWS * D * 2, KV_BYTES = KT * D * 2;
+    constexpr uint32_t Q_BYTES = ROWS * D * 2, K_BYTES = KT * D * 2, KV_BYTES = KT * (D + DV) * 2;      // KV: a stage's keys and values
     // tensor memory: two score buffers of 128 columns, the output's head_dim columns (128 kept), and two buffers of
     // probabilities of 64 columns (128 keys as bf16 pairs)
     constexpr int TMEM_COLS = 512;
@@ -162,7 +162,7 @@ attention_prefill_tc_kernel(Params p) {
             // the keys' stage is free as soon as the first product of three tiles ago has read it, the values' stage
             // only after the second
             if (j >= STAGES && !mbar_wait(smem_u32(&k_empty[st]), ((uint32_t)(j / STAGES) & 1u) ^ 1u)) { ok = false; break; }
-            const uint32_t ks = kv_s + (uint32_t)st * 2 * KV_BYTES, vs = ks + KV_BYTES;
+            const uint32_t ks = kv_s + (uint32_t)st * KV_BYTES, vs = ks + K_BYTES;
             const int key0 = key_begin + j * KT;
             // PIECES lanes share a key row (their 16-byte pieces make one coalesced request); lane j of them looks
             // up the row of pass j
@@ -186,11 +186,30 @@ attention_prefill_tc_kernel(Params p) {
                 }
                 cp_async_commit();
                 if (j >= STAGES && !mbar_wait(smem_u32(&v_empty[st]), ((uint32_t)(j / STAGES) & 1u) ^ 1u)) { ok = false; break; }
+                if constexpr (D == DV) {
 #pragma unroll
-                for (int i = 0; i < PASSES; ++i) {
-                    const bool valid = rows[i] >= 0;
-                    const size_t src = ((size_t)(valid ? rows[i] : 0) * p.nkv + kvh) * D + piece * 8;
-                    cp_async_16(vs + tile_offset<KT>(sub + i * ROWS_PER_PASS, piece), p.v_pages + src, valid);
+                    for (int i = 0; i < PASSES; ++i) {
+                        const bool valid = rows[i] >= 0;
+                        const size_t src = ((size_t)(valid ? rows[i] : 0) * p.nkv + kvh) * D + piece * 8;
+                        cp_async_16(vs + tile_offset<KT>(sub + i * ROWS_PER_PASS, piece), p.v_pages + src, valid);
+                    }
+                } else {
+                    // values of another size than the keys: their pieces and passes are their own
+                    constexpr int V_PIECES = DV / 8, V_ROWS = LOADERS / V_PIECES, V_PASSES = KT / V_ROWS;
+                    static_assert(V_PASSES <= V_PIECES, "one lane per pass");
+                    const int v_sub = lt / V_PIECES, v_piece = lt % V_PIECES, v_group = (lane / V_PIECES) * V_PIECES;
+                    int my_v_row = -1;
+                    if (v_piece < V_PASSES) {
+                        const int key = key0 + v_sub + v_piece * V_ROWS;
+                        if (key < key_end) my_v_row = cache_row_of(table, key, p.page_size, p.page_shift, p.num_pages, p.error_flag);
+                    }
+#pragma unroll
+                    for (int i = 0; i < V_PASSES; ++i) {
+                        const int row = __shfl_sync(0xffffffffu, my_v_row, v_group + i);
+                        const bool valid = row >= 0;
+                        const size_t src = ((size_t)(valid ? row : 0) * p.nkv + kvh) * DV + v_piece * 8;
+                        cp_async_16(vs + tile_offset<KT>(v_sub + i * V_ROWS, v_piece), p.v_pages + src, valid);
+                    }
                 }
                 cp_async_commit();
             }
@@ -209,19 +228,19 @@ attention_prefill_tc_kernel(Params p) {
         if (!ok && p.error_flag) atomicExch(p.error_flag, 3);
     } else if (warp == SOFTMAX_WARPS && lane == 0 && n_tiles > 0) {
         // ---- MMA issuer ----
-        const uint32_t idesc_s = instr_desc(ROWS, KT), idesc_o = instr_desc_b_mn(ROWS, D);
+        const uint32_t idesc_s = instr_desc(ROWS, KT), idesc_o = instr_desc_b_mn(ROWS, DV);
         bool ok = mbar_wait(smem_u32(&q_full), 0u);
         // the operands' descriptors: the tile's first plus an offset in their lowest field (the start address in 16-byte
         // units; shared memory ends below what the field holds), so that an MMA costs this thread an addition
         static_assert(ROWS == KT, "Q and K tiles share their offsets");
-        const uint64_t desc_q0 = smem_desc(q_s), desc_kv0 = smem_desc(kv_s), desc_v0 = smem_desc_mn(kv_s + KV_BYTES, KT * 128, 1024);
+        const uint64_t desc_q0 = smem_desc(q_s), desc_kv0 = smem_desc(kv_s), desc_v0 = smem_desc_mn(kv_s + K_BYTES, KT * 128, 1024);
         // S_j = Q K_j^T into score buffer j & 1: issued one tile ahead, so that it runs while the softmax of the
         // tile before is at work (that buffer's last reader arrived on p_ready two tiles ago)
         auto first_product = [&](int j) {
             const int st = j % STAGES;
             if (!mbar_wait(smem_u32(&k_full[st]), (uint32_t)(j / STAGES) & 1u)) { ok = false; return; }
             tc_fence_after();
-            const uint64_t desc_k = desc_kv0 + (uint64_t)((uint32_t)st * (2 * KV_BYTES >> 4));
+            const uint64_t desc_k = desc_kv0 + (uint64_t)((uint32_t)st * (KV_BYTES >> 4));
 #pragma unroll
             for (int kk = 0; kk < D / 16; ++kk) {
                 const uint64_t offset = (uint64_t)(((kk >> 2) * (ROWS * 128) + (kk & 3) * 32) >> 4);      // Q and K tiles are laid out alike
@@ -233,7 +252,7 @@ attention_prefill_tc_kernel(Params p) {
         if (ok) first_product(0);
         for (int j = 0; j < n_tiles && ok; ++j) {
             const int st = j % STAGES;
-            const uint64_t desc_v = desc_v0 + (uint64_t)((uint32_t)st * (2 * KV_BYTES >> 4));
+            const uint64_t desc_v = desc_v0 + (uint64_t)((uint32_t)st * (KV_BYTES >> 4));
             if (j + 1 < n_tiles) first_product(j + 1);
             if (!ok) break;
             // O += P V once the values lie in shared memory and the probabilities in TMEM (and O has been rescaled if it had to be)
@@ -340,7 +359,7 @@ attention_prefill_tc_kernel(Params p) {
                 if (!mbar_wait(smem_u32(&p_free[(j - 1) & 1]), (uint32_t)((j - 1) >> 1) & 1u)) { ok = false; break; }
                 tc_fence_after();
 #pragma unroll 1
-                for (int c0 = half * (D / 2); c0 < (half + 1) * (D / 2); c0 += 16) {
+                for (int c0 = half * (DV / 2); c0 < (half + 1) * (DV / 2); c0 += 16) {
                     float o[16];
                     tmem_load16(tmem_o + lane_base + (uint32_t)c0, o);
 #pragma unroll
@@ -368,9 +387,9 @@ attention_prefill_tc_kernel(Params p) {
                 p.partial_ms[plane * 2] = row_max;
                 p.partial_ms[plane * 2 + 1] = pair_sum[r] + pair_sum[ROWS + r];
             }
-            float* dst = p.partial_o + plane * D;
+            float* dst = p.partial_o + plane * DV;
 #pragma unroll 1
-            for (int c0 = half * (D / 2); c0 < (half + 1) * (D / 2); c0 += 16) {
+            for (int c0 = half * (DV / 2); c0 < (half + 1) * (DV / 2); c0 += 16) {
                 float o[16];
                 tmem_load16(tmem_o + lane_base + (uint32_t)c0, o);
                 if (row_ok) {
@@ -380,9 +399,9 @@ attention_prefill_tc_kernel(Params p) {
             }
         } else if (ok) {
             const float inv = 1.0f / (pair_sum[r] + pair_sum[ROWS + r] + (p.sink ? exp2f(-row_max) : 0.f));
-            __nv_bfloat16* dst = p.out + ((size_t)(q_offset + tok0 + (row_ok ? tok : 0)) * p.nq + kvh * group + head) * D;
+            __nv_bfloat16* dst = p.out + ((size_t)(q_offset + tok0 + (row_ok ? tok : 0)) * p.nq + kvh * group + head) * DV;
 #pragma unroll 1
-            for (int c0 = half * (D / 2); c0 < (half + 1) * (D / 2); c0 += 16) {
+            for (int c0 = half * (DV / 2); c0 < (half + 1) * (DV / 2); c0 += 16) {
                 float o[16];
                 tmem_load16(tmem_o + lane_base + (uint32_t)c0, o);           // every lane takes part in the load
                 if (row_ok) {
@@ -478,42 +497,42 @@ __global__ void __launch_bounds__(128) attention_prefill_merge_kernel(Params p) 
     for (int e = 0; e < E; e += 2) *reinterpret_cast<__nv_bfloat162*>(dst + e) = __floats2bfloat162_rn(acc[e] * inv, acc[e + 1] * inv);
 }
 
-template <int D, bool CAP = false>
+template <int D, int DV, bool CAP = false>
 int launch(const Params& p, int n_tiles, cudaStream_t stream) {
-    const size_t smem = (size_t)ROWS * D * 2 + (size_t)STAGES * 2 * KT * D * 2 + 1024;
+    const size_t smem = (size_t)ROWS * D * 2 + (size_t)STAGES * KT * (D + DV) * 2 + 1024;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_tc_kernel<D, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attention_prefill_tc_kernel<D, DV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return LIA_ERR_LAUNCH;
         configured = true;
     }
-    const int rc = lia_launch(attention_prefill_tc_kernel<D, CAP>, dim3(n_tiles, p.nkv, p.splits), dim3(THREADS), smem, stream, p);
+    const int rc = lia_launch(attention_prefill_tc_kernel<D, DV, CAP>, dim3(n_tiles, p.nkv, p.splits), dim3(THREADS), smem, stream, p);
     if (rc != LIA_OK || p.splits <= 1) return rc;
-    return lia_launch(attention_prefill_merge_kernel<D>, dim3(n_tiles, p.nkv, ROWS / 4), dim3(128), 0, stream, p);
+    return lia_launch(attention_prefill_merge_kernel<DV>, dim3(n_tiles, p.nkv, ROWS / 4), dim3(128), 0, stream, p);
 }
 }  // namespace
 
-// Tokens of a portion that one CTA takes for `group` query heads per kv head and this head size (0: the tcgen05
-// kernel does not take the combination; use lia_attention_prefill).
-LIA_EXPORT int lia_attention_prefill_tc_tokens_per_tile(int group, int d) {
-    if (d != 64 && d != 128) return 0;
+// Tokens of a portion that one CTA takes for `group` query heads per kv head and these head sizes of keys and values (0:
+// the tcgen05 kernel does not take the combination; use another kernel).
+LIA_EXPORT int lia_attention_prefill_tc_tokens_per_tile(int group, int d, int dv) {
+    if ((d != 64 && d != 128) || (dv != 64 && dv != 128)) return 0;
     return group >= 1 && group <= ROWS && ROWS % group == 0 ? ROWS / group : 0;
 }
 
 // Arguments as lia_attention_prefill; `n_tiles` = sum over portions of ceil(count / tokens_per_tile) with the
 // tokens per tile of this kernel.  With `splits` > 1 every CTA's keys are cut into that many ranges of whole
 // 128-key tiles, each range a CTA of its own, and a second kernel merges them (few tokens over a long context
-// would otherwise leave most SMs idle); `partial` then holds splits * n_tokens * nq * (head size + 2) 32-bit words,
+// would otherwise leave most SMs idle); `partial` then holds splits * n_tokens * nq * (the values' head size + 2) 32-bit words,
 // `n_tokens` being the tokens of the whole batch that `q` and `out` cover.
 LIA_EXPORT int lia_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* segments,
                                         int n_segments, int n_tiles, const int* slots, const int* block_table,
-                                        int table_stride, void* out, int nq, int nkv, int d, int page_size, int window,
+                                        int table_stride, void* out, int nq, int nkv, int d, int dv, int page_size, int window,
                                         float scale, int num_pages, int splits, float* partial, int n_tokens, int sink,
                                         float softcap, int* error_flag, cudaStream_t stream) {
     if (n_segments <= 0 || n_tiles <= 0) return LIA_OK;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || nkv > 65535) return LIA_ERR_SIZE;
     if (splits < 1 || splits > 32 || (splits > 1 && (!partial || n_tokens <= 0))) return LIA_ERR_SIZE;
-    const int per_tile = lia_attention_prefill_tc_tokens_per_tile(nq / nkv, d);
+    const int per_tile = lia_attention_prefill_tc_tokens_per_tile(nq / nkv, d, dv);
     if (per_tile == 0) return LIA_ERR_SIZE;
     if (((uintptr_t)q & 15u) || ((uintptr_t)out & 15u) || ((uintptr_t)k_pages & 15u) || ((uintptr_t)v_pages & 15u) ||
         ((uintptr_t)partial & 15u))
@@ -536,8 +555,12 @@ LIA_EXPORT int lia_attention_prefill_tc(const void* q, const void* k_pages, cons
     p.sink = sink ? 1 : 0;
     p.n_rows_total = (long long)n_tokens * nq;
     p.partial_o = partial;
-    p.partial_ms = partial ? partial + (size_t)splits * p.n_rows_total * d : nullptr;
-    if (p.cap_in != 0.f) return d == 128 ? launch<128, true>(p, n_tiles, stream) : launch<64, true>(p, n_tiles, stream);
-    if (d == 128) return launch<128>(p, n_tiles, stream);
-    return launch<64>(p, n_tiles, stream);
+    p.partial_ms = partial ? partial + (size_t)splits * p.n_rows_total * dv : nullptr;
+    if (d != dv) {
+        if (p.cap_in != 0.f) return LIA_ERR_SIZE;       // (a cap with unequal sizes: the caller's other kernel)
+        return d == 64 ? launch<64, 128>(p, n_tiles, stream) : launch<128, 64>(p, n_tiles, stream);
+    }
+    if (p.cap_in != 0.f) return d == 128 ? launch<128, 128, true>(p, n_tiles, stream) : launch<64, 64, true>(p, n_tiles, stream);
+    if (d == 128) return launch<128, 128>(p, n_tiles, stream);
+    return launch<64, 64>(p, n_tiles, stream);
 }

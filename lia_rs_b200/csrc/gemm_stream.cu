@@ -388,7 +388,7 @@ gemm_stream_kernel(Args a) {
                             value = fmaxf(value, 0.f);
                             value *= value;
                         } else if (MODE == GEMM_STORE_XIELU) {
-                            value = lia_xielu(value, a.act_p, a.act_n);
+                            value = lia_xielu_fast(value, a.act_p, a.act_n);
                         }
                         if (a.out_bf16) reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)token * a.ldo + f] = __float2bfloat16_rn(value);
                         else reinterpret_cast<float*>(a.out)[(size_t)token * a.ldo + f] = value;

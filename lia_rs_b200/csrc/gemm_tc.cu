@@ -127,7 +127,7 @@ __device__ __forceinline__ void apply_epilogue(TO* dst, float acc, float up, con
     const float alpha = s.alpha;
     if (MODE == GEMM_STORE) *dst = from_float<TO>(alpha * acc);
     else if (MODE == GEMM_STORE_RELU2) *dst = from_float<TO>(relu_squared(alpha * acc));
-    else if (MODE == GEMM_STORE_XIELU) *dst = from_float<TO>(lia_xielu(alpha * acc, s.act_p, s.act_n));
+    else if (MODE == GEMM_STORE_XIELU) *dst = from_float<TO>(lia_xielu_fast(alpha * acc, s.act_p, s.act_n));
     else if (MODE == GEMM_REGLU) *dst = from_float<TO>(up * fmaxf(acc, 0.f));
     else if (MODE == GEMM_ACCUM) *dst = from_float<TO>(to_float(*dst) + alpha * acc);
     else *dst = from_float<TO>(up * (acc / (1.0f + __expf(-acc))));
@@ -386,7 +386,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         if (MODE == GEMM_SWIGLU) v = up[c] * __fdividef(acc[c], 1.0f + __expf(-acc[c]));
                         else if (MODE == GEMM_REGLU) v = up[c] * fmaxf(acc[c], 0.f);
                         else if (MODE == GEMM_STORE_RELU2) v = relu_squared(s.alpha * acc[c]);
-                        else if (MODE == GEMM_STORE_XIELU) v = lia_xielu(s.alpha * acc[c], s.act_p, s.act_n);
+                        else if (MODE == GEMM_STORE_XIELU) v = lia_xielu_fast(s.alpha * acc[c], s.act_p, s.act_n);
                         else v = s.alpha * acc[c];
                         stage[c * TILE_F + group * 32 + lane] = from_float<TO>(v);
                     }

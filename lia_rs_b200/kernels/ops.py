@@ -51,10 +51,10 @@ class _Signatures:
                        ctypes.c_longlong, c_void_p]
     lia_wait_probe = [c_int, c_void_p, c_void_p, c_void_p]
     lia_attention_decode = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                            c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                            c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p]
-    lia_attention_decode_cluster_splits = [c_int, c_int, c_int, c_int]
-    lia_attention_decode_ctas_per_sm = [c_int, c_int]
+    lia_attention_decode_cluster_splits = [c_int, c_int, c_int, c_int, c_int]
+    lia_attention_decode_ctas_per_sm = [c_int, c_int, c_int]
     lia_gemm_tc = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                    c_void_p, ctypes.c_longlong, c_int, c_float, c_float, c_void_p, c_void_p]
     lia_gemm_cluster = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -69,9 +69,9 @@ class _Signatures:
     lia_attention_prefill = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
     lia_attention_prefill_tc = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
-                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int,
+                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int,
                                 c_float, c_void_p, c_void_p]
-    lia_attention_prefill_tc_tokens_per_tile = [c_int, c_int]
+    lia_attention_prefill_tc_tokens_per_tile = [c_int, c_int, c_int]
     lia_select_tokens = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                          ctypes.c_longlong, c_void_p]
     lia_select_tokens_scratch_floats = [c_int, c_int]
@@ -155,6 +155,9 @@ class _Signatures:
                       c_void_p]
     lia_rglru_gates = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                        c_void_p]
+    lia_rglru_gates_tc_accepts = [c_int, c_int]
+    lia_rglru_gates_tc = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                          c_void_p, c_void_p]
     lia_rglru_scan = [c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                       ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                       c_void_p]
@@ -552,7 +555,8 @@ def attention_generic(q, k_pages, v_pages, positions, slots, block_table, out, n
                "attention_generic")
 
 
-DECODE_HEAD_DIMS = (32, 64, 128)       # head sizes the tensor-core attention kernels are built for
+DECODE_HEAD_DIMS = (32, 64, 128)       # head sizes the tensor-core attention kernels are built for (keys' and values' equal)
+DECODE_HEAD_PAIRS = tuple((d, d) for d in DECODE_HEAD_DIMS) + ((64, 128), (128, 64), (32, 64), (64, 32))    # (keys', values')
 
 
 def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, out, partial, nq, nkv, d, window,
@@ -583,10 +587,13 @@ def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, o
         raise KernelError("attention_decode: counters must be int32, one per row and head group")
     if not (q.dtype == k_pages.dtype == v_pages.dtype == out.dtype == torch.bfloat16):
         raise KernelError("attention_decode is a bfloat16 kernel")
+    dv = v_pages.shape[-1]
+    if k_pages.shape[-1] != d or out.shape[-1] != nq * dv:
+        raise KernelError("attention_decode: pages and output must have the heads' sizes")
     with _timed("attention_decode", label, work_bytes):
         _check(lib().lia_attention_decode(_p(q), _p(k_pages), _p(v_pages), _p(rows), rows.shape[0], _p(positions),
                                           _p(slots), _p(block_table), block_table.shape[1], _p(out), _p(partial),
-                                          0 if partial is None else partial.numel(), _p(counters), q.shape[0], nq, nkv, d,
+                                          0 if partial is None else partial.numel(), _p(counters), q.shape[0], nq, nkv, d, dv,
                                           k_pages.shape[1], int(window or 0), scale, split_len, n_splits, _p(qkv), _p(inv_freq),
                                           int(rotary_dim), 1 if write_kv else 0, k_pages.shape[0], 1 if cluster else 0, 1 if all_new else 0,
                                           1 if sink else 0, float(softcap or 0.0), _p(error_flag),
@@ -594,15 +601,15 @@ def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, o
                "attention_decode")
 
 
-def attention_decode_cluster_splits(d: int, group: int, clusters: int, wanted: int) -> int:
+def attention_decode_cluster_splits(d: int, group: int, clusters: int, wanted: int, dv: int = None) -> int:
     """Ranges per token (2, 4, 8 or 16, at most `wanted`) with which `attention_decode(..., cluster=True)` can
     serve `clusters` (token, head group) pairs at once; 1: it cannot (one range, or too many clusters for the device)."""
-    return int(lib().lia_attention_decode_cluster_splits(d, group, clusters, wanted))
+    return int(lib().lia_attention_decode_cluster_splits(d, d if dv is None else dv, group, clusters, wanted))
 
 
-def attention_decode_ctas_per_sm(d: int, group: int) -> int:
+def attention_decode_ctas_per_sm(d: int, group: int, dv: int = None) -> int:
     """CTAs of `attention_decode` that one SM holds at once for this head size (0: unknown)."""
-    return int(lib().lia_attention_decode_ctas_per_sm(d, group))
+    return int(lib().lia_attention_decode_ctas_per_sm(d, d if dv is None else dv, group))
 
 
 def attention_prefill_tokens_per_tile(group: int) -> int:
@@ -624,10 +631,10 @@ def attention_prefill(q, k_pages, v_pages, segments, n_segments, n_tiles, slots,
                                            _p(error_flag), _stream()), "attention_prefill")
 
 
-def attention_prefill_tc_tokens_per_tile(group: int, d: int) -> int:
+def attention_prefill_tc_tokens_per_tile(group: int, d: int, dv: int = None) -> int:
     """Tokens of a portion that one CTA of the tcgen05 prefill kernel takes (0: it does not take this group
     size or head size)."""
-    return int(lib().lia_attention_prefill_tc_tokens_per_tile(group, d))
+    return int(lib().lia_attention_prefill_tc_tokens_per_tile(group, d, d if dv is None else dv))
 
 
 def attention_prefill_tc(q, k_pages, v_pages, segments, n_segments, n_tiles, slots, block_table, out, nq, nkv, d,
@@ -640,21 +647,23 @@ def attention_prefill_tc(q, k_pages, v_pages, segments, n_segments, n_tiles, slo
     _cuda(q, k_pages, v_pages, segments, slots, block_table, out, error_flag, partial)
     if not (q.dtype == k_pages.dtype == v_pages.dtype == out.dtype == torch.bfloat16):
         raise KernelError("attention_prefill_tc is a bfloat16 kernel")
-    splits = int(splits)
+    splits, dv = int(splits), v_pages.shape[-1]
+    if k_pages.shape[-1] != d or out.shape[-1] != nq * dv:
+        raise KernelError("attention_prefill_tc: pages and output must have the heads' sizes")
     if splits > 1 and (partial is None or partial.dtype != torch.float32
-                       or partial.numel() < attention_prefill_tc_partial_floats(q.shape[0], nq, d, splits)):
+                       or partial.numel() < attention_prefill_tc_partial_floats(q.shape[0], nq, dv, splits)):
         raise KernelError("attention_prefill_tc: the ranges need 32-bit scratch of attention_prefill_tc_partial_floats words")
     with _timed("attention_prefill_tc", label, 0, work_flops):
         _check(lib().lia_attention_prefill_tc(_p(q), _p(k_pages), _p(v_pages), _p(segments), n_segments, n_tiles,
-                                              _p(slots), _p(block_table), block_table.shape[1], _p(out), nq, nkv, d,
+                                              _p(slots), _p(block_table), block_table.shape[1], _p(out), nq, nkv, d, dv,
                                               k_pages.shape[1], int(window or 0), scale, k_pages.shape[0], splits,
                                               _p(partial) if splits > 1 else None, q.shape[0], 1 if sink else 0,
                                               float(softcap or 0.0), _p(error_flag), _stream()),
                "attention_prefill_tc")
 
 
-def attention_prefill_tc_partial_floats(n_tokens: int, nq: int, d: int, splits: int) -> int:
-    return int(splits) * int(n_tokens) * int(nq) * (int(d) + 2)
+def attention_prefill_tc_partial_floats(n_tokens: int, nq: int, dv: int, splits: int) -> int:
+    return int(splits) * int(n_tokens) * int(nq) * (int(dv) + 2)
 
 
 _select_scratch = {}
@@ -1512,6 +1521,29 @@ def rglru_gates(u, weight, bias, rate, slots, a_out, inflow, blocks: int):
                 flops=4 * n * width * size):
         _check(lib().lia_rglru_gates(_p(u), dtype_code(u.dtype), _p(weight), dtype_code(weight.dtype), _p(bias), _p(rate),
                                      _p(slots), _p(a_out), _p(inflow), n, width, int(blocks), _stream()), "rglru_gates")
+
+
+def rglru_gates_tc_accepts(width: int, blocks: int) -> bool:
+    """Whether the tcgen05 kernel takes parts of this size (bfloat16)."""
+    return bool(lib().lia_rglru_gates_tc_accepts(int(width), int(blocks)))
+
+
+def rglru_gates_tc(u, w_r, w_i, bias, rate, slots, a_out, inflow, blocks: int, error_flag=None):
+    """As `rglru_gates` on the tensor cores (bfloat16 u and weights): w_r, w_i [blocks, size, size] with a row per output
+    channel; see csrc/rglru_gates_tc.cu."""
+    _cuda(u, w_r, w_i, bias, rate, slots, a_out, inflow, error_flag)
+    _f32(bias, rate, a_out, inflow)
+    n, width = u.shape
+    size = width // blocks
+    if tuple(w_r.shape) != (blocks, size, size) or tuple(w_i.shape) != (blocks, size, size) or tuple(a_out.shape) != (n, width) or \
+            tuple(inflow.shape) != (n, width) or bias.numel() != 2 * width or rate.numel() != width or \
+            not (u.dtype == w_r.dtype == w_i.dtype == torch.bfloat16):
+        raise KernelError("rglru_gates_tc: shapes or element types do not agree")
+    _, sms = _device_scratch(u.device)
+    with _timed("rglru_gates_tc", nbytes=n * width * (u.element_size() + 8) + 2 * w_r.numel() * w_r.element_size(),
+                flops=4 * n * width * size):
+        _check(lib().lia_rglru_gates_tc(_p(u), _p(w_r), _p(w_i), _p(bias), _p(rate), _p(slots), _p(a_out), _p(inflow), n, width,
+                                        int(blocks), sms, _p(error_flag), _stream()), "rglru_gates_tc")
 
 
 def rglru_scan(a, inflow, y, x, y_bias, x_bias, ring, state, segments, n_segments: int, single_rows, positions, slots, out,

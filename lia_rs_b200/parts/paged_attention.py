@@ -7,6 +7,9 @@ once, and an unsupported size is refused there with its reason.  The kernels (cs
                      (attention_decode.cu), prompt portions to the tcgen05 kernel (attention_prefill_tc.cu) where it
                      takes the head size and group, else to the mma.sync kernel (attention_prefill.cu), else
                      (more than 64 query heads per kv head) to the kernel for every size;
+  With values of another head size than the keys' the same two kernels serve the pairs they are built for
+  (`ops.DECODE_HEAD_PAIRS`), and the kernel with a size for each (`ops.attention_general`) what they do not take;
+
   variant "generic"  everything else: the 32-bit path, and bfloat16 with another head size
                      (attention_generic.cu: a warp per token and head, 32-bit probabilities).  On the bfloat16
                      path this is a slow road, so it is said once when such a mixer is built.
@@ -35,8 +38,13 @@ class PagedAttention:
             raise ValueError(f"attention: head_dim {head_dim} is not a multiple of {ops.ATTENTION_HEAD_DIM_STEP} of at "
                              f"most {ops.ATTENTION_HEAD_DIM_MAX} (what the attention kernels take)")
 
+    @staticmethod
+    def takes(head_dim: int, v_head_dim: int, group: int) -> bool:
+        """Whether the tensor-core kernels take keys and values of these head sizes (bfloat16, no cap if unequal)."""
+        return (head_dim, v_head_dim) in ops.DECODE_HEAD_PAIRS and group <= 64
+
     def __init__(self, dtype: torch.dtype, heads: int, kv_heads: int, head_dim: int, window, scale: float,
-                 rotate_half=None, sink: bool = False, softcap=None):
+                 rotate_half=None, sink: bool = False, softcap=None, v_head_dim=None):
         """`rotate_half`: what the mixer's position encoding answers to `rotate_half()`; with it (and the
         tensor variant, and at most 16 query heads per kv head) decode-only steps encode, append and attend in
         one kernel (`forward_fused`).  `sink`: one is added to the softmax's denominator (the weight of a key of score 0
@@ -48,6 +56,9 @@ class PagedAttention:
         self.sink = bool(sink)
         self.softcap = None if softcap is None else float(softcap)
         self.nq, self.nkv, self.d = int(heads), int(kv_heads), int(head_dim)
+        self.dv = self.d if v_head_dim is None else int(v_head_dim)
+        if self.dv != self.d and (dtype != torch.bfloat16 or self.softcap or not self.takes(self.d, self.dv, self.nq // self.nkv)):
+            raise ValueError("attention: keys and values of unequal head sizes that no tensor-core kernel behind this class takes")
         self.window, self.scale = window, float(scale)
         self.group = self.nq // self.nkv
         self.variant = "tensor" if dtype == torch.bfloat16 and self.d in ops.DECODE_HEAD_DIMS else "generic"
@@ -60,7 +71,8 @@ class PagedAttention:
             print(f"[lia_rs_b200] bfloat16 attention with head size {self.d} runs on the kernel for every size "
                   f"(32-bit probabilities, a warp per token and head); the tensor-core kernels take "
                   f"{ops.DECODE_HEAD_DIMS}", file=sys.stderr, flush=True)
-        self.rotate_half = rotate_half if (self.variant == "tensor" and self.group <= 16 and not self.softcap) else None
+        self.rotate_half = rotate_half if (self.variant == "tensor" and self.group <= 16 and not self.softcap and
+                                           self.dv == self.d) else None
         self._prefill = None          # (kernel, tokens per tile), asked of the library at the first prompt portion
         self._decode_plans = {}       # (rows, wanted ranges) -> (ranges, as clusters)
         self._ctas_per_sm = None      # CTAs of the decode kernel that an SM holds, asked of the library at the first decode step
@@ -76,7 +88,7 @@ class PagedAttention:
         groups = self.nkv * ((self.group + 15) // 16)
         ctas = max(1, rows * groups)
         if self._ctas_per_sm is None:
-            self._ctas_per_sm = ops.attention_decode_ctas_per_sm(self.d, self.group) or 2
+            self._ctas_per_sm = ops.attention_decode_ctas_per_sm(self.d, self.group, self.dv) or 2
         wanted = (self._ctas_per_sm * ctx.runtime.sm_count) // ctas
         return max(1, min(wanted, 32, ctx.context_bucket // 256))
 
@@ -88,7 +100,7 @@ class PagedAttention:
         plan = self._decode_plans.get((rows, wanted))
         if plan is None:
             groups = self.nkv * ((self.group + 15) // 16)
-            clustered = ops.attention_decode_cluster_splits(self.d, self.group, rows * groups, wanted) if wanted >= 2 else 1
+            clustered = ops.attention_decode_cluster_splits(self.d, self.group, rows * groups, wanted, self.dv) if wanted >= 2 else 1
             plan = self._decode_plans[(rows, wanted)] = (clustered, True) if clustered >= 2 else (wanted, False)
         return plan
 
@@ -104,7 +116,7 @@ class PagedAttention:
     def _decode_scratch(self, ctx, rows: int, n_splits: int):
         if n_splits <= 1:
             return None, None
-        partial = ctx.runtime.scratch("attn.partial", ctx.n_tokens * self.nq * n_splits * (self.d + 1), torch.float32)
+        partial = ctx.runtime.scratch("attn.partial", ctx.n_tokens * self.nq * n_splits * (self.dv + 1), torch.float32)
         counters = ctx.runtime.counters(rows * self.nkv * ((self.group + 15) // 16))
         return partial, counters
 
@@ -116,16 +128,16 @@ class PagedAttention:
             return position + 1 if self.window is None else min(position + 1, self.window)
         keys = sum(visible(start) for _, start, count, _ in ctx.segments if count == 1)
         pairs = sum(visible(start + i) for _, start, count, _ in ctx.segments if count > 1 for i in range(count))
-        return keys * 2 * self.nkv * self.d * element_size, 4 * self.nq * self.d * pairs
+        return keys * self.nkv * (self.d + self.dv) * element_size, 2 * self.nq * (self.d + self.dv) * pairs
 
     def _prefill_kernel(self):
         """(kernel, tokens per tile) for prompt portions, asked of the library once."""
         if self._prefill is None:
-            per_tile = ops.attention_prefill_tc_tokens_per_tile(self.group, self.d)
+            per_tile = ops.attention_prefill_tc_tokens_per_tile(self.group, self.d, self.dv)
             if per_tile:
                 self._prefill = (ops.attention_prefill_tc, per_tile)
-            elif self.softcap:
-                self._prefill = (None, 0)           # the mma.sync prompt kernel has no cap: the kernel for every size serves
+            elif self.softcap or self.dv != self.d:
+                self._prefill = (None, 0)           # the mma.sync prompt kernel has no cap and one head size: the kernel for every size serves
             else:
                 self._prefill = (ops.attention_prefill, ops.attention_prefill_tokens_per_tile(self.group))
         return self._prefill
@@ -173,15 +185,16 @@ class PagedAttention:
                 if kernel is ops.attention_prefill_tc:
                     splits = self.prefill_splits(ctx, tiles)
                     if splits > 1:
-                        words = ops.attention_prefill_tc_partial_floats(ctx.n_tokens, nq, d, splits)
+                        words = ops.attention_prefill_tc_partial_floats(ctx.n_tokens, nq, self.dv, splits)
                         more = dict(splits=splits, partial=ctx.runtime.scratch("attn.prefill_partial", words, torch.float32))
                 kernel(q, kv.k_pages, kv.v_pages, ctx.prefill_segments, ctx.n_prefill_segments, tiles, ctx.slots,
                        kv.block_table, out, nq, nkv, d, self.window, self.scale, ctx.error_flag, work_flops=work_flops,
                        sink=self.sink, **more, **({"softcap": self.softcap} if self.softcap else {}))
-            elif self.softcap:
-                ops.attention_general(q, (nq * d, d), None, None, kv.k_pages, None, kv.v_pages, d, d, ctx.positions, ctx.slots,
-                                      kv.block_table, out, (nq * d, d), ctx.n_tokens, nq, nkv, self.window, self.scale,
-                                      rows=ctx.prefill_rows, error_flag=ctx.error_flag, softcap=self.softcap)
+            elif self.softcap or self.dv != d:
+                dv = self.dv
+                ops.attention_general(q, (nq * d, d), None, None, kv.k_pages, None, kv.v_pages, dv, dv, ctx.positions, ctx.slots,
+                                      kv.block_table, out, (nq * dv, dv), ctx.n_tokens, nq, nkv, self.window, self.scale,
+                                      sink=self.sink, rows=ctx.prefill_rows, error_flag=ctx.error_flag, softcap=self.softcap)
             else:
                 ops.attention_generic(q, kv.k_pages, kv.v_pages, ctx.positions, ctx.slots, kv.block_table, out, nq, nkv,
                                       d, self.window, self.scale, rows=ctx.prefill_rows, error_flag=ctx.error_flag)

@@ -83,8 +83,13 @@ class RGLRU(Mixer):
         self.w_o = prepare_weight(tensors[n["o"]], runtime)
         self.y_bias, self.x_bias = f32(tensors[n["y_bias"]]), f32(tensors[n["x_bias"]])
         self.conv, self.conv_bias = f32(tensors[n["conv"]].t()), f32(tensors[n["conv_bias"]])
-        # part b's two matrices side by side, transposed: [in][r's outputs | i's outputs]
-        self.w_gates = prepare_weight(torch.cat([tensors[n["r"]].transpose(1, 2), tensors[n["i"]].transpose(1, 2)], dim=2), runtime)
+        # bfloat16: the tensor-core kernel's matrices as they are stored; else part b's two side by side, transposed
+        # ([in][r's outputs | i's outputs])
+        self.tensor_cores = runtime.compute_dtype == torch.bfloat16 and ops.rglru_gates_tc_accepts(self.width, self.blocks)
+        if self.tensor_cores:
+            self.w_r, self.w_i = prepare_weight(tensors[n["r"]], runtime), prepare_weight(tensors[n["i"]], runtime)
+        else:
+            self.w_gates = prepare_weight(torch.cat([tensors[n["r"]].transpose(1, 2), tensors[n["i"]].transpose(1, 2)], dim=2), runtime)
         self.gate_bias = f32(torch.stack([tensors[n["r_bias"]].reshape(-1), tensors[n["i_bias"]].reshape(-1)]))
         self.rate = (8.0 * torch.nn.functional.softplus(tensors[n["lam"]].to(torch.float32))).contiguous()
 
@@ -102,7 +107,10 @@ class RGLRU(Mixer):
         ops.ring_conv(v, self.x_bias, self.conv, self.conv_bias, ring, ctx.positions, ctx.slots, u)
         a = ctx.buffer("rglru.a", (n, width), torch.float32)
         inflow = ctx.buffer("rglru.inflow", (n, width), torch.float32)
-        ops.rglru_gates(u, self.w_gates, self.gate_bias, self.rate, ctx.slots, a, inflow, self.blocks)
+        if self.tensor_cores:
+            ops.rglru_gates_tc(u, self.w_r, self.w_i, self.gate_bias, self.rate, ctx.slots, a, inflow, self.blocks, error_flag=flag)
+        else:
+            ops.rglru_gates(u, self.w_gates, self.gate_bias, self.rate, ctx.slots, a, inflow, self.blocks)
         out = ctx.buffer("rglru.out", (n, width), rt.compute_dtype)
         ops.rglru_scan(a, inflow, y, v, self.y_bias, self.x_bias, ring, memory, ctx.prefill_segments, ctx.n_prefill_segments,
                        ctx.decode_rows, ctx.positions, ctx.slots, out, taps)

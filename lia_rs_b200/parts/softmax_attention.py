@@ -33,8 +33,8 @@ layer has no W_dkv and reads the latents and rotated parts that another layer of
 pages (the model's schedule names that layer's cache), with W_uk, W_uv and queries of its own.
 
 Scores, softmax, norms and angles are 32-bit in both.  Which kernel serves which rows: the kernel for every size and
-element type (csrc/attention_generic.cu, `attention_general`); `sink_attention` in bfloat16 with equal key and value
-head sizes that the tensor-core kernels take uses those (`PagedAttention` with its `sink`)."""
+element type (csrc/attention_generic.cu, `attention_general`); `sink_attention` in bfloat16 with key and value head sizes
+that the tensor-core kernels take uses those (`PagedAttention` with its `sink`)."""
 from __future__ import annotations
 
 import torch
@@ -164,13 +164,13 @@ class SinkAttention(Mixer):
         self.rot_dims, self.freq = _frequencies(params.get("rot"), device)
         self.mix_mode = {None: 0, "source": 1, "mixed": 2}[params.get("value_mix")]
         self.mix_lambda = float(tensors[n["mix"]].to(torch.float32)) if self.mix_mode == 2 else 0.0
-        # bfloat16 with keys and values of one head size that the tensor-core kernels take: those kernels; else the
-        # kernel for every size
+        # bfloat16 with keys and values of head sizes that the tensor-core kernels take: those kernels; else the kernel
+        # for every size
         self.paged = None
-        if runtime.compute_dtype == torch.bfloat16 and self.d == self.dv and self.d in ops.DECODE_HEAD_DIMS and \
-                self.nq // self.nkv <= 64:
+        if runtime.compute_dtype == torch.bfloat16 and PagedAttention.takes(self.d, self.dv, self.nq // self.nkv) and \
+                not (self.softcap and self.d != self.dv):
             self.paged = PagedAttention(runtime.compute_dtype, self.nq, self.nkv, self.d, self.window, self.scale, sink=self.sink,
-                                        softcap=self.softcap)
+                                        softcap=self.softcap, v_head_dim=self.dv)
 
     def graph_key(self, ctx) -> tuple:
         return self.paged.graph_key(ctx) if self.paged is not None else ()
