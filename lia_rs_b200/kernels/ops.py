@@ -1558,7 +1558,7 @@ def rglru_scan(a, inflow, y, x, y_bias, x_bias, ring, state, segments, n_segment
             tuple(inflow.shape) != (n, width):
         raise KernelError("rglru_scan: shapes do not agree")
     stride = _slots_of(state, (width,), "rglru_scan")
-    if taps > 1 and _slots_of(ring, (taps, width), "rglru_scan") != stride:
+    if taps > 1 and _slots_of(ring, (taps, width), "rglru_scan") != stride and state.shape[0] > 1:
         raise KernelError("rglru_scan: ring and state must have one slot stride")
     with _timed("rglru_scan", nbytes=n * width * (12 + out.element_size())):
         _check(lib().lia_rglru_scan(_p(a), _p(inflow), _p(y), _p(x), y.stride(0), _p(y_bias), _p(x_bias),

@@ -145,7 +145,7 @@ def grouped_gated_norm(y, z, weight, groups, eps):
 def mamba2(h, w, m, eps):
     """[z | x | B | C | dt] = W_in h; x, B and C through the convolution and SiLU; dt <- softplus(dt + dt_bias); the
     heads' recurrence; the gated norm in groups; W_o."""
-    heads, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+    heads, P, N, G = m["heads"], m["vdim"], m["state"], m.get("groups", 1)
     inner, T = heads * P, h.shape[0]
     rows = h @ w["in"].to(F64).T
     z, xbc, dt = rows[:, :inner], rows[:, inner:2 * inner + 2 * G * N], rows[:, 2 * inner + 2 * G * N:]
@@ -155,7 +155,7 @@ def mamba2(h, w, m, eps):
     B = xbc[:, inner:inner + G * N].reshape(T, G, N)
     C = xbc[:, inner + G * N:].reshape(T, G, N)
     y, _ = head_recurrence(x, B, C, dt, w["A_log"], w["D"])
-    y = grouped_gated_norm(y.reshape(T, inner), z, w["norm"], m["norm_groups"], eps)
+    y = grouped_gated_norm(y.reshape(T, inner), z, w["norm"], m.get("norm_groups", 1), eps)
     return y @ w["o"].to(F64).T
 
 
@@ -187,7 +187,7 @@ def forward(config: dict, tensors: dict, tokens, layer_outputs=None):
     stream after every layer."""
     eps = float(config["norm"]["eps"])
     positions = torch.arange(len(tokens))
-    x = embedding(torch.tensor(list(tokens), dtype=torch.long), positions, tensors["embed"], float(config["embedding"]["scale"]))
+    x = embedding(torch.tensor(list(tokens), dtype=torch.long), positions, tensors["embed"], float((config.get("embedding") or {}).get("scale", 1.0)))
     for n, layer in enumerate(config["layers"]):
         w = _under(tensors, f"l{n}.")
         mixer = _under(w, "mix.")
