@@ -14,29 +14,26 @@
 //  * `gated_group_norm`: y * silu(z), in `groups` equal parts of a row each over its own root mean square, times a weight.
 // Everything is 32-bit; only the normed rows have the compute element type.  A row whose slot is negative belongs to nobody
 // and is skipped.
-#include "conv_ring.cuh"
 #include "linear_recurrence.cuh"
+#include "state_space.cuh"
 
 namespace {
-constexpr int SSD_THREADS = 256;
-constexpr int SSD_MAX = 256;                  // largest state size N and largest head size P
-constexpr float LOG2_E = 1.4426950408889634f;
-
-struct SsdArgs {
-    const float* xbc; long long ld;           // [n, ld] [x | B | C]
-    const float* dt; long long ld_dt;         // [n, ld_dt] raw step sizes, one a head
-    const float* dt_bias; const float* rate;  // [heads]; rate = exp(A_log)
-    const float* skip;                        // D [heads]
-    float* state; long long slot_stride;      // slot s: [heads, N, P]
-    const int* segments; int n_segments; const int* single_rows; const int* slots;
-    float* y;                                 // [n, heads P]
-    float* sums; float* totals;               // [chunks, heads, N, P], [chunks, heads]
-    int heads, groups, N, P, vec;
+// Where a single token's x, B and C come from: the convolution's rows (`raw` null), or the input product's rows, and the
+// kernel does the convolution of the channels that its head reads itself (a step of single tokens alone: no other row of
+// the step is an earlier input of a token, all of them lie in its ring).
+struct SingleInput {
+    const float* raw; long long ld_raw;       // [n, ld_raw] [x | B | C] ahead of the convolution
+    const float* weight; const float* bias;   // [taps, channels], [channels] or null
+    float* ring; long long ring_stride;       // slot s: [taps, channels]
+    const int* positions;
+    int taps, channels, round16;              // round16: the convolution's result is rounded to bfloat16, as its rows would be
+    const void* rows; int rows_bf16;          // [n, ld] out of the convolution
 };
 
+template <int VEC>                            // columns of the state that a thread takes (4: P and the addresses allow it)
 __global__ void __launch_bounds__(SSD_THREADS)
-ssd_single_kernel(SsdArgs p) {
-    extern __shared__ float ssd_single_shared[];          // B [N], C [N], partial sums [max(SSD_THREADS, P)]
+ssd_single_kernel(SsdArgs p, SingleInput in) {
+    extern __shared__ float ssd_single_shared[];          // B [N], C [N], x [P], partial sums [SSD_THREADS VEC]
     pdl_launch_dependents();
     pdl_wait();
     const int t = p.single_rows[blockIdx.x], h = blockIdx.y;
@@ -46,50 +43,86 @@ ssd_single_kernel(SsdArgs p) {
     const int N = p.N, P = p.P;
     float* bs = ssd_single_shared;
     float* cs = bs + N;
-    float* partial = cs + N;
-    const float* row = p.xbc + (size_t)t * p.ld;
-    const int g = h / (p.heads / p.groups);
-    for (int i = threadIdx.x; i < N; i += blockDim.x) {
-        bs[i] = row[(size_t)p.heads * P + (size_t)g * N + i];
-        cs[i] = row[(size_t)p.heads * P + (size_t)(p.groups + g) * N + i];
+    float* xs = cs + N;
+    float* partial = xs + P;
+    const int per_group = p.heads / p.groups, g = h / per_group;
+    const int b_at = p.heads * P + g * N, c_at = p.heads * P + (p.groups + g) * N;
+    const int pos = in.raw ? in.positions[t] : 0;
+    float* ring = in.ring ? in.ring + (size_t)slot * in.ring_stride : nullptr;
+    for (int e = threadIdx.x; e < 2 * N + P; e += SSD_THREADS) {
+        const int c = e < N ? b_at + e : e < 2 * N ? c_at + e - N : h * P + e - 2 * N;
+        float v;
+        if (in.raw) {
+            const float own = in.raw[(size_t)t * in.ld_raw + c];
+            v = in.bias ? in.bias[c] : 0.f;
+            for (int j = 0; j < in.taps - 1; ++j) {
+                const int k = in.taps - 1 - j;
+                const float earlier = pos - k >= 0 ? ring[(size_t)((pos - k) % in.taps) * in.channels + c] : 0.f;
+                v = fmaf(in.weight[(size_t)j * in.channels + c], earlier, v);
+            }
+            v = ring_silu(fmaf(in.weight[(size_t)(in.taps - 1) * in.channels + c], own, v));
+            if (in.round16) v = to_float(from_float<__nv_bfloat16>(v));
+            // the head's own channels, and the group's by its first head (the row written is none of those read)
+            if (in.taps > 1 && (e >= 2 * N || h == g * per_group)) ring[(size_t)(pos % in.taps) * in.channels + c] = own;
+        } else if (in.rows_bf16) {
+            v = to_float(reinterpret_cast<const __nv_bfloat16*>(in.rows)[(size_t)t * p.ld + c]);
+        } else {
+            v = reinterpret_cast<const float*>(in.rows)[(size_t)t * p.ld + c];
+        }
+        bs[e] = v;
     }
     const float dt = ring_softplus(p.dt[(size_t)t * p.ld_dt + h] + p.dt_bias[h]);
     const float decay = expf(-p.rate[h] * dt);
-    __syncthreads();
     float* S = p.state + (size_t)slot * p.slot_stride + (size_t)h * N * P;
-    int lanes = 32;
-    while (lanes < P && lanes < SSD_THREADS) lanes <<= 1;
-    const int rows = SSD_THREADS / lanes;
-    const int lane = threadIdx.x % lanes, group = threadIdx.x / lanes;
-    for (int j = lane; j < P; j += lanes) {
-        const float xj = dt * row[(size_t)h * P + j];
-        float acc = 0.f;
-        constexpr int AHEAD = 8;                          // (eight rows of the state at a time: their loads are in flight together)
-        for (int i0 = group; i0 < N; i0 += rows * AHEAD) {
-            float held[AHEAD];
+    const int lanes = P / VEC, rows = SSD_THREADS / lanes;
+    const int group = threadIdx.x / lanes, j = (threadIdx.x % lanes) * VEC;
+    constexpr int AHEAD = 8;                              // (eight rows of the state at a time: their loads are in flight together)
+    float held[AHEAD][VEC];
+    auto load = [&](int i0) {
 #pragma unroll
-            for (int k = 0; k < AHEAD; ++k) {
-                const int i = i0 + k * rows;
-                held[k] = i < N ? S[(size_t)i * P + j] : 0.f;
-            }
-#pragma unroll
-            for (int k = 0; k < AHEAD; ++k) {
-                const int i = i0 + k * rows;
-                if (i < N) {
-                    const float s = fmaf(decay, held[k], bs[i] * xj);
-                    S[(size_t)i * P + j] = s;
-                    acc = fmaf(s, cs[i], acc);
+        for (int k = 0; k < AHEAD; ++k) {
+            const int i = i0 + k * rows;
+            if (group < rows && i < N) {
+                if constexpr (VEC == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(S + (size_t)i * P + j);
+                    held[k][0] = v.x, held[k][1] = v.y, held[k][2] = v.z, held[k][3] = v.w;
+                } else {
+                    held[k][0] = S[(size_t)i * P + j];
                 }
             }
         }
-        if (rows > 1) partial[group * lanes + lane] = acc;
-        else partial[j] = acc;
+    };
+    load(group);                                          // (under way while x, B and C arrive)
+    __syncthreads();
+    if (group < rows) {
+        float xj[VEC], acc[VEC];
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) xj[v] = dt * xs[j + v], acc[v] = 0.f;
+        for (int i0 = group; i0 < N; i0 += rows * AHEAD) {
+            if (i0 != group) load(i0);
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) {
+                const int i = i0 + k * rows;
+                if (i >= N) break;
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) {
+                    held[k][v] = fmaf(decay, held[k][v], bs[i] * xj[v]);
+                    acc[v] = fmaf(held[k][v], cs[i], acc[v]);
+                }
+                if constexpr (VEC == 4)
+                    *reinterpret_cast<float4*>(S + (size_t)i * P + j) = make_float4(held[k][0], held[k][1], held[k][2], held[k][3]);
+                else
+                    S[(size_t)i * P + j] = held[k][0];
+            }
+        }
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) partial[group * P + j + v] = acc[v];
     }
     __syncthreads();
-    for (int j = threadIdx.x; j < P; j += blockDim.x) {
-        float o = partial[j];
-        for (int r = 1; r < rows; ++r) o += partial[r * lanes + j];
-        p.y[(size_t)t * p.heads * P + (size_t)h * P + j] = fmaf(p.skip[h], row[(size_t)h * P + j], o);
+    for (int c = threadIdx.x; c < P; c += SSD_THREADS) {
+        float o = partial[c];
+        for (int r = 1; r < rows; ++r) o += partial[r * P + c];
+        p.y[(size_t)t * p.heads * P + (size_t)h * P + c] = fmaf(p.skip[h], xs[c], o);
     }
 }
 
@@ -153,45 +186,6 @@ ssd_sums_kernel(SsdArgs p) {
 #pragma unroll
             for (int y = 0; y < 4; ++y)
                 if (i0 + x < N && j0 + y < P) U[(size_t)(i0 + x) * P + j0 + y] = acc[x][y];
-    }
-}
-
-// along each portion: scratch[c] <- the state chunk c starts from; S <- 2^C_len S + U_c; state <- the last S
-__global__ void __launch_bounds__(SSD_THREADS)
-ssd_carry_kernel(SsdArgs p, int chunk_length) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int s = blockIdx.x, h = blockIdx.y;
-    if (s >= p.n_segments) return;
-    const int first = p.segments[3 * s], count = p.segments[3 * s + 2];
-    const int slot = p.slots[first];
-    if (slot < 0) return;
-    int before = 0;
-    for (int q = 0; q < s; ++q) before += (p.segments[3 * q + 2] + chunk_length - 1) / chunk_length;
-    const int chunks = (count + chunk_length - 1) / chunk_length;
-    const int size = p.N * p.P;
-    float* S = p.state + (size_t)slot * p.slot_stride + (size_t)h * size;
-    const size_t chunk_stride = (size_t)p.heads * size;
-    const float* total = p.totals + (size_t)before * p.heads + h;
-    for (int e = blockIdx.z * blockDim.x + threadIdx.x; e < size; e += gridDim.z * blockDim.x) {
-        float value = S[e];
-        float* U = p.sums + ((size_t)before * p.heads + h) * size + e;
-        constexpr int AHEAD = 8;                          // (the loads of eight chunks are in flight together)
-        for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-            float u[AHEAD], a[AHEAD];
-#pragma unroll
-            for (int k = 0; k < AHEAD; ++k) {
-                u[k] = c0 + k < chunks ? U[(size_t)(c0 + k) * chunk_stride] : 0.f;
-                a[k] = c0 + k < chunks ? total[(size_t)(c0 + k) * p.heads] : 0.f;
-            }
-#pragma unroll
-            for (int k = 0; k < AHEAD; ++k)
-                if (c0 + k < chunks) {
-                    U[(size_t)(c0 + k) * chunk_stride] = value;
-                    value = fmaf(exp2f(a[k]), value, u[k]);
-                }
-        }
-        S[e] = value;
     }
 }
 
@@ -344,15 +338,15 @@ LIA_EXPORT long long lia_ssd_scratch_floats(int chunks, int heads, int N, int P)
 
 // xbc [n, ld] = [x: heads P | B: groups N | C: groups N], dt [n, ld_dt] (heads columns), dt_bias, rate, skip [heads], state
 // (slot s at + s slot_stride: [heads, N, P]), y [n, heads P], scratch: `lia_ssd_scratch_floats(max_chunks, ...)` words: all
-// 32-bit.  `segments` [n_segments, 3] and `single_rows` [n_single] name the step's runs.
+// 32-bit.  `segments` [n_segments, 3] names the step's portions; single tokens go to lia_ssd_single.
 LIA_EXPORT int lia_ssd(const float* xbc, long long ld, const float* dt, long long ld_dt, const float* dt_bias,
                        const float* rate, const float* skip, float* state, long long slot_stride, const int* segments,
-                       int n_segments, int max_chunks, const int* single_rows, int n_single, const int* slots, float* y,
+                       int n_segments, int max_chunks, const int* slots, float* y,
                        int heads, int groups, int N, int P, float* scratch, long long scratch_floats, cudaStream_t stream) {
     if (heads <= 0 || groups <= 0 || heads % groups || N <= 0 || P <= 0 || N > SSD_MAX || P > SSD_MAX ||
         ld < (long long)heads * P + 2LL * groups * N || ld_dt < heads || slot_stride < (long long)heads * N * P || heads > 65535)
         return LIA_ERR_SIZE;
-    SsdArgs p = {xbc, ld, dt, ld_dt, dt_bias, rate, skip, state, slot_stride, segments, n_segments, single_rows, slots, y,
+    SsdArgs p = {xbc, ld, dt, ld_dt, dt_bias, rate, skip, state, slot_stride, segments, n_segments, nullptr, slots, y,
                  scratch, nullptr, heads, groups, N, P, 0};
     int code = LIA_OK;
     if (n_segments > 0) {
@@ -376,11 +370,33 @@ LIA_EXPORT int lia_ssd(const float* xbc, long long ld, const float* dt, long lon
         code = lia_launch(ssd_output_kernel, dim3(max_chunks, heads), dim3(SSD_THREADS), out_bytes, stream, p);
         if (code != LIA_OK) return code;
     }
-    if (n_single > 0) {
-        const size_t bytes = ((size_t)2 * N + (P > SSD_THREADS ? P : SSD_THREADS)) * sizeof(float);
-        code = lia_launch(ssd_single_kernel, dim3(n_single, heads), dim3(SSD_THREADS), bytes, stream, p);
-    }
     return code;
+}
+
+// The single tokens alone.  With `raw` (the input product's rows [n, ld_raw]; a step of single tokens alone): the kernel does
+// the convolution (weight [taps, channels], bias [channels] or null, ring as for lia_ring_conv) and leaves each token's inputs
+// in its ring; `round16`: x, B and C are rounded to bfloat16.  Else xbc [n, ld] of xbc_dtype comes from the convolution.
+// The other arguments as for lia_ssd.
+LIA_EXPORT int lia_ssd_single(const void* xbc, int xbc_dtype, long long ld, const float* raw, long long ld_raw,
+                              const float* weight, const float* bias, float* ring, long long ring_stride, const int* positions,
+                              int taps, int round16, const float* dt, long long ld_dt, const float* dt_bias, const float* rate,
+                              const float* skip, float* state, long long slot_stride, const int* single_rows, int n_single,
+                              const int* slots, float* y, int heads, int groups, int N, int P, cudaStream_t stream) {
+    if (n_single <= 0) return LIA_OK;
+    const long long channels = (long long)heads * P + 2LL * groups * N;
+    if (heads <= 0 || groups <= 0 || heads % groups || N <= 0 || P <= 0 || N > SSD_MAX || P > SSD_MAX || ld_dt < heads ||
+        slot_stride < (long long)heads * N * P || heads > 65535 || channels > 2147483647LL)
+        return LIA_ERR_SIZE;
+    if (raw ? (taps < 1 || taps > RING_MAX_TAPS || ld_raw < channels || !weight || !positions || (taps > 1 && !ring)) : (!xbc || ld < channels))
+        return LIA_ERR_SIZE;
+    if (!raw && xbc_dtype != LIA_F32 && xbc_dtype != LIA_BF16) return LIA_ERR_DTYPE;
+    SsdArgs p = {nullptr, ld, dt, ld_dt, dt_bias, rate, skip, state, slot_stride, nullptr, 0, single_rows, slots, y,
+                 nullptr, nullptr, heads, groups, N, P, 0};
+    SingleInput in = {raw, ld_raw, weight, bias, ring, ring_stride, positions, taps, (int)channels, round16, xbc, xbc_dtype == LIA_BF16};
+    const bool four = P % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15u) == 0;
+    const size_t bytes = ((size_t)2 * N + P + SSD_THREADS * (four ? 4 : 1)) * sizeof(float);
+    if (four) return lia_launch(ssd_single_kernel<4>, dim3(n_single, heads), dim3(SSD_THREADS), bytes, stream, p, in);
+    return lia_launch(ssd_single_kernel<1>, dim3(n_single, heads), dim3(SSD_THREADS), bytes, stream, p, in);
 }
 
 // y [n, groups size] and z [n, ld_z] 32-bit, weight [groups size] 32-bit, out [n, groups size] of out_dtype.

@@ -162,8 +162,13 @@ class _Signatures:
                       ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                       c_void_p]
     lia_ssd = [c_void_p, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong,
-               c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
-               ctypes.c_longlong, c_void_p]
+               c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, ctypes.c_longlong, c_void_p]
+    lia_ssd_tc = lia_ssd
+    lia_ssd_tc_accepts = [c_int, c_int]
+    lia_ssd_tc_chunks = [c_int, c_int]
+    lia_ssd_single = [c_void_p, c_int, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p,
+                      ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p,
+                      c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
     lia_gated_group_norm = [c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
                             c_void_p]
     lia_retention_chunks = [c_int, c_int]
@@ -1571,24 +1576,70 @@ def ssd_scratch_floats(chunks: int, heads: int, states: int, size: int) -> int:
     return chunks * heads * (states * size + 1)
 
 
-def ssd(xbc, dt, dt_bias, rate, skip, state, segments, n_segments: int, max_chunks: int, single_rows, slots, y, heads: int,
-        groups: int, states: int, size: int, scratch=None):
-    """S <- exp(-rate dt) S + dt B x^T, y = S^T C + skip x per head with dt = softplus(dt + dt_bias), along the step's runs;
-    xbc [n, heads size + 2 groups states] = [x | B | C], dt [n, heads] columns of wider rows, state [slots, heads, states,
-    size], y [n, heads size]: all 32-bit; see csrc/state_space.cu."""
-    _cuda(dt_bias, rate, skip, segments, single_rows, slots, y, scratch)
-    _f32(xbc, dt, dt_bias, rate, skip, y, scratch)
-    n = y.shape[0]
-    n_single = 0 if single_rows is None else single_rows.numel()
-    if xbc.stride(1) != 1 or dt.stride(1) != 1 or xbc.shape[1] != heads * size + 2 * groups * states or dt.shape[1] != heads or \
-            xbc.shape[0] != n or dt.shape[0] != n or y.shape[1] != heads * size:
+def ssd_tc_accepts(states: int, size: int) -> bool:
+    """Whether the tensor-core kernels take portions with these sizes (bfloat16 x, B and C)."""
+    return bool(lib().lia_ssd_tc_accepts(int(states), int(size)))
+
+
+def ssd_chunks(portion_tokens: int, n_segments: int, tensor_cores: bool) -> int:
+    """Most chunks that a step's portions are cut into."""
+    fn = lib().lia_ssd_tc_chunks if tensor_cores else lib().lia_retention_chunks
+    return int(fn(int(portion_tokens), int(n_segments)))
+
+
+def _check_ssd(dt, state, y, heads, groups, states, size):
+    if dt.stride(1) != 1 or dt.shape[1] != heads or dt.shape[0] != y.shape[0] or y.shape[1] != heads * size:
         raise KernelError("ssd: shapes do not agree")
-    stride = _slots_of(state, (heads, states, size), "ssd")
-    with _timed("ssd", nbytes=n * heads * size * 8 + 2 * n_single * heads * states * size * 4,
-                flops=4 * n * heads * states * size):
-        _check(lib().lia_ssd(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(rate), _p(skip), _p(state), stride,
-                             _p(segments), int(n_segments), int(max_chunks), _p(single_rows), n_single, _p(slots), _p(y), heads,
-                             groups, states, size, _p(scratch), 0 if scratch is None else scratch.numel(), _stream()), "ssd")
+    return _slots_of(state, (heads, states, size), "ssd")
+
+
+def ssd(xbc, dt, dt_bias, rate, skip, state, segments, n_segments: int, max_chunks: int, slots, y, heads: int, groups: int,
+        states: int, size: int, scratch):
+    """S <- exp(-rate dt) S + dt B x^T, y = S^T C + skip x per head with dt = softplus(dt + dt_bias), along the step's portions;
+    xbc [n, heads size + 2 groups states] = [x | B | C], 32-bit (on the 32-bit pipes, csrc/state_space.cu) or bfloat16 (on the
+    tensor cores where `ssd_tc_accepts`, csrc/state_space_tc.cu); dt [n, heads] columns of wider rows, state [slots, heads,
+    states, size], y [n, heads size]: 32-bit."""
+    _cuda(dt_bias, rate, skip, segments, slots, y, scratch)
+    _f32(dt, dt_bias, rate, skip, y, scratch)
+    stride = _check_ssd(dt, state, y, heads, groups, states, size)
+    if xbc.stride(1) != 1 or xbc.shape[1] != heads * size + 2 * groups * states or xbc.shape[0] != y.shape[0] or \
+            xbc.dtype not in (torch.float32, torch.bfloat16):
+        raise KernelError("ssd: shapes do not agree")
+    n = y.shape[0]
+    fn, name = (lib().lia_ssd_tc, "ssd_tc") if xbc.dtype == torch.bfloat16 else (lib().lia_ssd, "ssd")
+    with _timed(name, nbytes=n * (heads * size * 4 + xbc.shape[1] * xbc.element_size()), flops=4 * n * heads * states * size):
+        _check(fn(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(rate), _p(skip), _p(state), stride,
+                  _p(segments), int(n_segments), int(max_chunks), _p(slots), _p(y), heads, groups, states, size, _p(scratch),
+                  0 if scratch is None else scratch.numel(), _stream()), name)
+
+
+def ssd_single(dt, dt_bias, rate, skip, state, single_rows, slots, y, heads: int, groups: int, states: int, size: int, xbc=None,
+               conv=None):
+    """The same recurrence for the step's single tokens, state in place: from the convolution's rows `xbc` (32-bit or bfloat16),
+    or with `conv` = (raw rows, weight [taps, channels], bias, ring, positions, rounded to bfloat16) in a step of single tokens
+    alone: the kernel does the convolution itself and leaves each token's inputs in its ring."""
+    _cuda(dt_bias, rate, skip, single_rows, slots, y)
+    _f32(dt, dt_bias, rate, skip, y)
+    stride = _check_ssd(dt, state, y, heads, groups, states, size)
+    channels, n_single = heads * size + 2 * groups * states, single_rows.numel()
+    raw = weight = bias = ring = positions = None
+    taps = ring_stride = round16 = 0
+    if conv is not None:
+        raw, weight, bias, ring, positions, round16 = conv
+        _cuda(weight, bias, positions)
+        _f32(raw, weight, bias)
+        taps = weight.shape[0]
+        if raw.stride(1) != 1 or raw.shape != (y.shape[0], channels) or weight.shape[1] != channels:
+            raise KernelError("ssd_single: rows and weight of the convolution's channels")
+        ring_stride = _slots_of(ring, (taps, channels), "ssd_single") if taps > 1 else 0
+    elif xbc is None or xbc.stride(1) != 1 or xbc.shape != (y.shape[0], channels):
+        raise KernelError("ssd_single: rows of the convolution's channels")
+    with _timed("ssd_single", nbytes=n_single * heads * (2 * states * size * 4 + size * 8)):
+        _check(lib().lia_ssd_single(_p(xbc), F32 if xbc is None else dtype_code(xbc.dtype), channels if xbc is None else xbc.stride(0),
+                                    _p(raw), 0 if raw is None else raw.stride(0), _p(weight), _p(bias), _p(ring) if taps > 1 else None,
+                                    ring_stride, _p(positions), taps, 1 if round16 else 0, _p(dt), dt.stride(0), _p(dt_bias), _p(rate),
+                                    _p(skip), _p(state), stride, _p(single_rows), n_single, _p(slots), _p(y), heads, groups, states,
+                                    size, _stream()), "ssd_single")
 
 
 def gated_group_norm(y, z, weight, slots, out, groups: int, eps: float):

@@ -9,8 +9,10 @@
 
 What a request carries from token to token is one 32-bit state per slot: the convolution's last inputs in a ring of `taps`
 rows (csrc/conv_ring.cuh) and S [heads, state, size].  Step sizes, decays, exponentials, the state, the sums over it, the
-gate and the norm are 32-bit (csrc/state_space.cu).  Single tokens update the state in place; prompt portions are cut into
-chunks that run side by side and continue from the slot's state.
+gate and the norm are 32-bit (csrc/state_space.cu).  Single tokens update the state in place (in a step of single tokens alone
+that kernel does the convolution too); prompt portions are cut into chunks that run side by side and continue from the slot's
+state, in bfloat16 on the tensor cores where they take the sizes (csrc/state_space_tc.cu: x, B and C are then rounded to
+bfloat16 behind the convolution, in every kind of step).
 
 Parameters: hidden, heads, size, state, groups, norm_groups, taps, norm_eps, and optionally `names`."""
 from __future__ import annotations
@@ -92,6 +94,8 @@ class StateSpace(Mixer):
         self.w_o = prepare_weight(tensors[n["o"]], runtime)
         self.conv, self.conv_bias = f32(tensors[n["conv"]].t()), f32(tensors[n["conv_bias"]])
         self.dt_bias, self.skip, self.norm = f32(tensors[n["dt_bias"]]), f32(tensors[n["D"]]), f32(tensors[n["norm"]])
+        # bfloat16 with sizes that the tensor-core kernels take: x, B and C are bfloat16 behind the convolution
+        self.tensor_cores = runtime.compute_dtype == torch.bfloat16 and ops.ssd_tc_accepts(self.states, self.size)
         self.rate = torch.exp(tensors[n["A_log"]].to(torch.float32)).contiguous()
 
     def forward(self, ctx, x, residual, scale, kv=None, state=None, store=False):
@@ -104,16 +108,24 @@ class StateSpace(Mixer):
         rows = ctx.buffer("ssd.in", (n, self.width), torch.float32)
         linear(rt, STORE, x, self.w_in, rows, error_flag=flag, name="ssd_in")
         z, raw, dt = rows[:, :inner], rows[:, inner:inner + conv], rows[:, inner + conv:inner + conv + heads]
-        xbc = ctx.buffer("ssd.xbc", (n, conv), torch.float32)
-        ops.ring_conv(raw, None, self.conv, self.conv_bias, ring, ctx.positions, ctx.slots, xbc, act=1)
-        if taps > 1:
-            ops.ring_store(raw, None, ring, ctx.positions, ctx.slots)
-        portions = ctx.n_prefill_segments
-        chunks = ops.retention_chunks(n - ctx.n_single, portions) if portions else 0
-        scratch = ctx.runtime.scratch("ssd.chunks", ops.ssd_scratch_floats(chunks, heads, states, size), torch.float32) if chunks else None
+        portions, single = ctx.n_prefill_segments, ctx.decode_rows
         y = ctx.buffer("ssd.y", (n, inner), torch.float32)
-        ops.ssd(xbc, dt, self.dt_bias, self.rate, self.skip, memory, ctx.prefill_segments, portions, chunks, ctx.decode_rows,
-                ctx.slots, y, heads, groups, states, size, scratch=scratch)
+        shared = (dt, self.dt_bias, self.rate, self.skip, memory)
+        sizes = (heads, groups, states, size)
+        if not portions:
+            # single tokens alone: the recurrence's kernel does its head's convolution, and its ring, itself
+            ops.ssd_single(*shared, single, ctx.slots, y, *sizes,
+                           conv=(raw, self.conv, self.conv_bias, ring, ctx.positions, self.tensor_cores))
+        else:
+            xbc = ctx.buffer("ssd.xbc", (n, conv), torch.bfloat16 if self.tensor_cores else torch.float32)
+            ops.ring_conv(raw, None, self.conv, self.conv_bias, ring, ctx.positions, ctx.slots, xbc, act=1)
+            if taps > 1:
+                ops.ring_store(raw, None, ring, ctx.positions, ctx.slots)
+            chunks = ops.ssd_chunks(n - ctx.n_single, portions, self.tensor_cores)
+            scratch = ctx.runtime.scratch("ssd.chunks", ops.ssd_scratch_floats(chunks, heads, states, size), torch.float32)
+            ops.ssd(xbc, *shared, ctx.prefill_segments, portions, chunks, ctx.slots, y, *sizes, scratch)
+            if single.numel():
+                ops.ssd_single(*shared, single, ctx.slots, y, *sizes, xbc=xbc)
         o = ctx.buffer("ssd.o", (n, inner), rt.compute_dtype)
         ops.gated_group_norm(y, z, self.norm, ctx.slots, o, self.norm_groups, self.eps)
         linear(rt, STORE if store else ACCUM, o, self.w_o, residual, scale, error_flag=flag, name="ssd_o")

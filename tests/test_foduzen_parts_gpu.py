@@ -370,7 +370,7 @@ def _request(d, dv, window):
 RIGHT = [dict(heads=4, vdim=12, state=20, groups=2, norm_groups=4, conv=3), dict(heads=3, vdim=8, state=6, groups=1, norm_groups=1, conv=5),
          dict(heads=1, vdim=32, state=32, groups=1, norm_groups=2, conv=4), dict(heads=8, vdim=6, state=10, groups=8, norm_groups=3, conv=8),
          dict(heads=4, vdim=64, state=64, groups=2, norm_groups=1, conv=4), dict(heads=2, vdim=64, state=128, groups=1, norm_groups=2, conv=4),
-         dict(heads=6, vdim=32, state=16, groups=3, norm_groups=6, conv=1), dict(heads=2, vdim=128, state=48, groups=2, norm_groups=1, conv=2),
+         dict(heads=6, vdim=32, state=16, groups=3, norm_groups=2, conv=1), dict(heads=2, vdim=128, state=48, groups=2, norm_groups=1, conv=2),
          dict(heads=2, vdim=200, state=256, groups=1, norm_groups=1, conv=4), dict(heads=2, vdim=40, state=24, groups=1, norm_groups=1, conv=4)]
 
 
@@ -396,6 +396,51 @@ def test_state_space_recurrence(m, dtype):
     for cut in CUTS:
         got = run_mixer("state_space", params, w, h, dtype, cut(T))
         close(got, want, 3e-5 if dtype == "float32" else 3e-2, f"{cut(T)[:2]}")
+
+
+@pytest.mark.parametrize("heads,P,N,G", [(4, 64, 64, 2), (2, 16, 16, 1), (6, 32, 48, 3), (3, 128, 128, 1), (2, 48, 96, 2),
+                                          (1, 64, 256, 1), (2, 80, 16, 2), (8, 32, 112, 4)])
+def test_state_space_portions_on_the_tensor_cores(heads, P, N, G):
+    """bfloat16 x, B and C given, so that nothing but the kernels' own sums and powers differs from the plain recurrence: portions
+    of 2 to 300 tokens in one step, from states in slots, heads that forget at once beside heads that keep everything; the same
+    rows on the 32-bit pipes and, as single tokens, in place."""
+    from lia_rs_b200.kernels import ops
+    assert ops.ssd_tc_accepts(N, P)
+    g = torch.Generator().manual_seed(heads * P + N)
+    r = lambda *shape: torch.randn(*shape, generator=g)
+    plan = [(2, 0, 129), (0, 7, 2), (3, 4, 300), (1, 9, 128), (4, 0, 33)]
+    positions, slots, segments, n_segments, _, n = runs(plan)
+    inner = heads * P
+    xbc, wide = bf(r(n, inner + 2 * G * N)), r(n, heads + 3) * 2
+    dt_bias, A_log, D = -1.0 + r(heads), torch.linspace(-8, 3, heads), r(heads)
+    state = r(6, heads, N, P)
+    arguments = [dev(dt_bias), dev(torch.exp(A_log)), dev(D)]
+    results = []
+    for rows in (dev(xbc), dev(xbc.float())):
+        memory, y = dev(state.clone()), torch.zeros(n, inner, device=DEV)
+        chunks = ops.ssd_chunks(n, n_segments, rows.dtype == BF16)
+        scratch = torch.empty(ops.ssd_scratch_floats(chunks, heads, N, P), device=DEV)
+        ops.ssd(rows, dev(wide)[:, 3:], *arguments, memory, segments, n_segments, chunks, slots, y, heads, G, N, P, scratch)
+        results.append((y.cpu().to(F64), memory.cpu().to(F64)))
+    at = 0
+    for slot, start, count in plan:
+        part = xbc[at:at + count].to(F64)
+        want, last = pf.head_recurrence(part[:, :inner].reshape(count, heads, P), part[:, inner:inner + G * N].reshape(count, G, N),
+                                        part[:, inner + G * N:].reshape(count, G, N),
+                                        pf.softplus(wide[at:at + count, 3:].to(F64) + dt_bias.to(F64)), A_log, D, state[slot])
+        for (y, memory), tolerance in zip(results, (6e-5, 2e-5)):
+            assert float((y[at:at + count] - want.reshape(count, inner)).abs().max()) <= tolerance * max(1.0, float(want.abs().max()))
+            assert float((memory[slot] - last).abs().max()) <= tolerance * max(1.0, float(last.abs().max()))
+        if slot == 0:
+            for rows in (dev(xbc), dev(xbc.float())):
+                memory = dev(state.clone())
+                for t in range(at, at + count):
+                    y = torch.zeros(n, inner, device=DEV)
+                    ops.ssd_single(dev(wide)[:, 3:], *arguments, memory, ints([t]), slots, y, heads, G, N, P, xbc=rows)
+                    close(y[t], want[t - at].reshape(-1), 5e-6)
+                close(memory[slot], last, 5e-6)
+        at += count
+    assert torch.equal(results[0][1][5].float(), state[5])
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
