@@ -5,7 +5,7 @@
 // before a request's first token.
 //  * `rglru_gates`: the parts' products on the 32-bit pipes and what follows from them, a and the inflow
 //    sqrt(1 - a^2) i u (1 - a^2 taken as -expm1(2 log a): no cancellation where a is close to one), 32-bit.
-//  * `rglru_scan`: the recurrence along the step's runs (prompt portions and single tokens).  A CTA owns 32 channels of one
+//  * `rglru_scan`: the recurrence along the step's runs (single tokens: a thread a channel; prompt portions:).  A CTA owns 32 channels of one
 //    run; its warps take WARP_TOKENS consecutive tokens each, all at once: every warp walks its tokens from zero, the
 //    warps' end states and products of decays meet in shared memory, every warp takes its true start state from those
 //    before it and walks again, writing the outputs.  Two passes over registers, one over memory.  It also leaves the
@@ -74,14 +74,7 @@ rglru_scan_kernel(ScanArgs p) {
     __shared__ float ends[SCAN_WARPS][32], decays[SCAN_WARPS][32], carry[32];
     pdl_launch_dependents();
     pdl_wait();
-    int first, count;
-    if ((int)blockIdx.x < p.n_segments) {
-        first = p.segments[3 * blockIdx.x];
-        count = p.segments[3 * blockIdx.x + 2];
-    } else {
-        first = p.single_rows[blockIdx.x - p.n_segments];
-        count = 1;
-    }
+    const int first = p.segments[3 * blockIdx.x], count = p.segments[3 * blockIdx.x + 2];
     if (first < 0 || count <= 0) return;
     const int slot = p.slots[first];
     if (slot < 0) return;
@@ -139,6 +132,25 @@ rglru_scan_kernel(ScanArgs p) {
         }
     }
 }
+// single tokens: a thread a channel
+template <typename TO>
+__global__ void rglru_step_kernel(ScanArgs p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = p.single_rows[blockIdx.x];
+    if (t < 0) return;
+    const int slot = p.slots[t];
+    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (slot < 0 || c >= p.width) return;
+    float* state = p.state + (size_t)slot * p.slot_stride + c;
+    const float S = fmaf(p.a[(size_t)t * p.width + c], *state, p.inflow[(size_t)t * p.width + c]);
+    const float gate = p.y[(size_t)t * p.ld + c] + (p.y_bias ? p.y_bias[c] : 0.f);
+    *state = S;
+    reinterpret_cast<TO*>(p.out)[(size_t)t * p.width + c] = from_float<TO>(S * ring_gelu_tanh(gate));
+    if (p.taps > 1)
+        p.ring[(size_t)slot * p.slot_stride + (size_t)(p.positions[t] % p.taps) * p.width + c] =
+            p.x[(size_t)t * p.ld + c] + (p.x_bias ? p.x_bias[c] : 0.f);
+}
 }  // namespace
 
 // u [n, width] of u_dtype; weight [blocks, size, 2 size] of w_dtype: part b's [in][r's outputs | i's outputs]; bias
@@ -176,14 +188,19 @@ LIA_EXPORT int lia_rglru_scan(const float* a, const float* inflow, const float* 
                               const int* segments, int n_segments, const int* single_rows, int n_single,
                               const int* positions, const int* slots, void* out, int out_dtype, int width, int taps,
                               cudaStream_t stream) {
-    const int runs = n_segments + n_single;
-    if (runs <= 0) return LIA_OK;
+    if (n_segments + n_single <= 0) return LIA_OK;
     if (width <= 0 || taps < 1 || taps > RING_MAX_TAPS || ld < width || n_segments < 0 || n_single < 0 || (taps > 1 && !ring))
         return LIA_ERR_SIZE;
+    if (out_dtype != LIA_F32 && out_dtype != LIA_BF16) return LIA_ERR_DTYPE;
     ScanArgs p = {a, inflow, y, ld, y_bias, x, x_bias, ring, state, slot_stride, segments, n_segments, single_rows, n_single,
                   positions, slots, out, width, taps};
-    const dim3 grid(runs, (width + 31) / 32);
-    if (out_dtype == LIA_F32) return lia_launch(rglru_scan_kernel<float>, grid, dim3(SCAN_WARPS * 32), 0, stream, p);
-    if (out_dtype == LIA_BF16) return lia_launch(rglru_scan_kernel<__nv_bfloat16>, grid, dim3(SCAN_WARPS * 32), 0, stream, p);
-    return LIA_ERR_DTYPE;
+    if (n_segments > 0) {
+        const dim3 grid(n_segments, (width + 31) / 32);
+        const int rc = out_dtype == LIA_F32 ? lia_launch(rglru_scan_kernel<float>, grid, dim3(SCAN_WARPS * 32), 0, stream, p)
+                                            : lia_launch(rglru_scan_kernel<__nv_bfloat16>, grid, dim3(SCAN_WARPS * 32), 0, stream, p);
+        if (rc != LIA_OK || n_single <= 0) return rc;
+    }
+    const dim3 grid(n_single, (width + 127) / 128);
+    if (out_dtype == LIA_F32) return lia_launch(rglru_step_kernel<float>, grid, dim3(128), 0, stream, p);
+    return lia_launch(rglru_step_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p);
 }

@@ -280,7 +280,7 @@ ssd_output_kernel(SsdArgs p) {
 }
 
 // out[t, part] = rms(y * silu(z)) * weight over each of `groups` parts of `size` elements: a CTA a (token, part)
-template <typename TO>
+template <typename TO, int PER>                  // PER: quads a thread keeps in registers; 0: any size, the row read twice
 __global__ void gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, long long ld_z,
                                         const float* __restrict__ weight, const int* __restrict__ slots, TO* __restrict__ out,
                                         int groups, int size, float eps) {
@@ -291,16 +291,47 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, const float
     if (slots[t] < 0) return;
     const float* yr = y + (size_t)t * groups * size + (size_t)g * size;
     const float* zr = z + (size_t)t * ld_z + (size_t)g * size;
-    float sum = 0.f;
-    for (int i = threadIdx.x; i < size; i += blockDim.x) {
-        const float v = yr[i] * ring_silu(zr[i]);
-        sum = fmaf(v, v, sum);
-    }
-    sum = block_sum(sum, scratch);
-    const float inv = 1.0f / sqrtf(sum / (float)size + eps);
     TO* dst = out + (size_t)t * groups * size + (size_t)g * size;
     const float* w = weight + (size_t)g * size;
-    for (int i = threadIdx.x; i < size; i += blockDim.x) dst[i] = from_float<TO>(yr[i] * ring_silu(zr[i]) * inv * w[i]);
+    float sum = 0.f;
+    if constexpr (PER > 0) {
+        const int quads = size / 4;
+        float4 v[PER], gate[PER];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int q = threadIdx.x + i * blockDim.x;
+            v[i] = q < quads ? reinterpret_cast<const float4*>(yr)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+            gate[i] = q < quads ? reinterpret_cast<const float4*>(zr)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            v[i].x *= ring_silu(gate[i].x), v[i].y *= ring_silu(gate[i].y);
+            v[i].z *= ring_silu(gate[i].z), v[i].w *= ring_silu(gate[i].w);
+            sum = fmaf(v[i].x, v[i].x, sum), sum = fmaf(v[i].y, v[i].y, sum);
+            sum = fmaf(v[i].z, v[i].z, sum), sum = fmaf(v[i].w, v[i].w, sum);
+        }
+        const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)size + eps);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int q = threadIdx.x + i * blockDim.x;
+            if (q >= quads) break;
+            const float4 f = reinterpret_cast<const float4*>(w)[q];
+            const float r[4] = {v[i].x * inv * f.x, v[i].y * inv * f.y, v[i].z * inv * f.z, v[i].w * inv * f.w};
+            if constexpr (sizeof(TO) == 4) {
+                *reinterpret_cast<float4*>(dst + 4 * q) = make_float4(r[0], r[1], r[2], r[3]);
+            } else {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+                *reinterpret_cast<uint2*>(dst + 4 * q) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < size; i += blockDim.x) {
+            const float v = yr[i] * ring_silu(zr[i]);
+            sum = fmaf(v, v, sum);
+        }
+        const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)size + eps);
+        for (int i = threadIdx.x; i < size; i += blockDim.x) dst[i] = from_float<TO>(yr[i] * ring_silu(zr[i]) * inv * w[i]);
+    }
 }
 
 // the last inputs of every run's convolution into the slot's ring: a CTA a row, rows further than `taps` from their run's end skip
@@ -405,12 +436,27 @@ LIA_EXPORT int lia_gated_group_norm(const float* y, const float* z, long long ld
                                     cudaStream_t stream) {
     if (n_tokens <= 0) return LIA_OK;
     if (groups <= 0 || groups > 65535 || size <= 0 || ld_z < (long long)groups * size) return LIA_ERR_SIZE;
-    const int threads = size >= 1024 ? 256 : 128;
-    if (out_dtype == LIA_F32)
-        return lia_launch(gated_group_norm_kernel<float>, dim3(n_tokens, groups), dim3(threads), 0, stream, y, z, ld_z, weight,
-                          slots, (float*)out, groups, size, eps);
-    if (out_dtype == LIA_BF16)
-        return lia_launch(gated_group_norm_kernel<__nv_bfloat16>, dim3(n_tokens, groups), dim3(threads), 0, stream, y, z, ld_z,
-                          weight, slots, (__nv_bfloat16*)out, groups, size, eps);
+    const uintptr_t bits = (uintptr_t)y | (uintptr_t)z | (uintptr_t)weight | (uintptr_t)out;
+    int per = 0, threads = size >= 1024 ? 256 : 128;
+    if (size % 4 == 0 && ld_z % 4 == 0 && (bits & 15u) == 0 && size <= 8192) {
+        const int quads = size / 4;
+        threads = quads <= 32 ? 32 : quads <= 64 ? 64 : quads <= 128 ? 128 : quads <= 256 ? 256 : 512;
+        per = (quads + threads - 1) / threads;
+        per = per > 2 ? 4 : per;
+    }
+#define LIA_GATED(TO, PER)                                                                                                    \
+    return lia_launch(gated_group_norm_kernel<TO, PER>, dim3(n_tokens, groups), dim3(threads), 0, stream, y, z, ld_z, weight, \
+                      slots, (TO*)out, groups, size, eps)
+#define LIA_GATED_PER(TO)                    \
+    {                                        \
+        if (per == 1) LIA_GATED(TO, 1);      \
+        if (per == 2) LIA_GATED(TO, 2);      \
+        if (per == 4) LIA_GATED(TO, 4);      \
+        LIA_GATED(TO, 0);                    \
+    }
+    if (out_dtype == LIA_F32) LIA_GATED_PER(float)
+    if (out_dtype == LIA_BF16) LIA_GATED_PER(__nv_bfloat16)
+#undef LIA_GATED_PER
+#undef LIA_GATED
     return LIA_ERR_DTYPE;
 }

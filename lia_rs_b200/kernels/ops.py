@@ -158,6 +158,10 @@ class _Signatures:
     lia_rglru_gates_tc_accepts = [c_int, c_int]
     lia_rglru_gates_tc = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                           c_void_p, c_void_p]
+    lia_rglru_single_accepts = [c_int, c_int]
+    lia_rglru_single = [c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                        c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                        c_void_p]
     lia_rglru_scan = [c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                       ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                       c_void_p]
@@ -1570,6 +1574,32 @@ def rglru_scan(a, inflow, y, x, y_bias, x_bias, ring, state, segments, n_segment
                                     _p(ring) if taps > 1 else None, _p(state), stride, _p(segments), int(n_segments),
                                     _p(single_rows), n_single, _p(positions), _p(slots), _p(out), dtype_code(out.dtype), width,
                                     int(taps), _stream()), "rglru_scan")
+
+
+def rglru_single_accepts(width: int, blocks: int) -> bool:
+    """Whether `rglru_single` takes parts of this size (bfloat16)."""
+    return bool(lib().lia_rglru_single_accepts(int(width), int(blocks)))
+
+
+def rglru_single(y, x, y_bias, x_bias, conv, conv_bias, w_r, w_i, bias, rate, ring, state, positions, slots, out, blocks: int):
+    """Everything between the unit's two products in a step whose rows are single tokens: convolution, gates, recurrence and the
+    gate branch, with state [slots, width] and ring [slots, taps, width] brought up to date (bfloat16 weights and output); see
+    csrc/rglru_single.cu."""
+    _cuda(y_bias, x_bias, conv, conv_bias, w_r, w_i, bias, rate, positions, slots, out)
+    _f32(y, x, y_bias, x_bias, conv, conv_bias, bias, rate)
+    n, width = out.shape
+    taps, size = conv.shape[0], width // blocks
+    if y.stride(1) != 1 or x.stride(1) != 1 or y.stride(0) != x.stride(0) or y.shape != (n, width) or x.shape != (n, width) or \
+            tuple(w_r.shape) != (blocks, size, size) or tuple(w_i.shape) != (blocks, size, size) or conv.shape[1] != width or \
+            not (w_r.dtype == w_i.dtype == out.dtype == torch.bfloat16):
+        raise KernelError("rglru_single: shapes or element types do not agree")
+    stride = _slots_of(state, (width,), "rglru_single")
+    if taps > 1 and _slots_of(ring, (taps, width), "rglru_single") != stride and state.shape[0] > 1:
+        raise KernelError("rglru_single: ring and state must have one slot stride")
+    with _timed("rglru_single", nbytes=2 * w_r.numel() * 2 + n * width * (10 + 4 * (taps + 3))):
+        _check(lib().lia_rglru_single(_p(y), _p(x), y.stride(0), _p(y_bias), _p(x_bias), _p(conv), _p(conv_bias), _p(w_r), _p(w_i),
+                                      _p(bias), _p(rate), _p(ring) if taps > 1 else None, _p(state), stride, _p(positions),
+                                      _p(slots), _p(out), n, width, int(blocks), taps, _stream()), "rglru_single")
 
 
 def ssd_scratch_floats(chunks: int, heads: int, states: int, size: int) -> int:

@@ -9,7 +9,8 @@
 What a request carries from token to token is one 32-bit state per slot: the convolution's last inputs in a ring of `taps`
 rows (csrc/conv_ring.cuh) and S.  The two branches are one product with 32-bit rows.  The convolution's sums and GELU are
 32-bit; u is rounded once to the compute element type, and everything behind it (the gates with their products, decays, the
-inflow, the state) is 32-bit.  A step's portions are walked by many warps at once (csrc/rglru.cu), continuing from the slot's
+inflow, the state) is 32-bit.  In bfloat16 a step of single tokens is one kernel between the two products
+(csrc/rglru_single.cu) and the gates of other steps are a tcgen05 kernel (csrc/rglru_gates_tc.cu).  A step's portions are walked by many warps at once (csrc/rglru.cu), continuing from the slot's
 state, so a portion cut anywhere gives what token-by-token steps give, up to the order of the operations.
 
 Parameters: hidden, width, blocks, taps, and optionally `names`."""
@@ -86,6 +87,7 @@ class RGLRU(Mixer):
         # bfloat16: the tensor-core kernel's matrices as they are stored; else part b's two side by side, transposed
         # ([in][r's outputs | i's outputs])
         self.tensor_cores = runtime.compute_dtype == torch.bfloat16 and ops.rglru_gates_tc_accepts(self.width, self.blocks)
+        self.one_kernel = self.tensor_cores and ops.rglru_single_accepts(self.width, self.blocks)
         if self.tensor_cores:
             self.w_r, self.w_i = prepare_weight(tensors[n["r"]], runtime), prepare_weight(tensors[n["i"]], runtime)
         else:
@@ -103,6 +105,12 @@ class RGLRU(Mixer):
         rows = ctx.buffer("rglru.in", (n, 2 * self.branch), torch.float32)
         linear(rt, STORE, x, self.w_in, rows, error_flag=flag, name="yx")
         y, v = rows[:, :width], rows[:, self.branch:self.branch + width]
+        out = ctx.buffer("rglru.out", (n, width), rt.compute_dtype)
+        if self.one_kernel and ctx.decode_only:
+            ops.rglru_single(y, v, self.y_bias, self.x_bias, self.conv, self.conv_bias, self.w_r, self.w_i, self.gate_bias, self.rate,
+                             ring, memory, ctx.positions, ctx.slots, out, self.blocks)
+            linear(rt, STORE if store else ACCUM, out, self.w_o, residual, scale, error_flag=flag, name="o")
+            return
         u = ctx.buffer("rglru.u", (n, width), rt.compute_dtype)
         ops.ring_conv(v, self.x_bias, self.conv, self.conv_bias, ring, ctx.positions, ctx.slots, u)
         a = ctx.buffer("rglru.a", (n, width), torch.float32)
@@ -111,7 +119,6 @@ class RGLRU(Mixer):
             ops.rglru_gates_tc(u, self.w_r, self.w_i, self.gate_bias, self.rate, ctx.slots, a, inflow, self.blocks, error_flag=flag)
         else:
             ops.rglru_gates(u, self.w_gates, self.gate_bias, self.rate, ctx.slots, a, inflow, self.blocks)
-        out = ctx.buffer("rglru.out", (n, width), rt.compute_dtype)
         ops.rglru_scan(a, inflow, y, v, self.y_bias, self.x_bias, ring, memory, ctx.prefill_segments, ctx.n_prefill_segments,
                        ctx.decode_rows, ctx.positions, ctx.slots, out, taps)
         linear(rt, STORE if store else ACCUM, out, self.w_o, residual, scale, error_flag=flag, name="o")
