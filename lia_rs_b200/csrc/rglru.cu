@@ -87,17 +87,23 @@ rglru_scan_kernel(ScanArgs p) {
     if (warp == 0) carry[lane] = live ? *state : 0.f;
     __syncthreads();
     TO* out = reinterpret_cast<TO*>(p.out);
-    for (int base = 0; base < count; base += SCAN_SPAN) {
-        const int r0 = base + warp * WARP_TOKENS;
-        float a[WARP_TOKENS], b[WARP_TOKENS], g[WARP_TOKENS];
+    float a[WARP_TOKENS], b[WARP_TOKENS], g[WARP_TOKENS], na[WARP_TOKENS], nb[WARP_TOKENS], ng[WARP_TOKENS];
+    auto fetch = [&](int r0) {
 #pragma unroll
         for (int k = 0; k < WARP_TOKENS; ++k) {
             const bool there = r0 + k < count;
             const size_t t = (size_t)first + (there ? r0 + k : 0);
-            a[k] = there ? p.a[t * p.width + cc] : 1.f;
-            b[k] = there ? p.inflow[t * p.width + cc] : 0.f;
-            g[k] = there ? p.y[t * p.ld + cc] : 0.f;
+            na[k] = there ? p.a[t * p.width + cc] : 1.f;
+            nb[k] = there ? p.inflow[t * p.width + cc] : 0.f;
+            ng[k] = there ? p.y[t * p.ld + cc] : 0.f;
         }
+    };
+    fetch(warp * WARP_TOKENS);
+    for (int base = 0; base < count; base += SCAN_SPAN) {
+        const int r0 = base + warp * WARP_TOKENS;
+#pragma unroll
+        for (int k = 0; k < WARP_TOKENS; ++k) a[k] = na[k], b[k] = nb[k], g[k] = ng[k];
+        if (base + SCAN_SPAN < count) fetch(r0 + SCAN_SPAN);      // the next span's rows travel while this one is walked
         float end = 0.f, decay = 1.f;
 #pragma unroll
         for (int k = 0; k < WARP_TOKENS; ++k) {

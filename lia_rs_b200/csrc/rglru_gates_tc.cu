@@ -31,6 +31,21 @@ struct GatesArgs {
 };
 
 __device__ __forceinline__ float fast_sigmoid(float v) { return __fdividef(1.0f, 1.0f + __expf(-v)); }
+// 1 - e^x for x <= 0: near zero the exponential's series to x^7 (what is left out is below 2^-28 of the sum), else as it stands
+__device__ __forceinline__ float one_minus_exp(float x) {
+    float s = fmaf(x, 1.0f / 7.0f, 1.0f);
+    s = fmaf(x * s, 1.0f / 6.0f, 1.0f);
+    s = fmaf(x * s, 0.2f, 1.0f);
+    s = fmaf(x * s, 0.25f, 1.0f);
+    s = fmaf(x * s, 1.0f / 3.0f, 1.0f);
+    s = fmaf(x * s, 0.5f, 1.0f);
+    return x > -0.25f ? -x * s : 1.0f - __expf(x);
+}
+__device__ __forceinline__ float fast_sqrt(float v) {
+    float y;
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v));
+    return y;
+}
 
 __global__ void __launch_bounds__(GATES_THREADS, 2)
 rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_constant__ CUtensorMap map_i,
@@ -134,16 +149,24 @@ rglru_gates_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
                 tmem_load16(at + (uint32_t)c0, r);
                 tmem_load16(at + (uint32_t)(p.n_tile + c0), i);
                 if (!live) continue;
+                const int there = min(16, p.n_tokens - (t0 + c0));
+                const size_t first = (size_t)(t0 + c0) * p.width + c;
+                float u[16];
+#pragma unroll
+                for (int k = 0; k < 16; ++k) u[k] = k < there ? to_float(p.u[first + (size_t)k * p.width]) : 0.f;
 #pragma unroll
                 for (int k = 0; k < 16; ++k) {
-                    const int t = t0 + c0 + k;
-                    if (t >= p.n_tokens) break;
-                    const float uv = to_float(p.u[(size_t)t * p.width + c]);
-                    const float w = -expm1f(-rate * fast_sigmoid(r[k] + br));
+                    const float w = one_minus_exp(-rate * fast_sigmoid(r[k] + br));
                     const float a = 1.0f - w;
-                    p.a_out[(size_t)t * p.width + c] = a;
-                    p.inflow[(size_t)t * p.width + c] = sqrtf(w * (1.0f + a)) * fast_sigmoid(i[k] + bi) * uv;
+                    r[k] = a;
+                    i[k] = fast_sqrt(w * (1.0f + a)) * fast_sigmoid(i[k] + bi) * u[k];
                 }
+#pragma unroll
+                for (int k = 0; k < 16; ++k)
+                    if (k < there) {
+                        p.a_out[first + (size_t)k * p.width] = r[k];
+                        p.inflow[first + (size_t)k * p.width] = i[k];
+                    }
             }
             tc_fence_before();
         } else if (lane == 0 && p.error_flag) {

@@ -30,7 +30,8 @@ __global__ void __launch_bounds__(STEP_THREADS)
 rglru_single_kernel(StepArgs p) {
     extern __shared__ __align__(16) uint8_t step_raw[];      // weights [2 SLICE][size + 8], u [STEP_TOKENS][size + 8]
     __shared__ float sums[2 * SLICE][STEP_TOKENS + 1];
-    __shared__ int token_slot[STEP_TOKENS], token_pos[STEP_TOKENS];
+    __shared__ int token_slot[STEP_TOKENS];
+    __shared__ int ring_row[STEP_TOKENS][RING_MAX_TAPS];       // [j]: the ring's row of tap j's input, -1 before the start; [taps - 1]: the token's own row
     const int size = p.size, pitch = size + 8;
     __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(step_raw);
     __nv_bfloat16* us = ws + 2 * SLICE * pitch;
@@ -47,8 +48,12 @@ rglru_single_kernel(StepArgs p) {
     asm volatile("cp.async.commit_group;" ::: "memory");
     if (tid < STEP_TOKENS) {                                 // (the step's metadata depends on no kernel of the step)
         const bool there = t0 + tid < p.n_tokens;
+        const int pos = there ? p.positions[t0 + tid] : 0;
         token_slot[tid] = there ? p.slots[t0 + tid] : -1;
-        token_pos[tid] = there ? p.positions[t0 + tid] : 0;
+        for (int j = 0; j < p.taps; ++j) {
+            const int at = pos - (p.taps - 1 - j);
+            ring_row[tid][j] = at >= 0 ? at % p.taps : -1;
+        }
     }
     pdl_launch_dependents();
     pdl_wait();
@@ -72,26 +77,28 @@ rglru_single_kernel(StepArgs p) {
             for (int k = tid % across; k < size; k += across) {
                 const int c = part * size + k;
                 const float xb = p.x_bias[c], cb = p.conv_bias[c];
-                float w[RING_MAX_TAPS];
+                float w[RING_MAX_TAPS - 1];
 #pragma unroll
-                for (int j = 0; j < RING_MAX_TAPS; ++j) w[j] = j < p.taps ? p.conv[(size_t)j * p.width + c] : 0.f;
+                for (int j = 0; j < RING_MAX_TAPS - 1; ++j) w[j] = j < p.taps - 1 ? p.conv[(size_t)j * p.width + c] : 0.f;
+                const float w_own = p.conv[(size_t)(p.taps - 1) * p.width + c];
 #pragma unroll 4
                 for (int tok = row; tok < STEP_TOKENS; tok += down) {
-                    const int slot = token_slot[tok], pos = token_pos[tok];
+                    const int slot = token_slot[tok];
                     float v = 0.f;
                     if (slot >= 0) {
                         float* ring = p.ring + (size_t)slot * p.slot_stride + c;
                         const float own = p.x[(size_t)(t0 + tok) * p.ld + c] + xb;
-                        v = cb;
+                        float earlier[RING_MAX_TAPS - 1];
 #pragma unroll
                         for (int j = 0; j < RING_MAX_TAPS - 1; ++j) {
-                            const int back = p.taps - 1 - j;
-                            if (j < p.taps - 1 && pos - back >= 0) v = fmaf(w[j], ring[(size_t)((pos - back) % p.taps) * p.width], v);
+                            const int row = j < p.taps - 1 ? ring_row[tok][j] : -1;
+                            earlier[j] = row >= 0 ? ring[(size_t)row * p.width] : 0.f;
                         }
+                        v = cb;
 #pragma unroll
-                        for (int j = 0; j < RING_MAX_TAPS; ++j)
-                            if (j == p.taps - 1) v = fmaf(w[j], own, v);
-                        if (p.taps > 1 && k >= o0 && k < o0 + SLICE) ring[(size_t)(pos % p.taps) * p.width] = own;
+                        for (int j = 0; j < RING_MAX_TAPS - 1; ++j) v = fmaf(j < p.taps - 1 ? w[j] : 0.f, earlier[j], v);
+                        v = fmaf(w_own, own, v);
+                        if (p.taps > 1 && k >= o0 && k < o0 + SLICE) ring[(size_t)ring_row[tok][p.taps - 1] * p.width] = own;
                     }
                     us[tok * pitch + k] = __float2bfloat16_rn(v);
                 }

@@ -178,6 +178,10 @@ class Mixer(Part):
     # True: the mixer's result is a sum that it leaves to the arrangement: `output_terms` stands in for `forward` (an
     # arrangement that norms the mixer's output takes both; the others refuse such a mixer).
     gives_terms = False
+    # True: everything the mixer reads of its input is one product x w_in^T (`w_in` [width, hidden], a multiple of 8 rows), and
+    # `forward` takes that product's 32-bit rows as `projected` (any row stride) in place of making them: mixers that read the
+    # same input can then share one product.
+    projects_input = False
 
     @staticmethod
     def cache_request(params: dict) -> Optional[KVCacheRequest]:

@@ -6,7 +6,8 @@ Each member is a registered mixer with its own parameters and checkpoint prefix.
 into the residual stream itself (a mixer's `forward` does `residual += scale * f(x)`, so the weights ride on the members'
 last products and no sum is formed anywhere else).  With norms every member stores into rows of its own, and the sum is
 left to the arrangement as terms (`Mixer.output_terms`), which norms, adds and joins the stream in one kernel; an output
-bias of such a member is added there too.  At most one member may ask for a paged cache and at most one for per-request
+bias of such a member is added there too.  Members that read their input through one product each (`projects_input`) then
+share one product.  At most one member may ask for a paged cache and at most one for per-request
 state: the layer's cache and state are handed to those.
 
 Parameters: `members`: a list of {"kind", "params", "prefix", "scale", "norm": {"tensor", "hidden", "eps"} (absent: none; the
@@ -18,6 +19,7 @@ import torch
 from ..kernels import ops
 from ..weights import TensorSpec
 from .base import MIXERS, Mixer, lookup, register_mixer
+from .linear import STORE, linear
 
 
 @register_mixer("side_by_side")
@@ -76,6 +78,16 @@ class SideBySide(Mixer):
         self.norms = [(tensors[prefix + m["norm"]["tensor"]].to(torch.float32).contiguous(), float(m["norm"]["eps"]))
                       for m in params["members"] if m.get("norm")]
         self.gives_terms = bool(self.norms)
+        # members whose input products can be one product over the same rows
+        self.runtime, self.w_in, self.columns = runtime, None, []
+        if self.gives_terms and all(part.projects_input for part, _, _, _ in self.members):
+            at = 0
+            for part, _, _, _ in self.members:
+                self.columns.append((at, at + part.w_in.shape[0]))
+                at += part.w_in.shape[0]
+            self.w_in = torch.cat([part.w_in for part, _, _, _ in self.members], dim=0)
+            for part, _, _, _ in self.members:
+                part.w_in = None
         self.graph_safe = all(part.graph_safe for part, _, _, _ in self.members)
         self.takes_deferred_norm = all(part.takes_deferred_norm for part, _, _, _ in self.members)
 
@@ -86,10 +98,15 @@ class SideBySide(Mixer):
         return key
 
     def output_terms(self, ctx, x, kv=None, state=None):
-        n, terms = x.shape[0], []
+        n, terms, projected = x.shape[0], [], [{} for _ in self.members]
+        if self.w_in is not None:
+            shared = ctx.buffer("side_by_side.in", (n, self.w_in.shape[0]), torch.float32)
+            linear(self.runtime, STORE, x, self.w_in, shared, error_flag=ctx.error_flag, name="mixers_in")
+            projected = [{"projected": shared[:, begin:end]} for begin, end in self.columns]
         for i, ((part, weight, wants_cache, wants_state), (norm, eps)) in enumerate(zip(self.members, self.norms)):
             rows = ctx.buffer(f"side_by_side.{i}", (n, norm.numel()), torch.float32)
-            part.forward(ctx, x, rows, 1.0, kv=kv if wants_cache else None, state=state if wants_state else None, store=True)
+            part.forward(ctx, x, rows, 1.0, kv=kv if wants_cache else None, state=state if wants_state else None, store=True,
+                         **projected[i])
             terms.append(ops.NormTerm(rows, bias=part.output_bias, weight=norm, scale=weight, eps=eps))
         return terms
 

@@ -73,6 +73,7 @@ class SinkAttention(Mixer):
     graph_safe = True
     takes_deferred_norm = True
     can_store = True
+    projects_input = True
     NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "o_bias": "o.b",
              "q_norm": "q.norm", "k_norm": "k.norm", "mix": "vmix", "gate": "g"}
 
@@ -175,12 +176,13 @@ class SinkAttention(Mixer):
     def graph_key(self, ctx) -> tuple:
         return self.paged.graph_key(ctx) if self.paged is not None else ()
 
-    def forward(self, ctx, x, residual, scale, kv=None, state=None, store=False):
+    def forward(self, ctx, x, residual, scale, kv=None, state=None, store=False, projected=None):
         rt, n = self.runtime, x.shape[0]
         nq, nkv, d, dv = self.nq, self.nkv, self.d, self.dv
         flag = ctx.error_flag
-        projected = ctx.buffer("sinkattn.in", (n, self.width), torch.float32)
-        linear(rt, STORE, x, self.w_in, projected, error_flag=flag, name="qkv")
+        if projected is None:
+            projected = ctx.buffer("sinkattn.in", (n, self.width), torch.float32)
+            linear(rt, STORE, x, self.w_in, projected, error_flag=flag, name="qkv")
         q = ctx.buffer("sinkattn.q", (n, nq * d), rt.compute_dtype)
         v_first = ctx.buffer("sinkattn.v_first", (n, nkv * dv), torch.float32) if self.mix_mode else None
         ops.qkv_prepare(projected, self.bias_in, self.q_norm, self.k_norm, self.eps, self.freq, self.rot_dims,

@@ -30,6 +30,7 @@ class StateSpace(Mixer):
     graph_safe = True
     takes_deferred_norm = True
     can_store = True
+    projects_input = True
     NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm",
              "o": "o"}
 
@@ -98,15 +99,17 @@ class StateSpace(Mixer):
         self.tensor_cores = runtime.compute_dtype == torch.bfloat16 and ops.ssd_tc_accepts(self.states, self.size)
         self.rate = torch.exp(tensors[n["A_log"]].to(torch.float32)).contiguous()
 
-    def forward(self, ctx, x, residual, scale, kv=None, state=None, store=False):
+    def forward(self, ctx, x, residual, scale, kv=None, state=None, store=False, projected=None):
         rt, n = self.runtime, x.shape[0]
         heads, size, states, groups, inner, taps = self.heads, self.size, self.states, self.groups, self.inner, self.taps
         flag, conv = ctx.error_flag, self.conv_width
         slots, split = state.shape[0], self._ring(self.params)
         ring = state[:, :taps * conv].view(slots, taps, conv) if taps > 1 else None
         memory = state[:, split:split + heads * states * size].view(slots, heads, states, size)
-        rows = ctx.buffer("ssd.in", (n, self.width), torch.float32)
-        linear(rt, STORE, x, self.w_in, rows, error_flag=flag, name="ssd_in")
+        rows = projected
+        if rows is None:
+            rows = ctx.buffer("ssd.in", (n, self.width), torch.float32)
+            linear(rt, STORE, x, self.w_in, rows, error_flag=flag, name="ssd_in")
         z, raw, dt = rows[:, :inner], rows[:, inner:inner + conv], rows[:, inner + conv:inner + conv + heads]
         portions, single = ctx.n_prefill_segments, ctx.decode_rows
         y = ctx.buffer("ssd.y", (n, inner), torch.float32)

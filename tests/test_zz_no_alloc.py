@@ -4,6 +4,7 @@ The entry point serves hosts that must not call cudaMalloc when they need a prod
 pool, a plug-in whose host owns device memory): its split-K scratch is a static array inside the
 library.  This file is collected last on purpose: if it fails, a run that stops at the first failure has
 already run every other test.  It must pass alone in a fresh process and after the other tests."""
+import gc
 import math
 from ctypes import c_float, c_int, c_longlong, c_void_p
 
@@ -69,6 +70,7 @@ def test_no_alloc_product_equals_the_ordinary_one_on_two_calls_in_a_row():
         base = torch.randn(M, N, device=DEV)
         want, got = base.clone(), base.clone()
         ops.gemm_tc(mode, a, w, want, 0.5, flag)
+        gc.collect()                          # what earlier tests left to the collector goes now, not between the two readings
         held, free = torch.cuda.memory_allocated(DEV), free_bytes()
         assert call(fn, mode, a, w, got, 0.5, flag, sms) == 0
         assert free_bytes() == free and torch.cuda.memory_allocated(DEV) == held      # neither the driver nor torch gave memory out
@@ -91,7 +93,7 @@ def test_no_alloc_refuses_what_its_array_cannot_hold():
     from lia_rs_b200.kernels import ops
     fn, need = entry_points()
     sms = torch.cuda.get_device_properties(DEV).multi_processor_count
-    M, N, K = 128, 12288, 2048                                     # two ranges or more x 128 x 12288 floats > 8 MiB
+    M, N, K = 128, 9216, 2048                                      # two ranges or more x 128 x 9216 floats > 8 MiB
     assert need(ops.GEMM_STORE, M, N, K, sms) > SCRATCH_FLOATS
     a = torch.randn(M, K, device=DEV).to(torch.bfloat16)
     w = torch.randn(N, K, device=DEV).to(torch.bfloat16)
