@@ -235,6 +235,37 @@ __global__ void gate_rows_kernel(T* __restrict__ o, long long ld_o, const float*
     }
 }
 
+// the same for span 1, four elements a thread: width and strides multiples of 4 from 16-byte (o: four elements') aligned bases
+template <typename T, int ACT>
+__global__ void gate_rows4_kernel(T* __restrict__ o, long long ld_o, const float* __restrict__ g, long long ld_g, int quads) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int q = blockIdx.y * blockDim.x + threadIdx.x;
+    if (q >= quads) return;
+    const float4 z = *reinterpret_cast<const float4*>(g + blockIdx.x * ld_g + 4 * q);
+    T* dst = o + blockIdx.x * ld_o + 4 * q;
+    float v[4], f[4] = {z.x, z.y, z.z, z.w};
+    if constexpr (sizeof(T) == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(dst);
+        v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+    } else {
+        const uint2 x = *reinterpret_cast<const uint2*>(dst);
+        const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&x.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+        v[0] = __low2float(lo), v[1] = __high2float(lo), v[2] = __low2float(hi), v[3] = __high2float(hi);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float s = 1.0f / (1.0f + expf(-f[i]));
+        v[i] *= ACT == 2 ? f[i] * s : s;
+    }
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+
 int grid_for(long long total) {
     const long long blocks = (total + 255) / 256;
     return (int)(blocks < 8192 ? blocks : 8192);
@@ -305,6 +336,22 @@ LIA_EXPORT int lia_gate_rows(void* o, int dtype, long long ld_o, const float* g,
                              int act, int span, cudaStream_t stream) {
     if (rows <= 0 || width <= 0) return LIA_OK;
     if (span <= 0 || ld_o < width || ld_g < (width + span - 1) / span || act < 1 || act > 2) return LIA_ERR_SIZE;
+    if (span == 1 && width % 4 == 0 && ld_o % 4 == 0 && ld_g % 4 == 0 && ((uintptr_t)g & 15u) == 0 &&
+        ((uintptr_t)o & (dtype == LIA_F32 ? 15u : 7u)) == 0) {
+        const int quads = width / 4, threads = quads >= 256 ? 256 : 128;
+        const dim3 grid(rows, (quads + threads - 1) / threads);
+#define LIA_GATE4(T, ACT) return lia_launch(gate_rows4_kernel<T, ACT>, grid, dim3(threads), 0, stream, (T*)o, ld_o, g, ld_g, quads)
+        if (dtype == LIA_F32) {
+            if (act == 1) LIA_GATE4(float, 1);
+            LIA_GATE4(float, 2);
+        }
+        if (dtype == LIA_BF16) {
+            if (act == 1) LIA_GATE4(__nv_bfloat16, 1);
+            LIA_GATE4(__nv_bfloat16, 2);
+        }
+#undef LIA_GATE4
+        return LIA_ERR_DTYPE;
+    }
     const int blocks = grid_for((long long)rows * width);
 #define LIA_GATE(T, ACT)                                                                                             \
     return lia_launch(gate_rows_kernel<T, ACT>, dim3(blocks), dim3(256), 0, stream, (T*)o, ld_o, g, ld_g, rows, width, span)

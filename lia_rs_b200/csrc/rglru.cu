@@ -5,11 +5,12 @@
 // before a request's first token.
 //  * `rglru_gates`: the parts' products on the 32-bit pipes and what follows from them, a and the inflow
 //    sqrt(1 - a^2) i u (1 - a^2 taken as -expm1(2 log a): no cancellation where a is close to one), 32-bit.
-//  * `rglru_scan`: the recurrence along the step's runs (single tokens: a thread a channel; prompt portions:).  A CTA owns 32 channels of one
-//    run; its warps take WARP_TOKENS consecutive tokens each, all at once: every warp walks its tokens from zero, the
-//    warps' end states and products of decays meet in shared memory, every warp takes its true start state from those
-//    before it and walks again, writing the outputs.  Two passes over registers, one over memory.  It also leaves the
-//    convolution's last inputs in the slot's ring.
+//  * `rglru_scan`: the recurrence along the step's runs.  Single tokens: a thread a channel.  Prompt portions: a CTA owns a few
+//    channels of one portion; groups of threads take TOKENS_AHEAD consecutive tokens each, all at once: every group walks its
+//    tokens from zero, the groups' end states and products of decays meet by shuffles and in shared memory, every group takes
+//    its true start state from those before it and walks again, writing the outputs, while the rows of the next span of
+//    tokens are on their way.  Two passes over registers, one over memory.  It also leaves the convolution's last inputs in
+//    the slot's ring.
 // A row whose slot is negative belongs to nobody and is skipped.
 #include "conv_ring.cuh"
 
@@ -57,7 +58,8 @@ rglru_gates_kernel(const TU* __restrict__ u, const TW* __restrict__ weight, cons
     }
 }
 
-constexpr int SCAN_WARPS = 16, WARP_TOKENS = 16, SCAN_SPAN = SCAN_WARPS * WARP_TOKENS;
+// LANES channels side by side, SCAN_THREADS / LANES groups of TOKENS_AHEAD tokens at once
+constexpr int SCAN_THREADS = 256, SCAN_WARPS = SCAN_THREADS / 32, TOKENS_AHEAD = 8;
 
 struct ScanArgs {
     const float* a; const float* inflow;                  // [n, width]
@@ -69,75 +71,106 @@ struct ScanArgs {
 };
 
 template <typename TO>
-__global__ void __launch_bounds__(SCAN_WARPS * 32)
+__device__ __forceinline__ float gate_of(float z) {
+    if (sizeof(TO) == 4) return ring_gelu_tanh(z);
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);       // (rounded to 16 bits with S: the hardware's exponential)
+    return __fdividef(z, 1.0f + __expf(fminf(-2.0f * u, 80.f)));
+}
+
+template <typename TO, int LANES>
+__global__ void __launch_bounds__(SCAN_THREADS)
 rglru_scan_kernel(ScanArgs p) {
-    __shared__ float ends[SCAN_WARPS][32], decays[SCAN_WARPS][32], carry[32];
+    constexpr int SPAN = SCAN_THREADS / LANES * TOKENS_AHEAD;
+    __shared__ float2 ends[SCAN_WARPS][LANES];              // per warp: (product of the decays, end state from zero)
+    __shared__ float carry[LANES];
     pdl_launch_dependents();
     pdl_wait();
     const int first = p.segments[3 * blockIdx.x], count = p.segments[3 * blockIdx.x + 2];
     if (first < 0 || count <= 0) return;
     const int slot = p.slots[first];
     if (slot < 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.y * 32 + lane;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & (LANES - 1), group = threadIdx.x / LANES;
+    const int c = blockIdx.y * LANES + lane;
     const bool live = c < p.width;
     const int cc = live ? c : 0;
     float* state = p.state + (size_t)slot * p.slot_stride + cc;
     const float y_bias = p.y_bias ? p.y_bias[cc] : 0.f;
-    if (warp == 0) carry[lane] = live ? *state : 0.f;
+    if (group == 0) carry[lane] = live ? *state : 0.f;
     __syncthreads();
-    TO* out = reinterpret_cast<TO*>(p.out);
-    float a[WARP_TOKENS], b[WARP_TOKENS], g[WARP_TOKENS], na[WARP_TOKENS], nb[WARP_TOKENS], ng[WARP_TOKENS];
+    const size_t step_w = p.width, step_y = p.ld;
+    const float* a_at = p.a + (size_t)first * step_w + cc;
+    const float* b_at = p.inflow + (size_t)first * step_w + cc;
+    const float* g_at = p.y + (size_t)first * step_y + cc;
+    TO* out = reinterpret_cast<TO*>(p.out) + (size_t)first * step_w + cc;
+    float a[TOKENS_AHEAD], b[TOKENS_AHEAD], g[TOKENS_AHEAD], na[TOKENS_AHEAD], nb[TOKENS_AHEAD], ng[TOKENS_AHEAD];
     auto fetch = [&](int r0) {
 #pragma unroll
-        for (int k = 0; k < WARP_TOKENS; ++k) {
+        for (int k = 0; k < TOKENS_AHEAD; ++k) {
             const bool there = r0 + k < count;
-            const size_t t = (size_t)first + (there ? r0 + k : 0);
-            na[k] = there ? p.a[t * p.width + cc] : 1.f;
-            nb[k] = there ? p.inflow[t * p.width + cc] : 0.f;
-            ng[k] = there ? p.y[t * p.ld + cc] : 0.f;
+            na[k] = there ? a_at[(size_t)(r0 + k) * step_w] : 1.f;
+            nb[k] = there ? b_at[(size_t)(r0 + k) * step_w] : 0.f;
+            ng[k] = there ? g_at[(size_t)(r0 + k) * step_y] : 0.f;
         }
     };
-    fetch(warp * WARP_TOKENS);
-    for (int base = 0; base < count; base += SCAN_SPAN) {
-        const int r0 = base + warp * WARP_TOKENS;
+    fetch(group * TOKENS_AHEAD);
+    for (int base = 0; base < count; base += SPAN) {
+        const int r0 = base + group * TOKENS_AHEAD;
 #pragma unroll
-        for (int k = 0; k < WARP_TOKENS; ++k) a[k] = na[k], b[k] = nb[k], g[k] = ng[k];
-        if (base + SCAN_SPAN < count) fetch(r0 + SCAN_SPAN);      // the next span's rows travel while this one is walked
+        for (int k = 0; k < TOKENS_AHEAD; ++k) a[k] = na[k], b[k] = nb[k], g[k] = ng[k];
+        if (base + SPAN < count) fetch(r0 + SPAN);          // the next span's rows travel while this one is walked
         float end = 0.f, decay = 1.f;
 #pragma unroll
-        for (int k = 0; k < WARP_TOKENS; ++k) {
+        for (int k = 0; k < TOKENS_AHEAD; ++k) {
             end = fmaf(a[k], end, b[k]);
             decay *= a[k];
         }
-        ends[warp][lane] = end;
-        decays[warp][lane] = decay;
+        // the groups of a warp, then the warps
+        const int in_warp = threadIdx.x & 31;
+#pragma unroll
+        for (int o = LANES; o < 32; o *= 2) {
+            const float other_end = __shfl_up_sync(0xffffffffu, end, o), other_decay = __shfl_up_sync(0xffffffffu, decay, o);
+            if (in_warp >= o) {
+                end = fmaf(decay, other_end, end);
+                decay *= other_decay;
+            }
+        }
+        float before_end = 0.f, before_decay = 1.f;         // of this warp's groups ahead of this one
+        if (LANES < 32) {
+            const float e = __shfl_up_sync(0xffffffffu, end, LANES % 32), d = __shfl_up_sync(0xffffffffu, decay, LANES % 32);
+            if (in_warp >= LANES) before_end = e, before_decay = d;
+        }
+        if (in_warp >= 32 - LANES) ends[warp][lane] = make_float2(decay, end);
         __syncthreads();
         float S = carry[lane];
-        for (int w = 0; w < warp; ++w) S = fmaf(decays[w][lane], S, ends[w][lane]);
 #pragma unroll
-        for (int k = 0; k < WARP_TOKENS; ++k) {
+        for (int w = 0; w < SCAN_WARPS - 1; ++w) {
+            const float2 e = ends[w][lane];
+            if (w < warp) S = fmaf(e.x, S, e.y);
+        }
+        S = fmaf(before_decay, S, before_end);
+#pragma unroll
+        for (int k = 0; k < TOKENS_AHEAD; ++k) {
             S = fmaf(a[k], S, b[k]);
-            if (live && r0 + k < count)
-                out[((size_t)first + r0 + k) * p.width + c] = from_float<TO>(S * ring_gelu_tanh(g[k] + y_bias));
+            if (live && r0 + k < count) out[(size_t)(r0 + k) * step_w] = from_float<TO>(S * gate_of<TO>(g[k] + y_bias));
         }
         __syncthreads();
-        if (warp == SCAN_WARPS - 1) carry[lane] = S;       // (tokens that are not there leave S as it is)
+        if (group == SCAN_THREADS / LANES - 1) carry[lane] = S;      // (tokens that are not there leave S as it is)
         __syncthreads();
     }
-    if (warp == 0 && live) *state = carry[lane];
+    if (group == 0 && live) *state = carry[lane];
     // the convolution's last inputs, each in its position's row of the ring
     if (p.taps > 1 && live) {
         const int kept = min(count, p.taps);
         const float x_bias = p.x_bias ? p.x_bias[c] : 0.f;
         const int pos0 = p.positions[first];
-        for (int k = warp; k < kept; k += SCAN_WARPS) {
+        for (int k = group; k < kept; k += SCAN_THREADS / LANES) {
             const int r = count - kept + k;
             p.ring[(size_t)slot * p.slot_stride + (size_t)((pos0 + r) % p.taps) * p.width + c] =
                 p.x[((size_t)first + r) * p.ld + c] + x_bias;
         }
     }
 }
+
 // single tokens: a thread a channel
 template <typename TO>
 __global__ void rglru_step_kernel(ScanArgs p) {
@@ -201,9 +234,17 @@ LIA_EXPORT int lia_rglru_scan(const float* a, const float* inflow, const float* 
     ScanArgs p = {a, inflow, y, ld, y_bias, x, x_bias, ring, state, slot_stride, segments, n_segments, single_rows, n_single,
                   positions, slots, out, width, taps};
     if (n_segments > 0) {
-        const dim3 grid(n_segments, (width + 31) / 32);
-        const int rc = out_dtype == LIA_F32 ? lia_launch(rglru_scan_kernel<float>, grid, dim3(SCAN_WARPS * 32), 0, stream, p)
-                                            : lia_launch(rglru_scan_kernel<__nv_bfloat16>, grid, dim3(SCAN_WARPS * 32), 0, stream, p);
+        // as many channels a CTA as still give about two CTAs an SM (32 channels: whole 128-byte rows)
+        const int lanes = (long long)n_segments * width / 32 >= 256 ? 32 : (long long)n_segments * width / 16 >= 256 ? 16 : 8;
+        const dim3 grid(n_segments, (width + lanes - 1) / lanes);
+        int rc;
+#define LIA_SCAN(TO)                                                                                                          \
+    rc = lanes == 32   ? lia_launch(rglru_scan_kernel<TO, 32>, grid, dim3(SCAN_THREADS), 0, stream, p)                         \
+         : lanes == 16 ? lia_launch(rglru_scan_kernel<TO, 16>, grid, dim3(SCAN_THREADS), 0, stream, p)                         \
+                       : lia_launch(rglru_scan_kernel<TO, 8>, grid, dim3(SCAN_THREADS), 0, stream, p)
+        if (out_dtype == LIA_F32) LIA_SCAN(float);
+        else LIA_SCAN(__nv_bfloat16);
+#undef LIA_SCAN
         if (rc != LIA_OK || n_single <= 0) return rc;
     }
     const dim3 grid(n_single, (width + 127) / 128);

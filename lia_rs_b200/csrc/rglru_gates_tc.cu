@@ -200,7 +200,7 @@ LIA_EXPORT int lia_rglru_gates_tc(const void* u, const void* w_r, const void* w_
     p.n_tokens = n_tokens; p.width = width; p.size = width / blocks; p.error_flag = error_flag;
     p.kblocks = (p.size + BLOCK_K - 1) / BLOCK_K;
     const int f_tiles = (p.size + TILE_F - 1) / TILE_F;
-    p.n_tile = 128;                                     // as wide as still gives every SM a CTA, 32 at least
+    p.n_tile = 64;                                      // as wide as still gives every SM a CTA, 32 at least
     while (p.n_tile > 32 && (long long)((n_tokens + p.n_tile - 1) / p.n_tile) * f_tiles * blocks < sm_count) p.n_tile /= 2;
     p.tmem_cols = 2 * p.n_tile;                         // 64, 128 or 256: two CTAs an SM fit
     CUtensorMap mr, mi, mu;

@@ -89,6 +89,12 @@ __global__ void ring_conv_run_kernel(const float* __restrict__ x, long long ld, 
         return v;
     };
     float4 own[RUN];
+    int row_slot[RUN], row_pos[RUN];
+#pragma unroll
+    for (int r = 0; r < RUN; ++r) {
+        row_slot[r] = t0 + r < n_tokens ? slots[t0 + r] : -1;
+        row_pos[r] = t0 + r < n_tokens ? positions[t0 + r] : 0;
+    }
 #pragma unroll
     for (int r = 0; r < RUN; ++r) own[r] = t0 + r < n_tokens ? input(t0 + r) : zero;
     const float4 b = bias ? *reinterpret_cast<const float4*>(bias + c) : zero;
@@ -100,7 +106,7 @@ __global__ void ring_conv_run_kernel(const float* __restrict__ x, long long ld, 
     for (int r = 0; r < RUN; ++r) {
         const int t = t0 + r;
         if (t >= n_tokens) break;
-        const int slot = slots[t], pos = positions[t];
+        const int slot = row_slot[r], pos = row_pos[r];
         if (slot >= 0) {
             if (slot != last_slot || pos != last_pos + 1) {
                 const int m = ring_run_before(positions, slots, t, slot, pos, TAPS - 1);

@@ -31,23 +31,43 @@ struct SingleInput {
 };
 
 template <int VEC>                            // columns of the state that a thread takes (4: P and the addresses allow it)
-__global__ void __launch_bounds__(SSD_THREADS)
+__global__ void __launch_bounds__(SSD_THREADS, 4)
 ssd_single_kernel(SsdArgs p, SingleInput in) {
     extern __shared__ float ssd_single_shared[];          // B [N], C [N], x [P], partial sums [SSD_THREADS VEC]
     pdl_launch_dependents();
-    pdl_wait();
+    // (the step's metadata depends on no kernel of the step)
     const int t = p.single_rows[blockIdx.x], h = blockIdx.y;
-    if (t < 0) return;
-    const int slot = p.slots[t];
+    const int slot = t >= 0 ? p.slots[t] : -1;
+    const int pos = in.raw && t >= 0 ? in.positions[t] : 0;
+    pdl_wait();
     if (slot < 0) return;
     const int N = p.N, P = p.P;
+    float* S = p.state + (size_t)slot * p.slot_stride + (size_t)h * N * P;
+    const int lanes = P / VEC, rows = SSD_THREADS / lanes;
+    const int group = threadIdx.x / lanes, j = (threadIdx.x % lanes) * VEC;
+    constexpr int AHEAD = 8;                              // (eight rows of the state at a time: their loads are in flight together)
+    float held[AHEAD][VEC];
+    auto load = [&](int i0) {
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+            const int i = i0 + k * rows;
+            if (group < rows && i < N) {
+                if constexpr (VEC == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(S + (size_t)i * P + j);
+                    held[k][0] = v.x, held[k][1] = v.y, held[k][2] = v.z, held[k][3] = v.w;
+                } else {
+                    held[k][0] = S[(size_t)i * P + j];
+                }
+            }
+        }
+    };
+    load(group);                                          // (under way while x, B and C arrive)
     float* bs = ssd_single_shared;
     float* cs = bs + N;
     float* xs = cs + N;
     float* partial = xs + P;
     const int per_group = p.heads / p.groups, g = h / per_group;
     const int b_at = p.heads * P + g * N, c_at = p.heads * P + (p.groups + g) * N;
-    const int pos = in.raw ? in.positions[t] : 0;
     float* ring = in.ring ? in.ring + (size_t)slot * in.ring_stride : nullptr;
     for (int e = threadIdx.x; e < 2 * N + P; e += SSD_THREADS) {
         const int c = e < N ? b_at + e : e < 2 * N ? c_at + e - N : h * P + e - 2 * N;
@@ -73,26 +93,6 @@ ssd_single_kernel(SsdArgs p, SingleInput in) {
     }
     const float dt = ring_softplus(p.dt[(size_t)t * p.ld_dt + h] + p.dt_bias[h]);
     const float decay = expf(-p.rate[h] * dt);
-    float* S = p.state + (size_t)slot * p.slot_stride + (size_t)h * N * P;
-    const int lanes = P / VEC, rows = SSD_THREADS / lanes;
-    const int group = threadIdx.x / lanes, j = (threadIdx.x % lanes) * VEC;
-    constexpr int AHEAD = 8;                              // (eight rows of the state at a time: their loads are in flight together)
-    float held[AHEAD][VEC];
-    auto load = [&](int i0) {
-#pragma unroll
-        for (int k = 0; k < AHEAD; ++k) {
-            const int i = i0 + k * rows;
-            if (group < rows && i < N) {
-                if constexpr (VEC == 4) {
-                    const float4 v = *reinterpret_cast<const float4*>(S + (size_t)i * P + j);
-                    held[k][0] = v.x, held[k][1] = v.y, held[k][2] = v.z, held[k][3] = v.w;
-                } else {
-                    held[k][0] = S[(size_t)i * P + j];
-                }
-            }
-        }
-    };
-    load(group);                                          // (under way while x, B and C arrive)
     __syncthreads();
     if (group < rows) {
         float xj[VEC], acc[VEC];

@@ -168,7 +168,8 @@ ssd_sums_tc_kernel(SsdArgs p) {
 template <int TILES>
 __global__ void __launch_bounds__(TC_THREADS)
 ssd_output_tc_kernel(SsdArgs p) {
-    // C [TOKENS][N + 8], B [TOKENS][N + 8], x [TOKENS][P + 8], the incoming state near and rest [N][P + 8] each
+    // C [TOKENS][N + 8], x [TOKENS][P + 8], then B [TOKENS][N + 8] and, in the same room once the chunk's own tokens are done
+    // with, the incoming state near and rest [N][P + 8] each: two CTAs an SM at the sizes of real models
     extern __shared__ __align__(16) uint8_t out_raw[];
     __shared__ float steps[TOKENS], logs[TOKENS], scratch[4];
     pdl_launch_dependents();
@@ -177,64 +178,31 @@ ssd_output_tc_kernel(SsdArgs p) {
     if (!find_tokens(p, blockIdx.x, &first, &len)) return;
     const int h = blockIdx.y, N = p.N, P = p.P, ns = N + 8, ps = P + 8;
     __nv_bfloat16* cs = reinterpret_cast<__nv_bfloat16*>(out_raw);
-    __nv_bfloat16* bs = cs + TOKENS * ns;
-    __nv_bfloat16* xs = bs + TOKENS * ns;
-    __nv_bfloat16* sh = xs + TOKENS * ps;
+    __nv_bfloat16* xs = cs + TOKENS * ns;
+    __nv_bfloat16* bs = xs + TOKENS * ps;
+    __nv_bfloat16* sh = bs;
     __nv_bfloat16* sl = sh + N * ps;
     const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(p.xbc) + (size_t)first * p.ld;
     const int g = h / (p.heads / p.groups);
     bring_rows(cs, rows + (size_t)p.heads * P + (size_t)(p.groups + g) * N, p.ld, len, N);
     bring_rows(bs, rows + (size_t)p.heads * P + (size_t)g * N, p.ld, len, N);
     bring_rows(xs, rows + (size_t)h * P, p.ld, len, P);
-    const float* S = p.sums + ((size_t)blockIdx.x * p.heads + h) * N * P;
-#pragma unroll 4
-    for (int e = threadIdx.x; e < N * (P / 4); e += TC_THREADS) {
-        const int n = e / (P / 4), i = (e - n * (P / 4)) * 4;
-        const float4 v = *reinterpret_cast<const float4*>(S + (size_t)n * P + i);
-        uint2 near, rest;
-        split_pair(v.x, v.y, near.x, rest.x);
-        split_pair(v.z, v.w, near.y, rest.y);
-        *reinterpret_cast<uint2*>(sh + n * ps + i) = near;
-        *reinterpret_cast<uint2*>(sl + n * ps + i) = rest;
-    }
     token_steps(p, first, len, h, steps, logs, scratch);
     rows_there();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, tq = lane & 3;
     const int r0 = warp * 16;
-    if (r0 >= len) return;
+    const bool active = r0 < len;
     const int col_tiles = P / 16, k_tiles = N / 16;
     float acc[2 * TILES][4];
 #pragma unroll
     for (int j = 0; j < 2 * TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     const uint32_t c_at = shared_address(cs + (r0 + (lane & 15)) * ns + (lane >> 4) * 8);
-    // what comes in from the chunk's start: C_t . S_in, decayed
-    for (int k = 0; k < k_tiles; ++k) {
-        uint32_t a[4];
-        ldsm4(c_at + k * 32, a);
-#pragma unroll
-        for (int c = 0; c < TILES; ++c) {
-            if (c >= col_tiles) break;
-            uint32_t b[4], d[4];
-            const int at = (k * 16 + (lane & 15)) * ps + c * 16 + (lane >> 4) * 8;
-            ldsm4_trans(shared_address(sh + at), b);
-            ldsm4_trans(shared_address(sl + at), d);
-            mma(acc[2 * c], a, b[0], b[1]);
-            mma(acc[2 * c + 1], a, b[2], b[3]);
-            mma(acc[2 * c], a, d[0], d[1]);
-            mma(acc[2 * c + 1], a, d[2], d[3]);
-        }
-    }
     const int t_low = r0 + gr, t_high = t_low + 8;
     const float log_low = logs[t_low], log_high = logs[t_high];
-    {
-        const float w_low = pow2(log_low), w_high = pow2(log_high);
-#pragma unroll
-        for (int j = 0; j < 2 * TILES; ++j) acc[j][0] *= w_low, acc[j][1] *= w_low, acc[j][2] *= w_high, acc[j][3] *= w_high;
-    }
     // the chunk's own tokens up to this warp's, 32 at a time
     const float skip = p.skip[h];
-    for (int j0 = 0; j0 < r0 + 16; j0 += 32) {
+    for (int j0 = 0; active && j0 < r0 + 16; j0 += 32) {
         float s[4][4];
 #pragma unroll
         for (int q = 0; q < 4; ++q) s[q][0] = s[q][1] = s[q][2] = s[q][3] = 0.f;
@@ -278,6 +246,45 @@ ssd_output_tc_kernel(SsdArgs p) {
             }
         }
     }
+    // what comes in from the chunk's start: C_t . S_in, decayed
+    __syncthreads();
+    const float* S = p.sums + ((size_t)blockIdx.x * p.heads + h) * N * P;
+#pragma unroll 8
+    for (int e = threadIdx.x; e < N * (P / 4); e += TC_THREADS) {
+        const int n = e / (P / 4), i = (e - n * (P / 4)) * 4;
+        const float4 v = *reinterpret_cast<const float4*>(S + (size_t)n * P + i);
+        uint2 near, rest;
+        split_pair(v.x, v.y, near.x, rest.x);
+        split_pair(v.z, v.w, near.y, rest.y);
+        *reinterpret_cast<uint2*>(sh + n * ps + i) = near;
+        *reinterpret_cast<uint2*>(sl + n * ps + i) = rest;
+    }
+    __syncthreads();
+    if (!active) return;
+    const float w_low = pow2(log_low), w_high = pow2(log_high);
+#pragma unroll
+    for (int c = 0; c < TILES; ++c) {
+        if (c >= col_tiles) break;
+        float in[2][4] = {};
+        for (int k = 0; k < k_tiles; ++k) {
+            uint32_t a[4], b[4], d[4];
+            ldsm4(c_at + k * 32, a);
+            const int at = (k * 16 + (lane & 15)) * ps + c * 16 + (lane >> 4) * 8;
+            ldsm4_trans(shared_address(sh + at), b);
+            ldsm4_trans(shared_address(sl + at), d);
+            mma(in[0], a, b[0], b[1]);
+            mma(in[1], a, b[2], b[3]);
+            mma(in[0], a, d[0], d[1]);
+            mma(in[1], a, d[2], d[3]);
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            acc[2 * c + e][0] = fmaf(w_low, in[e][0], acc[2 * c + e][0]);
+            acc[2 * c + e][1] = fmaf(w_low, in[e][1], acc[2 * c + e][1]);
+            acc[2 * c + e][2] = fmaf(w_high, in[e][2], acc[2 * c + e][2]);
+            acc[2 * c + e][3] = fmaf(w_high, in[e][3], acc[2 * c + e][3]);
+        }
+    }
     float* y = p.y + (size_t)(first + r0) * p.heads * P + (size_t)h * P;
 #pragma unroll
     for (int j = 0; j < 2 * TILES; ++j) {
@@ -289,7 +296,10 @@ ssd_output_tc_kernel(SsdArgs p) {
 }
 
 size_t sums_bytes(int N, int P) { return (size_t)TOKENS * ((N + 8) + 2 * (P + 8)) * 2; }
-size_t output_bytes(int N, int P) { return ((size_t)TOKENS * (2 * (N + 8) + P + 8) + (size_t)2 * N * (P + 8)) * 2; }
+size_t output_bytes(int N, int P) {
+    const size_t b = (size_t)TOKENS * (N + 8), state = (size_t)2 * N * (P + 8);
+    return ((size_t)TOKENS * (N + 8 + P + 8) + (b > state ? b : state)) * 2;
+}
 constexpr size_t MOST_BYTES = 225 * 1024;
 
 template <int TILES>
