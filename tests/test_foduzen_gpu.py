@@ -128,6 +128,30 @@ def test_mixed_batches_on_reused_pages_and_slots(models, name, dtype):
                         f"{name} mixed {request}", model["config"])
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["fod-A", "fod-C"])
+def test_nineteen_requests_decode_together(models, name, dtype):
+    """More single tokens than a tile of the recurrent unit's step holds, with rows of nobody behind them; launched, captured and
+    replayed steps; three requests end on the way."""
+    model = models[name]
+    engine = make_engine(model, dtype, 19 * 48, max_seqs=19)
+    replay = helpers.Replayer(engine)
+    tokens = {f"r{i}": tokens_of(model, 15 + i % 5, 200 + i) for i in range(19)}
+    heads = {r: 2 + i % 4 for i, r in enumerate(tokens)}
+    rows = {r: [] for r in tokens}
+    for r, t in tokens.items():
+        rows[r].append(replay.step([(r, t[:heads[r]], range(heads[r]))]))
+    for step in range(10):
+        live = [r for i, r in enumerate(tokens) if not (step >= 7 and i in (0, 7, 18))]
+        ends = [r for i, r in enumerate(tokens) if step == 6 and i in (0, 7, 18)]
+        out = replay.step([(r, [tokens[r][heads[r] + step]], [0]) for r in live], end=ends)
+        for r, row in zip(live, out):
+            rows[r].append(row[None])
+    for r, t in tokens.items():
+        got = np.concatenate(rows[r])
+        fh.assert_close(got, fh.plain_logits(model, t)[:len(got)], dtype, f"{name} {r}", model["config"])
+
+
 @pytest.mark.parametrize("name", MODELS)
 def test_ways_of_cutting_agree_in_32_bit(models, name):
     """Whole, portions and token by token give the same logits far inside the 32-bit tolerance."""

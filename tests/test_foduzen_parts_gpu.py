@@ -365,6 +365,60 @@ def _request(d, dv, window):
     return KVCacheRequest(1, d, window, v_head_dim=dv)
 
 
+@pytest.mark.parametrize("window", [None, 300])
+@pytest.mark.parametrize("d,dv,heads,kv_heads", [(64, 128, 8, 2), (128, 64, 4, 4), (32, 64, 12, 1), (64, 32, 6, 3), (64, 128, 24, 2)])
+def test_unequal_head_sizes_with_keys_cut_into_ranges(d, dv, heads, kv_heads, window):
+    """A token's keys cut into ranges that meet through scratch memory (by the last of its CTAs and by the merging kernel) and as
+    clusters; a portion's keys cut into ranges of the prompt kernel where it takes the sizes."""
+    from lia_rs_b200.kernels import ops
+    g = torch.Generator().manual_seed(d + dv + heads)
+    T, page = 700, 16
+    pages = (T + page - 1) // page
+    k, v = bf(torch.randn(pages * page, kv_heads, d, generator=g)), bf(torch.randn(pages * page, kv_heads, dv, generator=g))
+    q = bf(torch.randn(T, heads, d, generator=g))
+    order = torch.randperm(pages, generator=g)
+    kp, vp = torch.empty(pages, page, kv_heads, d, dtype=BF16), torch.empty(pages, page, kv_heads, dv, dtype=BF16)
+    kp[order], vp[order] = k.view(pages, page, kv_heads, d), v.view(pages, page, kv_heads, dv)
+    kp, vp, table = dev(kp), dev(vp), ints(order.tolist()).view(1, pages)
+    scale = d ** -0.5
+    visible = pf.window_mask(torch.arange(T), window)
+    want = torch.zeros(T, heads, dv, dtype=F64)
+    for a in range(heads):
+        scores = q[:, a].to(F64) @ k[:T, a // (heads // kv_heads)].to(F64).T * scale
+        want[:, a] = torch.softmax(scores.masked_fill(~visible, float("-inf")), dim=-1) @ v[:T, a // (heads // kv_heads)].to(F64)
+    want = want.reshape(T, heads * dv)
+    positions, slots, qd = ints(range(T)), ints([0] * T), dev(q.reshape(T, heads * d))
+    picked = [0, 63, 64, 299, 300, 301, 699]
+    rows = ints(picked)
+    groups = kv_heads * ((heads // kv_heads + 15) // 16)
+    for splits in (1, 3, 11):
+        for counted in (True, False):
+            partial = torch.full((T * heads * splits * (dv + 1),), float("nan"), device=DEV) if splits > 1 else None
+            counters = torch.zeros(len(picked) * groups, dtype=torch.int32, device=DEV) if counted else None
+            out = torch.zeros(T, heads * dv, dtype=BF16, device=DEV)
+            ops.attention_decode(qd, kp, vp, rows, positions, slots, table, out, partial, heads, kv_heads, d, window, scale, 0, splits,
+                                 counters)
+            close(out[picked], want[picked], 1.5e-2, f"{splits} ranges, counted {counted}")
+            assert counters is None or int(counters.abs().max()) == 0
+    fit = ops.attention_decode_cluster_splits(d, heads // kv_heads, len(picked) * groups, 8, dv)
+    if fit > 1:
+        out = torch.zeros(T, heads * dv, dtype=BF16, device=DEV)
+        ops.attention_decode(qd, kp, vp, rows, positions, slots, table, out, None, heads, kv_heads, d, window, scale, 0, fit, None,
+                             cluster=True)
+        close(out[picked], want[picked], 1.5e-2, f"clusters of {fit}")
+    per_tile = ops.attention_prefill_tc_tokens_per_tile(heads // kv_heads, d, dv)
+    assert (per_tile > 0) == (d >= 64 and dv >= 64 and 128 % (heads // kv_heads) == 0)
+    if per_tile:
+        for splits in (1, 3):
+            segments = ints([0, 0, 500, 500, 500, 200])
+            tiles = -(-500 // per_tile) - (-200 // per_tile)
+            partial = torch.full((ops.attention_prefill_tc_partial_floats(T, heads, dv, splits),), float("nan"), device=DEV) if splits > 1 else None
+            out = torch.zeros(T, heads * dv, dtype=BF16, device=DEV)
+            ops.attention_prefill_tc(qd, kp, vp, segments, 2, tiles, slots, table, out, heads, kv_heads, d, window, scale,
+                                     splits=splits, partial=partial)
+            close(out, want, 1.5e-2, f"portions, {splits} ranges")
+
+
 # ---- the state-space recurrence ----
 
 RIGHT = [dict(heads=4, vdim=12, state=20, groups=2, norm_groups=4, conv=3), dict(heads=3, vdim=8, state=6, groups=1, norm_groups=1, conv=5),
