@@ -279,7 +279,7 @@ attention_decode_kernel(Params p) {
 
     // ---- Q fragments: rows = heads (row r -> head h0 + r), zero beyond `heads` ----
     uint32_t qb[D / 16][NH][2];          // Q^T as the MMA's second operand: lane (g, t) holds head g (+ 8), d = 2t, 2t + 1 (+ 8)
-    if constexpr (D == DV) if (p.qkv) {
+    if (D == DV && p.qkv) {
         __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + STAGES * STAGE_BYTES);       // [16][D]
         const int width = (p.nq + 2 * p.nkv) * D;
         const float* row = p.qkv + (size_t)t * width;
@@ -387,8 +387,7 @@ attention_decode_kernel(Params p) {
                 qb[kk][h][0] = *reinterpret_cast<const uint32_t*>(src);
                 qb[kk][h][1] = *reinterpret_cast<const uint32_t*>(src + 8);
             }
-    }
-    if (D != DV || !p.qkv) {
+    } else {
         pdl_wait();
         const int r0 = lane >> 2, c = (lane & 3) * 2;
         const __nv_bfloat16* base = p.q + ((size_t)t * p.nq + h0) * D;

@@ -37,6 +37,8 @@
 //
 // Epilogues as in the other product kernels: STORE out = alpha*acc; ACCUM out += alpha*acc;
 // SWIGLU: a block's 16 rows are 8 gate rows and the 8 matching up rows, out = up * gate/(1+exp(-gate)).
+#include <string.h>
+
 #include "common.cuh"
 
 #define GEMM_STORE 0
@@ -125,9 +127,8 @@ struct Args {
     int stages, early, chunks, ck;   // ring; stages asked for before the tokens' rows; K chunks per block; elements of K per chunk (a multiple of 64)
     int blocks, x_pitch, stage_bytes, half_bytes;
     int norm, out_bf16;              // norm: 0 none, 1 weight bf16, 2 weight f32
-    float act_p, act_n;              // xIELU's two constants
     int activation;                  // STORE only: 0 none, 1 GELU (tanh form), 2 SiLU, applied to alpha * sum before the store
-    float alpha, eps;
+    float alpha, eps;                // (GEMM_STORE_XIELU: alpha is 1; `alpha` is xIELU's first constant, `activation` the second's bits)
     int* error_flag;
 };
 
@@ -388,7 +389,7 @@ gemm_stream_kernel(Args a) {
                             value = fmaxf(value, 0.f);
                             value *= value;
                         } else if (MODE == GEMM_STORE_XIELU) {
-                            value = lia_xielu_fast(value, a.act_p, a.act_n);
+                            value = lia_xielu_fast(total, a.alpha, __int_as_float(a.activation));
                         }
                         if (a.out_bf16) reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)token * a.ldo + f] = __float2bfloat16_rn(value);
                         else reinterpret_cast<float*>(a.out)[(size_t)token * a.ldo + f] = value;
@@ -735,7 +736,7 @@ LIA_EXPORT int lia_gemm_stream_stages(int mode, int M, int N, int K, int with_no
 // pointers that are not 16-byte aligned (bulk copies and 16-byte loads need both), and sizes whose rows do not
 // fit in shared memory beside a ring (ask lia_gemm_stream_stages first).  `stages_cap` > 0 limits the ring;
 // `early_stages` > 0 sets how many stages the producer asks for before the tokens' rows have been asked for (default 2).
-// `activation`: STORE: 1 the tanh form of GELU, 2 SiLU, 3 the square of ReLU, 5 xIELU with the constants act_p, act_n; SWIGLU: 4 makes the gate a ReLU; applied to the 32-bit result before it is stored.
+// `activation`: STORE: 1 the tanh form of GELU, 2 SiLU, 3 the square of ReLU, 5 xIELU with the constants act_p, act_n (alpha 1); SWIGLU: 4 makes the gate a ReLU; applied to the 32-bit result before it is stored.
 LIA_EXPORT int lia_gemm_stream(int mode, const void* X, int ldx, const void* W, int ldw, void* out, int out_dtype,
                                int ldo, int M, int N, int K, float alpha, const float* norm_src, int ld_norm,
                                const void* norm_weight, int norm_weight_dtype, float eps, int sms, int stages_cap,
@@ -766,8 +767,12 @@ LIA_EXPORT int lia_gemm_stream(int mode, const void* X, int ldx, const void* W, 
     a.norm = !norm_src ? 0 : (norm_weight_dtype == LIA_BF16 ? 1 : 2);
     a.out_bf16 = out_dtype == LIA_BF16;
     a.activation = activation;
-    a.act_p = act_p; a.act_n = act_n;
     a.ldw = ldw; a.ldx = ldx; a.ldo = ldo; a.M = M; a.N = N; a.K = K; a.alpha = alpha; a.error_flag = error_flag;
+    if (form == GEMM_STORE_XIELU) {
+        if (alpha != 1.0f) return LIA_ERR_SIZE;
+        a.alpha = act_p;
+        memcpy(&a.activation, &act_n, sizeof(float));
+    }
     chunking(K, &a.chunks, &a.ck);
     const long long blocks = mode == GEMM_SWIGLU ? (N + HALF_ROWS - 1) / HALF_ROWS : (N + ROWS - 1) / ROWS;
     if (blocks > 2147483647LL) return LIA_ERR_SIZE;
