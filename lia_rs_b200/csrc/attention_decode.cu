@@ -48,11 +48,15 @@ struct Params {
     int rotary_dim, write_kv, num_pages;
     int cluster;                     // the CTAs of a token's ranges are one cluster (gridDim.z of them) and merge in shared memory
     int all_new;                     // any of a row's keys may have been written by this step's kernels (rows of prompt portions), not only its own
-    int sink;                        // 1: one is added to the softmax's denominator (a key of score 0 without a value), where a token's ranges meet
+    int sink;                        // 1: exp(the head's sink) is added to the softmax's denominator (a key of that score without a value), where a token's ranges meet
+    const float* sinks;              // [nq] the heads' sinks; null: zero for every head
     int* error_flag;
 };
 
 constexpr int MAX_FUSED_SPLITS = 128;     // ranges that the last CTA of a token can merge (its weights lie in shared memory)
+
+// The sink of head h as a base-2 logarithm.
+__device__ __forceinline__ float sink_log2(const Params& p, int h) { return p.sinks ? p.sinks[h] * LOG2E : 0.f; }
 
 // Keys per range for a token that sees `span` keys: the given length, or (split_len 0) the span cut into
 // n_splits ranges of a multiple of 64 keys.  The second rule depends on the token's own span and on
@@ -151,7 +155,7 @@ __device__ __forceinline__ void cluster_merge(const Params& p, uint8_t* smem, in
                 acc[0] += w * v[c].x; acc[1] += w * v[c].y; acc[2] += w * v[c].z; acc[3] += w * v[c].w;
             }
         }
-        if (p.sink) total += exp2f(-top);
+        if (p.sink) total += exp2f(sink_log2(p, h0 + r) - top);
         const float inv = total > 0.f ? 1.0f / total : 0.f;
         uint2 packed;
         packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
@@ -550,7 +554,7 @@ attention_decode_kernel(Params p) {
             f[w] = exp2_whole(merge_m[w * 16 + r] - top);             // both are whole numbers (or -infinity)
             total += f[w] * merge_l[w * 16 + r];
         }
-        if (p.sink && !p.cluster && p.n_splits <= 1) total += exp2f(-top);
+        if (p.sink && !p.cluster && p.n_splits <= 1) total += exp2f(sink_log2(p, h0 + r) - top);
         const float inv = 1.0f / total;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) merge_f[w * 16 + r] = f[w] * inv;
@@ -638,7 +642,7 @@ attention_decode_kernel(Params p) {
                 acc[0] += w * v[j][0].x; acc[1] += w * v[j][0].y; acc[2] += w * v[j][0].z; acc[3] += w * v[j][0].w;
                 acc[4] += w * v[j][1].x; acc[5] += w * v[j][1].y; acc[6] += w * v[j][1].z; acc[7] += w * v[j][1].w;
             }
-            if (p.sink) total += exp2f(-top);
+            if (p.sink) total += exp2f(sink_log2(p, h0 + r) - top);
             const float inv = 1.0f / total;
             uint4 packed;
             packed.x = pack_bf16(acc[0] * inv, acc[1] * inv);
@@ -663,7 +667,7 @@ attention_decode_kernel(Params p) {
             total += f;
         }
         total = warp_sum(total);                  // the order of this sum depends on `used` alone
-        if (p.sink) total += exp2f(-top);
+        if (p.sink) total += exp2f(sink_log2(p, h0 + r) - top);
         if (lane == 0) totals[r] = total;
     }
     __syncthreads();
@@ -715,7 +719,7 @@ __global__ void attention_merge_kernel(Params p) {
             total += f;
             value += f * p.partial[(at + s) * D + dcol];
         }
-        if (p.sink) total += exp2f(-top);
+        if (p.sink) total += exp2f(sink_log2(p, h) - top);
         p.out[((size_t)t * p.nq + h) * D + dcol] = __float2bfloat16_rn(value / total);
     }
 }
@@ -887,6 +891,7 @@ LIA_EXPORT long long lia_attention_decode_scratch_floats(int n_tokens, int nq, i
 // `cluster` non-zero: `n_splits` is what lia_attention_decode_cluster_splits gave; `partial` and `counters` are not used.
 // `all_new` non-zero: the rows may be tokens of prompt portions of this step, whose earlier keys the kernels ahead
 // have written too; zero: only a row's own key is of this step (decoded tokens), and older tiles are fetched early.
+// `sink`: one is added to the softmax's denominator; `sinks` [nq] (32-bit, or null): exp(sinks[h]) instead, of head h.
 // `n_splits` ranges of `split_len` keys each must cover the longest visible span among the rows;
 // split_len 0 lets every row cut its own span into n_splits ranges (see range_length).
 LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const void* v_pages, const int* rows,
@@ -894,7 +899,7 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
                                     int table_stride, void* out, float* partial, long long partial_floats,
                                     int* counters, int n_tokens, int nq, int nkv, int d, int dv, int page_size, int window, float scale,
                                     int split_len, int n_splits, const float* qkv, const float* inv_freq, int rotary_dim,
-                                    int write_kv, int num_pages, int cluster, int all_new, int sink, float softcap,
+                                    int write_kv, int num_pages, int cluster, int all_new, int sink, const float* sinks, float softcap,
                                     int* error_flag, cudaStream_t stream) {
     if (n_rows <= 0) return LIA_OK;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || split_len < 0 || split_len % TILE_KEYS || n_splits <= 0 ||
@@ -916,7 +921,8 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
     p.error_flag = error_flag;
     p.cluster = cluster ? 1 : 0;
     p.all_new = all_new ? 1 : 0;
-    p.sink = sink ? 1 : 0;
+    p.sink = sink || sinks ? 1 : 0;
+    p.sinks = sinks;
     p.page_shift = -1;
     for (int b = 0; b < 31; ++b)
         if (page_size == (1 << b)) p.page_shift = b;
@@ -929,10 +935,9 @@ LIA_EXPORT int lia_attention_decode(const void* q, const void* k_pages, const vo
     }
     const bool wide = nq / nkv > 8;             // more than 8 query heads per kv head: two groups of 8 per CTA
     if (p.cap_in != 0.f) {
-        if (d != dv) return LIA_ERR_SIZE;       // (a cap with unequal sizes: the caller's other kernel)
-        if (d == 128) return wide ? launch_decode<128, 128, 2, true>(p, n_rows, stream) : launch_decode<128, 128, 1, true>(p, n_rows, stream);
-        if (d == 64) return wide ? launch_decode<64, 64, 2, true>(p, n_rows, stream) : launch_decode<64, 64, 1, true>(p, n_rows, stream);
-        if (d == 32) return wide ? launch_decode<32, 32, 2, true>(p, n_rows, stream) : launch_decode<32, 32, 1, true>(p, n_rows, stream);
+#define LIA_CASE(D, DV) return wide ? launch_decode<D, DV, 2, true>(p, n_rows, stream) : launch_decode<D, DV, 1, true>(p, n_rows, stream)
+        LIA_DECODE_SIZES(LIA_CASE)
+#undef LIA_CASE
         return LIA_ERR_SIZE;
     }
 #define LIA_CASE(D, DV) return wide ? launch_decode<D, DV, 2>(p, n_rows, stream) : launch_decode<D, DV, 1>(p, n_rows, stream)

@@ -126,7 +126,7 @@ LIA_EXPORT int lia_attention_generic(const void* q, const void* k_pages, const v
 // leading part of the first key part (attention through a shared latent: k1 = v = the latent, k2 = the rotated part)
 // passes the k1 pages as values with v_stride = dk1.  q1, q2 and out are addressed by a token stride and a head stride,
 // so that heads may lie side by side in a token's row or in planes of their own.  `sink`: one is added to the softmax's
-// denominator (a key of score 0 that has no value).  `softcap` > 0: score <- softcap * tanh(score / softcap) ahead of
+// denominator (a key of score 0 that has no value); `sinks` [nq]: exp(sinks[h]) instead, of head h.  `softcap` > 0: score <- softcap * tanh(score / softcap) ahead of
 // the softmax.  Sizes: dk1 + dk2 up to 1,024, dv up to 512.
 namespace {
 constexpr int GENERAL_MAX_DK = 1024;
@@ -139,7 +139,8 @@ attention_general_kernel(const T* __restrict__ q1, long long q1_ts, long long q1
                          const int* __restrict__ positions, const int* __restrict__ slots,
                          const int* __restrict__ block_table, int table_stride, const int* __restrict__ rows,
                          T* __restrict__ out, long long o_ts, long long o_hs, int n_tokens, int nq, int nkv,
-                         int page_size, int window, float scale, float softcap, int sink, int num_pages, int* __restrict__ error_flag) {
+                         int page_size, int window, float scale, float softcap, int sink, const float* __restrict__ sinks,
+                         int num_pages, int* __restrict__ error_flag) {
     extern __shared__ float q_general[];                    // [WARPS][dk1 + dk2]
     pdl_launch_dependents();
     pdl_wait();
@@ -166,8 +167,9 @@ attention_general_kernel(const T* __restrict__ q1, long long q1_ts, long long q1
     float acc[DVC];
 #pragma unroll
     for (int c = 0; c < DVC; ++c) acc[c] = 0.f;
-    // with a sink the walk starts from a key of score 0 that has been seen already: maximum 0, sum exp(0 - 0) = 1
-    float running_max = sink ? 0.f : -INFINITY, running_sum = sink ? 1.f : 0.f;
+    // with a sink the walk starts from a key of the sink's score (0 without `sinks`) that has been seen already: its score is
+    // the maximum, the sum is exp(0) = 1
+    float running_max = sinks ? sinks[h] : sink ? 0.f : -INFINITY, running_sum = sinks || sink ? 1.f : 0.f;
 
     for (int base = first; base <= pos; base += 32) {
         const int j = base + lane;
@@ -225,7 +227,7 @@ int launch_general(const void* q1, long long q1_ts, long long q1_hs, const void*
                    const void* k1_pages, int dk1, const void* k2_pages, int dk2, const void* v_pages, int v_stride, int dv,
                    const int* positions, const int* slots, const int* block_table, int table_stride, const int* rows,
                    void* out, long long o_ts, long long o_hs, int n_tokens, int nq, int nkv, int page_size, int window,
-                   float scale, float softcap, int sink, int num_pages, int* error_flag, cudaStream_t stream) {
+                   float scale, float softcap, int sink, const float* sinks, int num_pages, int* error_flag, cudaStream_t stream) {
     const long long blocks = ((long long)n_tokens * nq + WARPS - 1) / WARPS;
     if (blocks > 2147483647LL) return LIA_ERR_SIZE;
     const size_t smem = (size_t)WARPS * (dk1 + dk2) * sizeof(float);
@@ -235,7 +237,7 @@ int launch_general(const void* q1, long long q1_ts, long long q1_hs, const void*
                       (const T*)q1, q1_ts, q1_hs, (const T*)q2, q2_ts, q2_hs, (const T*)k1_pages, dk1,                \
                       (const T*)k2_pages, dk2, (const T*)v_pages, v_stride, dv, positions, slots, block_table,        \
                       table_stride, rows, (T*)out, o_ts, o_hs, n_tokens, nq, nkv, page_size, window, scale, softcap, sink,     \
-                      num_pages, error_flag)
+                      sinks, num_pages, error_flag)
     if (chunks <= 2) LIA_GENERAL(2);
     if (chunks <= 4) LIA_GENERAL(4);
     if (chunks <= 8) LIA_GENERAL(8);
@@ -249,7 +251,8 @@ LIA_EXPORT int lia_attention_general(const void* q1, long long q1_ts, long long 
                                      const void* v_pages, int v_stride, int dv, int dtype, const int* positions,
                                      const int* slots, const int* block_table, int table_stride, const int* rows,
                                      void* out, long long o_ts, long long o_hs, int n_tokens, int nq, int nkv,
-                                     int page_size, int window, float scale, float softcap, int sink, int num_pages, int* error_flag,
+                                     int page_size, int window, float scale, float softcap, int sink, const float* sinks,
+                                     int num_pages, int* error_flag,
                                      cudaStream_t stream) {
     if (n_tokens <= 0) return LIA_OK;
     if (nq <= 0 || nkv <= 0 || nq % nkv || dk1 <= 0 || dk2 < 0 || dk1 + dk2 > GENERAL_MAX_DK || dv <= 0 || dv > 512 ||
@@ -258,11 +261,11 @@ LIA_EXPORT int lia_attention_general(const void* q1, long long q1_ts, long long 
     if (dtype == LIA_F32)
         return launch_general<float>(q1, q1_ts, q1_hs, q2, q2_ts, q2_hs, k1_pages, dk1, k2_pages, dk2, v_pages, v_stride,
                                      dv, positions, slots, block_table, table_stride, rows, out, o_ts, o_hs, n_tokens, nq,
-                                     nkv, page_size, window, scale, softcap, sink, num_pages, error_flag, stream);
+                                     nkv, page_size, window, scale, softcap, sink, sinks, num_pages, error_flag, stream);
     if (dtype == LIA_BF16)
         return launch_general<__nv_bfloat16>(q1, q1_ts, q1_hs, q2, q2_ts, q2_hs, k1_pages, dk1, k2_pages, dk2, v_pages,
                                              v_stride, dv, positions, slots, block_table, table_stride, rows, out, o_ts,
-                                             o_hs, n_tokens, nq, nkv, page_size, window, scale, softcap, sink, num_pages,
+                                             o_hs, n_tokens, nq, nkv, page_size, window, scale, softcap, sink, sinks, num_pages,
                                              error_flag, stream);
     return LIA_ERR_DTYPE;
 }

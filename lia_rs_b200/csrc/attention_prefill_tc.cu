@@ -68,8 +68,12 @@ struct Params {
     float* partial_o;                // [splits][tokens * nq][DV]
     float* partial_ms;               // [splits][tokens * nq][2]: reference point (a whole number, or -infinity), sum
     long long n_rows_total;          // tokens * nq
-    int sink;                        // 1: one is added to the softmax's denominator (a key of score 0 without a value)
+    int sink;                        // 1: exp(the head's sink) is added to the softmax's denominator (a key of that score without a value)
+    const float* sinks;              // [nq] the heads' sinks; null: zero for every head
 };
+
+// The sink of head h as a base-2 logarithm.
+__device__ __forceinline__ float sink_log2(const Params& p, int h) { return p.sinks ? p.sinks[h] * LOG2E : 0.f; }
 
 // CAP: the scores pass a tanh cap (an instantiation of its own, so that the kernel without a cap is what it was)
 template <int D, int DV, bool CAP = false>
@@ -398,7 +402,7 @@ attention_prefill_tc_kernel(Params p) {
                 }
             }
         } else if (ok) {
-            const float inv = 1.0f / (pair_sum[r] + pair_sum[ROWS + r] + (p.sink ? exp2f(-row_max) : 0.f));
+            const float inv = 1.0f / (pair_sum[r] + pair_sum[ROWS + r] + (p.sink ? exp2f(sink_log2(p, kvh * group + head) - row_max) : 0.f));
             __nv_bfloat16* dst = p.out + ((size_t)(q_offset + tok0 + (row_ok ? tok : 0)) * p.nq + kvh * group + head) * DV;
 #pragma unroll 1
             for (int c0 = half * (DV / 2); c0 < (half + 1) * (DV / 2); c0 += 16) {
@@ -490,7 +494,7 @@ __global__ void __launch_bounds__(128) attention_prefill_merge_kernel(Params p) 
             acc[e + 1] = fmaf(w, v.y, acc[e + 1]);
         }
     }
-    if (p.sink) total += exp2f(-top);                  // the sink joins once, where the ranges meet
+    if (p.sink) total += exp2f(sink_log2(p, kvh * group + head) - top);                  // the sink joins once, where the ranges meet
     const float inv = 1.0f / total;
     __nv_bfloat16* dst = p.out + row * D + lane * E;
 #pragma unroll
@@ -523,12 +527,13 @@ LIA_EXPORT int lia_attention_prefill_tc_tokens_per_tile(int group, int d, int dv
 // tokens per tile of this kernel.  With `splits` > 1 every CTA's keys are cut into that many ranges of whole
 // 128-key tiles, each range a CTA of its own, and a second kernel merges them (few tokens over a long context
 // would otherwise leave most SMs idle); `partial` then holds splits * n_tokens * nq * (the values' head size + 2) 32-bit words,
-// `n_tokens` being the tokens of the whole batch that `q` and `out` cover.
+// `n_tokens` being the tokens of the whole batch that `q` and `out` cover.  `sink`: one is added to the softmax's denominator;
+// `sinks` [nq] (32-bit, or null): exp(sinks[h]) instead, of head h.
 LIA_EXPORT int lia_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* segments,
                                         int n_segments, int n_tiles, const int* slots, const int* block_table,
                                         int table_stride, void* out, int nq, int nkv, int d, int dv, int page_size, int window,
                                         float scale, int num_pages, int splits, float* partial, int n_tokens, int sink,
-                                        float softcap, int* error_flag, cudaStream_t stream) {
+                                        const float* sinks, float softcap, int* error_flag, cudaStream_t stream) {
     if (n_segments <= 0 || n_tiles <= 0) return LIA_OK;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || nkv > 65535) return LIA_ERR_SIZE;
     if (splits < 1 || splits > 32 || (splits > 1 && (!partial || n_tokens <= 0))) return LIA_ERR_SIZE;
@@ -552,12 +557,13 @@ LIA_EXPORT int lia_attention_prefill_tc(const void* q, const void* k_pages, cons
     for (int b = 0; b < 31; ++b)
         if (page_size == (1 << b)) p.page_shift = b;
     p.splits = splits;
-    p.sink = sink ? 1 : 0;
+    p.sink = sink || sinks ? 1 : 0;
+    p.sinks = sinks;
     p.n_rows_total = (long long)n_tokens * nq;
     p.partial_o = partial;
     p.partial_ms = partial ? partial + (size_t)splits * p.n_rows_total * dv : nullptr;
     if (d != dv) {
-        if (p.cap_in != 0.f) return LIA_ERR_SIZE;       // (a cap with unequal sizes: the caller's other kernel)
+        if (p.cap_in != 0.f) return d == 64 ? launch<64, 128, true>(p, n_tiles, stream) : launch<128, 64, true>(p, n_tiles, stream);
         return d == 64 ? launch<64, 128>(p, n_tiles, stream) : launch<128, 64>(p, n_tiles, stream);
     }
     if (p.cap_in != 0.f) return d == 128 ? launch<128, 128, true>(p, n_tiles, stream) : launch<64, 64, true>(p, n_tiles, stream);

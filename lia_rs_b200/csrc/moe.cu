@@ -1,11 +1,11 @@
 // A mixture of gated feed-forward experts: each token goes to the `top` experts with the largest router scores.
 //
 //  * `moe_route`: z = W_router x in 32-bit (W_router 32-bit, x in the compute element type), s = softmax(z) over all
-//    router outputs, the `top` outputs with the largest choice score chosen (the lower index wins a tie), their
+//    router outputs or, with `sigmoid`, the logistic function of each, the `top` outputs with the largest choice score chosen (the lower index wins a tie), their
 //    weights s_e * scale, or with `renormalise` s_e / (sum of the chosen s + 1e-20) * scale.  The choice score is s, or
 //    s + correction with a 32-bit `correction` per output; with `groups` > 1 the outputs form that many equal groups
-//    of neighbours, a group's score is its largest choice score, and only outputs of the `keep` best groups can be
-//    chosen.  Outputs from `experts` on name no expert (their pairs belong to no row of the products; `moe_combine`
+//    of neighbours, a group's score is its largest choice score (with `two_best` the sum of its two largest), and only
+//    outputs of the `keep` best groups can be chosen.  Outputs from `experts` on name no expert (their pairs belong to no row of the products; `moe_combine`
 //    adds the token's own input for them).  An optional extra row of the router matrix gives one more logit a token,
 //    whose logistic function is the gate of a shared expert.
 //  * `moe_plan`: the (token, choice) pairs grouped by expert: where each expert's rows begin, which pair each sorted row
@@ -31,9 +31,9 @@ constexpr int MOE_MAX_EXPERTS = 1024, MOE_MAX_TOP = 32;
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ router, int hidden,
                                  int experts, int top, float scale, int extra, const float* __restrict__ correction,
-                                 int groups, int keep, int renormalise, int* __restrict__ ids,
+                                 int groups, int keep, int renormalise, int sigmoid, int two_best, int* __restrict__ ids,
                                  float* __restrict__ weights, float* __restrict__ shared_gate) {
-    extern __shared__ __align__(16) float route_shared[];  // x [hidden], z [experts + extra], choice scores [experts]
+    extern __shared__ __align__(16) float route_shared[];  // x [hidden], z [experts + extra], choice scores [experts], groups' scores [groups]
     __shared__ int picked[MOE_MAX_TOP];
     pdl_launch_dependents();
     pdl_wait();
@@ -66,32 +66,38 @@ __global__ void moe_route_kernel(const T* __restrict__ x, long long ld, const fl
     }
     __syncthreads();
     if (threadIdx.x != 0) return;
-    float largest = -INFINITY;
-    for (int e = 0; e < experts; ++e) largest = fmaxf(largest, z[e]);
-    float total = 0.f;
-    for (int e = 0; e < experts; ++e) {
-        z[e] = expf(z[e] - largest);
-        total += z[e];
+    if (sigmoid) {
+        for (int e = 0; e < experts; ++e) z[e] = 1.0f / (1.0f + expf(-z[e]));
+    } else {
+        float largest = -INFINITY;
+        for (int e = 0; e < experts; ++e) largest = fmaxf(largest, z[e]);
+        float total = 0.f;
+        for (int e = 0; e < experts; ++e) {
+            z[e] = expf(z[e] - largest);
+            total += z[e];
+        }
+        const float inv = 1.0f / total;
+        for (int e = 0; e < experts; ++e) z[e] *= inv;
     }
-    const float inv = 1.0f / total;
-    for (int e = 0; e < experts; ++e) {
-        z[e] *= inv;                                       // the score s_e
-        choice[e] = z[e] + (correction ? correction[e] : 0.f);
-    }
+    for (int e = 0; e < experts; ++e) choice[e] = z[e] + (correction ? correction[e] : 0.f);      // z: the scores s_e
     if (groups > 1) {
-        // the `keep` groups with the largest best choice score stay (the lower group wins a tie); the others' outputs
-        // cannot be chosen
+        // the `keep` groups with the largest group score stay (the lower group wins a tie); the others' outputs cannot
+        // be chosen
         const int size = experts / groups;
+        float* judged = choice + experts;
         for (int g = 0; g < groups; ++g) {
-            float best = -INFINITY;
-            for (int e = g * size; e < (g + 1) * size; ++e) best = fmaxf(best, choice[e]);
-            int ahead = 0;
-            for (int o = 0; o < groups; ++o) {
-                if (o == g) continue;
-                float other = -INFINITY;
-                for (int e = o * size; e < (o + 1) * size; ++e) other = fmaxf(other, choice[e]);
-                if (other > best || (other == best && o < g)) ++ahead;
+            float best = -INFINITY, second = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) {
+                const float v = choice[e];
+                if (v > best) second = best, best = v;
+                else second = fmaxf(second, v);
             }
+            judged[g] = two_best && size > 1 ? best + second : best;
+        }
+        for (int g = 0; g < groups; ++g) {
+            int ahead = 0;
+            for (int o = 0; o < groups; ++o)
+                if (o != g && (judged[o] > judged[g] || (judged[o] == judged[g] && o < g))) ++ahead;
             if (ahead >= keep) {
                 // NaN marks an output that is out of the choice (a choice score may be any number, minus infinity too)
                 for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = __int_as_float(0x7fc00000);
@@ -275,7 +281,7 @@ __global__ void moe_combine_kernel(float* __restrict__ residual, const float* __
         w[threadIdx.x] = weights[(size_t)t * top + threadIdx.x];
     }
     __syncthreads();
-    const float gate = shared_y ? shared_gate[t] : 0.f;
+    const float gate = shared_y ? (shared_gate ? shared_gate[t] : 1.f) : 0.f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float acc = 0.f;
         for (int c = 0; c < top; ++c) {
@@ -297,14 +303,15 @@ LIA_EXPORT int lia_moe_tile_rows() { return TILE_M; }
 // hold at least `top` outputs.  `experts` counts every router output, also those that name no expert.
 LIA_EXPORT int lia_moe_route(const void* x, int dtype, long long ld, const float* router, int n, int hidden, int experts,
                              int top, float scale, int extra, const float* correction, int groups, int keep,
-                             int renormalise, int* ids, float* weights, float* shared_gate, cudaStream_t stream) {
+                             int renormalise, int sigmoid, int two_best, int* ids, float* weights, float* shared_gate,
+                             cudaStream_t stream) {
     if (n <= 0) return LIA_OK;
     if (hidden <= 0 || experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts || top > MOE_MAX_TOP ||
-        extra < 0 || extra > 1 || (extra && !shared_gate) || ld < hidden || (size_t)(hidden + 2 * experts + 1) * 4 > 200 * 1024)
+        extra < 0 || extra > 1 || (extra && !shared_gate) || ld < hidden || (size_t)(hidden + 3 * experts + 1) * 4 > 200 * 1024)
         return LIA_ERR_SIZE;
     if (groups > 1 && (experts % groups || keep < 1 || keep > groups || (long long)keep * (experts / groups) < top))
         return LIA_ERR_SIZE;
-    const size_t bytes = (size_t)(hidden + 2 * experts + extra) * sizeof(float);
+    const size_t bytes = (size_t)(hidden + 2 * experts + extra + (groups > 1 ? groups : 0)) * sizeof(float);
     static bool raised = false;
     if (!raised) {
         cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -313,11 +320,12 @@ LIA_EXPORT int lia_moe_route(const void* x, int dtype, long long ld, const float
     }
     if (dtype == LIA_F32)
         return lia_launch(moe_route_kernel<float>, dim3(n), dim3(256), bytes, stream, (const float*)x, ld, router, hidden,
-                          experts, top, scale, extra, correction, groups, keep, renormalise, ids, weights, shared_gate);
+                          experts, top, scale, extra, correction, groups, keep, renormalise, sigmoid, two_best, ids,
+                          weights, shared_gate);
     if (dtype == LIA_BF16)
         return lia_launch(moe_route_kernel<__nv_bfloat16>, dim3(n), dim3(256), bytes, stream, (const __nv_bfloat16*)x, ld,
-                          router, hidden, experts, top, scale, extra, correction, groups, keep, renormalise, ids, weights,
-                          shared_gate);
+                          router, hidden, experts, top, scale, extra, correction, groups, keep, renormalise, sigmoid, two_best, ids,
+                          weights, shared_gate);
     return LIA_ERR_DTYPE;
 }
 
@@ -372,13 +380,13 @@ LIA_EXPORT int lia_moe_gemm(int mode, const void* a, int dtype, long long lda, c
     return LIA_ERR_DTYPE;
 }
 
-// residual [n, hidden] 32-bit (+)= alpha * (sum_c weights[t, c] y[inverse[t, c]] + shared_gate[t] shared_y[t]); where
+// residual [n, hidden] 32-bit (+)= alpha * (sum_c weights[t, c] y[inverse[t, c]] + shared_gate[t] shared_y[t]) (shared_gate null: ones); where
 // inverse[t, c] < 0 the term is weights[t, c] x[t] (x [n, ld_x] of `x_dtype`; null: such terms are zero).
 LIA_EXPORT int lia_moe_combine(float* residual, const float* y, const int* inverse, const float* weights,
                                const float* shared_y, const float* shared_gate, const void* x, int x_dtype, long long ld_x,
                                int n, int hidden, int top, float alpha, int store, cudaStream_t stream) {
     if (n <= 0) return LIA_OK;
-    if (hidden <= 0 || top <= 0 || top > MOE_MAX_TOP || (shared_y && !shared_gate) || (x && ld_x < hidden)) return LIA_ERR_SIZE;
+    if (hidden <= 0 || top <= 0 || top > MOE_MAX_TOP || (x && ld_x < hidden)) return LIA_ERR_SIZE;
     const int threads = hidden >= 1024 ? 256 : 128;
     if (x && x_dtype == LIA_BF16)
         return lia_launch(moe_combine_kernel<__nv_bfloat16>, dim3(n), dim3(threads), 0, stream, residual, y, inverse, weights,

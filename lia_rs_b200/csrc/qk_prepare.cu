@@ -3,8 +3,8 @@
 //
 //  * `qkv_prepare`: rows [q heads | k heads | v heads] (keys of size d, values of size dv) get, in this order, a bias
 //    (the projection's), an RMS norm per head of q and of k with a weight of size d shared by the heads, the
-//    rotate-half encoding over the first `rot_dims` elements of every q and k head (element i with i + rot_dims/2,
-//    angle position * freq[i]), and a mixing of the values with those that an earlier layer left for the same token,
+//    rotary encoding over the first `rot_dims` elements of every q and k head (element i with i + rot_dims/2, or with
+//    `pairs` 2i with 2i + 1; angle position * freq[i]), with `norm_behind` an RMS norm per head without a weight, and a mixing of the values with those that an earlier layer left for the same token,
 //    v <- (1 - lambda) v + lambda v_first (mode 2; mode 1 leaves v for later layers; mode 0 neither).  q goes out in the
 //    compute element type, k and the mixed v are appended to the pages.
 //  * `latent_prepare`: attention through a latent.  The query rows hold, per head, `d` unrotated elements and then
@@ -33,16 +33,17 @@ __device__ __forceinline__ long long page_row(const int* __restrict__ block_tabl
 }
 
 // One warp norms (optionally) and rotates one head that lies in `h` (shared memory, 32-bit, `d` elements; the rotated
-// span begins at `offset` and is `rot_dims` long), in place.
+// span begins at `offset` and is `rot_dims` long), in place; `behind`: the norm follows the rotation and has no weight.
 __device__ __forceinline__ void norm_and_rotate(float* h, int d, const float* __restrict__ norm_weight, float eps,
                                                 int offset, int rot_dims, const float* rotation, int lane,
-                                                bool pairs = false) {
-    if (norm_weight) {
+                                                bool pairs = false, bool behind = false) {
+    if (norm_weight || behind) {
+        // (a rotation leaves the sum of the squares as it is, so what follows it can be multiplied ahead of it)
         float sum = 0.f;
         for (int i = lane; i < d; i += 32) sum = fmaf(h[i], h[i], sum);
         sum = warp_sum(sum);
         const float inv = 1.0f / sqrtf(sum / (float)d + eps);
-        for (int i = lane; i < d; i += 32) h[i] = h[i] * inv * norm_weight[i];
+        for (int i = lane; i < d; i += 32) h[i] = h[i] * inv * (norm_weight ? norm_weight[i] : 1.0f);
         __syncwarp();
     }
     const int half = rot_dims / 2;
@@ -64,7 +65,8 @@ qkv_prepare_kernel(const float* __restrict__ rows, long long ld, const float* __
                    float* __restrict__ v_first, const int* __restrict__ positions, const int* __restrict__ slots,
                    const int* __restrict__ block_table, int table_stride, T* __restrict__ q_out,
                    T* __restrict__ k_pages, T* __restrict__ v_pages, int n_tokens, int nq, int nkv, int d, int dv,
-                   int page_size, int num_pages, int write_kv, int norm_whole, int* __restrict__ error_flag) {
+                   int page_size, int num_pages, int write_kv, int norm_whole, int pairs, int norm_behind,
+                   int* __restrict__ error_flag) {
     extern __shared__ float prep_shared[];                 // [rot_dims] cosines then sines, then [PREP_WARPS][d]
     __shared__ float whole_scratch[32];
     pdl_launch_dependents();
@@ -105,7 +107,8 @@ qkv_prepare_kernel(const float* __restrict__ rows, long long ld, const float* __
             for (int i = lane; i < d; i += 32) h[i] = h[i] * whole_inv[is_q ? 0 : 1] * w[i];
         }
         __syncwarp();
-        norm_and_rotate(h, d, norm_whole ? nullptr : (is_q ? q_norm : k_norm), eps, 0, rot_dims, rotation, lane);
+        norm_and_rotate(h, d, norm_whole ? nullptr : (is_q ? q_norm : k_norm), eps, 0, rot_dims, rotation, lane, pairs != 0,
+                        norm_behind != 0);
         if (is_q) {
             T* dst = q_out + ((size_t)t * nq + head) * d;
             for (int i = lane; i < d; i += 32) dst[i] = from_float<T>(h[i]);
@@ -193,16 +196,18 @@ latent_prepare_kernel(const float* __restrict__ q_rows, long long ld_q, const fl
 
 // rows [n, ld] 32-bit: nq heads of d, nkv heads of d, nkv heads of dv.  bias (32-bit, the rows' layout) or null;
 // q_norm, k_norm (32-bit [d]; with `norm_whole` [nq d] and [nkv d]: one norm over all of q and one over all of k) or
-// null; freq (32-bit [rot_dims / 2]; rot_dims 0: no encoding).  vmix_mode 1 writes,
+// null; freq (32-bit [rot_dims / 2]; rot_dims 0: no encoding; `pairs`: element 2i turns with 2i + 1).  `norm_behind`: every q
+// and k head is divided by its root mean square behind the encoding (no weights then).  vmix_mode 1 writes,
 // 2 reads v_first (32-bit [n, nkv dv]).  q_out [n, nq d], k_pages [pages, page_size, nkv, d], v_pages [.., nkv, dv].
 LIA_EXPORT int lia_qkv_prepare(const float* rows, long long ld, const float* bias, const float* q_norm,
                                const float* k_norm, float eps, const float* freq, int rot_dims, int vmix_mode,
                                float lambda, float* v_first, const int* positions, const int* slots,
                                const int* block_table, int table_stride, void* q_out, void* k_pages, void* v_pages,
                                int dtype, int n_tokens, int nq, int nkv, int d, int dv, int page_size, int num_pages,
-                               int write_kv, int norm_whole, int* error_flag, cudaStream_t stream) {
+                               int write_kv, int norm_whole, int pairs, int norm_behind, int* error_flag,
+                               cudaStream_t stream) {
     if (n_tokens <= 0) return LIA_OK;
-    if (norm_whole && (!q_norm || !k_norm)) return LIA_ERR_SIZE;
+    if ((norm_whole && (!q_norm || !k_norm)) || (norm_behind && (q_norm || k_norm))) return LIA_ERR_SIZE;
     if (nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0 || rot_dims < 0 || rot_dims > d || (rot_dims & 1) ||
         (rot_dims > 0 && !freq) || ld < (long long)(nq + nkv) * d + (long long)nkv * dv || vmix_mode < 0 || vmix_mode > 2 ||
         (vmix_mode && !v_first) || d > 4096)
@@ -212,7 +217,7 @@ LIA_EXPORT int lia_qkv_prepare(const float* rows, long long ld, const float* bia
     return lia_launch(qkv_prepare_kernel<T>, dim3(n_tokens), dim3(PREP_WARPS * 32), smem, stream, rows, ld, bias,     \
                       q_norm, k_norm, eps, freq, rot_dims, vmix_mode, lambda, v_first, positions, slots, block_table, \
                       table_stride, (T*)q_out, (T*)k_pages, (T*)v_pages, n_tokens, nq, nkv, d, dv, page_size,         \
-                      num_pages, write_kv, norm_whole, error_flag)
+                      num_pages, write_kv, norm_whole, pairs, norm_behind, error_flag)
     if (dtype == LIA_BF16) LIA_PREP(__nv_bfloat16);
     if (dtype == LIA_F32) LIA_PREP(float);
 #undef LIA_PREP

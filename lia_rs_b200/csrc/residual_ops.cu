@@ -2,7 +2,8 @@
 //  * the embedding gather with a learned position vector added, optionally leaving a second copy of the result
 //    (a model that feeds the embedding output in again later keeps it);
 //  * the input of a re-injection x <- W [x; x0] + b: the two streams side by side in the product's element type,
-//    and x set to b in every row so that the product can add into it.
+//    and x set to b in every row so that the product can add into it;
+//  * the sum x <- x + x0 + b of the stream, an earlier copy of it and one vector (either may be absent).
 #include "common.cuh"
 
 namespace {
@@ -43,6 +44,20 @@ __global__ void reinject_input_kernel(float* __restrict__ x, const float* __rest
         xr[i] = bias ? to_float(bias[i]) : 0.f;
     }
 }
+
+template <typename TB>
+__global__ void stream_sum_kernel(float* __restrict__ x, const float* __restrict__ x0, const TB* __restrict__ bias,
+                                  int n_tokens, int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long total = (long long)n_tokens * hidden;
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+        float v = x[e];
+        if (x0) v += x0[e];
+        if (bias) v += to_float(bias[e % hidden]);
+        x[e] = v;
+    }
+}
 }  // namespace
 
 // out[t, :] = table[token_t, :] * scale + position_table[position_t, :], 32-bit; `copy` (optional) receives the same.
@@ -79,5 +94,19 @@ LIA_EXPORT int lia_reinject_input(float* x, const float* x0, const void* bias, i
     if (out_dtype == LIA_F32 && bias_dtype == LIA_BF16) LIA_REINJECT(float, __nv_bfloat16);
     if (out_dtype == LIA_F32 && bias_dtype == LIA_F32) LIA_REINJECT(float, float);
 #undef LIA_REINJECT
+    return LIA_ERR_DTYPE;
+}
+
+// x[t] += x0[t] + bias (x0 [n_tokens, hidden] and bias [hidden] may be null).
+LIA_EXPORT int lia_stream_sum(float* x, const float* x0, const void* bias, int bias_dtype, int n_tokens, int hidden,
+                              cudaStream_t stream) {
+    if (n_tokens <= 0 || (!x0 && !bias)) return LIA_OK;
+    if (hidden <= 0) return LIA_ERR_SIZE;
+    const long long blocks = ((long long)n_tokens * hidden + 255) / 256;
+    const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
+    if (bias_dtype == LIA_BF16)
+        return lia_launch(stream_sum_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, x, x0, (const __nv_bfloat16*)bias, n_tokens, hidden);
+    if (bias_dtype == LIA_F32)
+        return lia_launch(stream_sum_kernel<float>, grid, dim3(256), 0, stream, x, x0, (const float*)bias, n_tokens, hidden);
     return LIA_ERR_DTYPE;
 }

@@ -52,7 +52,8 @@ class _Signatures:
     lia_wait_probe = [c_int, c_void_p, c_void_p, c_void_p]
     lia_attention_decode = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                            c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p]
+                            c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+                            c_void_p]
     lia_attention_decode_cluster_splits = [c_int, c_int, c_int, c_int, c_int]
     lia_attention_decode_ctas_per_sm = [c_int, c_int, c_int]
     lia_gemm_tc = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -70,7 +71,7 @@ class _Signatures:
                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
     lia_attention_prefill_tc = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                                 c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int,
-                                c_float, c_void_p, c_void_p]
+                                c_void_p, c_float, c_void_p, c_void_p]
     lia_attention_prefill_tc_tokens_per_tile = [c_int, c_int, c_int]
     lia_select_tokens = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                          ctypes.c_longlong, c_void_p]
@@ -88,6 +89,18 @@ class _Signatures:
                       c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]
     lia_embedding_positions = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                c_int, c_float, c_void_p, c_void_p]
+    lia_stream_sum = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
+    lia_mlstm = [c_void_p, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_float, c_void_p,
+                 ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int,
+                 c_void_p, ctypes.c_longlong, c_void_p]
+    lia_mlstm_tc = [c_void_p, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_float, c_void_p,
+                    ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
+                    c_int, c_void_p, ctypes.c_longlong, c_void_p]
+    lia_mlstm_tc_chunks = [c_int, c_int]
+    lia_mlstm_tc_pieces = [c_int, c_int]
+    lia_mlstm_single = [c_void_p, c_int, ctypes.c_longlong, c_int, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_float,
+                        c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int,
+                        c_int, c_int, c_void_p]
     lia_reinject_input = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]
     lia_sigmoid_attention_tc_tokens_per_tile = [c_int, c_int, c_int]
     lia_sigmoid_attention_tc = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
@@ -102,10 +115,10 @@ class _Signatures:
     lia_attention_general = [c_void_p, ctypes.c_longlong, ctypes.c_longlong, c_void_p, ctypes.c_longlong, ctypes.c_longlong,
                              c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                              c_int, c_void_p, c_void_p, ctypes.c_longlong, ctypes.c_longlong, c_int, c_int, c_int, c_int,
-                             c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p]
+                             c_int, c_float, c_float, c_int, c_void_p, c_int, c_void_p, c_void_p]
     lia_qkv_prepare = [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float,
                        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
     lia_latent_prepare = [c_void_p, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_void_p, c_float, c_void_p, c_int,
                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                           c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
@@ -131,7 +144,7 @@ class _Signatures:
     lia_gate_rows = [c_void_p, c_int, ctypes.c_longlong, c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p]
     lia_moe_tile_rows = []
     lia_moe_route = [c_void_p, c_int, ctypes.c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                     c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
+                     c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
     lia_moe_plan = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]
     lia_moe_gather = [c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]
     lia_moe_gemm = [c_int, c_void_p, c_int, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong,
@@ -564,13 +577,19 @@ def attention_generic(q, k_pages, v_pages, positions, slots, block_table, out, n
                "attention_generic")
 
 
+def _check_sinks(sinks, nq: int):
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nq):
+        raise KernelError("attention: sinks are one 32-bit number a query head")
+
+
 DECODE_HEAD_DIMS = (32, 64, 128)       # head sizes the tensor-core attention kernels are built for (keys' and values' equal)
 DECODE_HEAD_PAIRS = tuple((d, d) for d in DECODE_HEAD_DIMS) + ((64, 128), (128, 64), (32, 64), (64, 32))    # (keys', values')
 
 
 def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, out, partial, nq, nkv, d, window,
                      scale, split_len, n_splits, counters=None, qkv=None, inv_freq=None, rotary_dim=0, write_kv=True,
-                     error_flag=None, label=None, work_bytes=0, cluster=False, all_new=False, sink=False, softcap=None):
+                     error_flag=None, label=None, work_bytes=0, cluster=False, all_new=False, sink=False, softcap=None,
+                     sinks=None):
     """Split-key decode attention (bfloat16) for the single-token rows of the batch; see
     csrc/attention_decode.cu.  `partial` is 32-bit scratch for the ranges' partial results.
     `split_len` 0: every row cuts its own visible span into `n_splits` ranges.  `counters` (int32, at
@@ -584,9 +603,10 @@ def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, o
     `partial` nor `counters` is used.  `all_new`: the rows may be tokens of this step's prompt portions, so any of
     their keys may have been written by the kernels ahead (otherwise only a row's own key is taken to be of this step,
     and the kernel fetches older tiles before it waits for those kernels).  `sink`: one is added to the softmax's denominator
-    (a key of score 0 without a value), once, where a token's ranges meet.  `softcap`: the scores pass
-    cap * tanh(score / cap) ahead of the softmax (the hardware's tanh approximation)."""
-    _cuda(q, k_pages, v_pages, rows, positions, slots, block_table, out, partial, counters, qkv, inv_freq, error_flag)
+    (a key of score 0 without a value), once, where a token's ranges meet; `sinks` (32-bit [nq]): exp(sinks[h]) instead, of
+    head h.  `softcap`: the scores pass cap * tanh(score / cap) ahead of the softmax."""
+    _cuda(q, k_pages, v_pages, rows, positions, slots, block_table, out, partial, counters, qkv, inv_freq, error_flag, sinks)
+    _check_sinks(sinks, nq)
     if qkv is not None:
         if qkv.dtype != torch.float32 or qkv.shape[1] != (nq + 2 * nkv) * d:
             raise KernelError("attention_decode: qkv must be 32-bit q|k|v rows")
@@ -605,7 +625,7 @@ def attention_decode(q, k_pages, v_pages, rows, positions, slots, block_table, o
                                           0 if partial is None else partial.numel(), _p(counters), q.shape[0], nq, nkv, d, dv,
                                           k_pages.shape[1], int(window or 0), scale, split_len, n_splits, _p(qkv), _p(inv_freq),
                                           int(rotary_dim), 1 if write_kv else 0, k_pages.shape[0], 1 if cluster else 0, 1 if all_new else 0,
-                                          1 if sink else 0, float(softcap or 0.0), _p(error_flag),
+                                          1 if sink else 0, _p(sinks), float(softcap or 0.0), _p(error_flag),
                                           _stream()),
                "attention_decode")
 
@@ -648,12 +668,13 @@ def attention_prefill_tc_tokens_per_tile(group: int, d: int, dv: int = None) -> 
 
 def attention_prefill_tc(q, k_pages, v_pages, segments, n_segments, n_tiles, slots, block_table, out, nq, nkv, d,
                          window, scale, error_flag=None, label=None, work_flops=0, splits=1, partial=None, sink=False,
-                         softcap=None):
+                         softcap=None, sinks=None):
     """Prompt-portion attention on the tcgen05 tensor cores (bfloat16, head size 64 or 128, heads per kv head a
     divisor of 128); see csrc/attention_prefill_tc.cu.  Arguments as `attention_prefill`.  `splits` > 1 cuts every
     CTA's keys into that many ranges that run side by side and are merged by a second kernel; `partial` is their
-    32-bit scratch, `attention_prefill_tc_partial_floats` words long."""
-    _cuda(q, k_pages, v_pages, segments, slots, block_table, out, error_flag, partial)
+    32-bit scratch, `attention_prefill_tc_partial_floats` words long.  `sink`, `sinks`, `softcap`: as for `attention_decode`."""
+    _cuda(q, k_pages, v_pages, segments, slots, block_table, out, error_flag, partial, sinks)
+    _check_sinks(sinks, nq)
     if not (q.dtype == k_pages.dtype == v_pages.dtype == out.dtype == torch.bfloat16):
         raise KernelError("attention_prefill_tc is a bfloat16 kernel")
     splits, dv = int(splits), v_pages.shape[-1]
@@ -666,7 +687,7 @@ def attention_prefill_tc(q, k_pages, v_pages, segments, n_segments, n_tiles, slo
         _check(lib().lia_attention_prefill_tc(_p(q), _p(k_pages), _p(v_pages), _p(segments), n_segments, n_tiles,
                                               _p(slots), _p(block_table), block_table.shape[1], _p(out), nq, nkv, d, dv,
                                               k_pages.shape[1], int(window or 0), scale, k_pages.shape[0], splits,
-                                              _p(partial) if splits > 1 else None, q.shape[0], 1 if sink else 0,
+                                              _p(partial) if splits > 1 else None, q.shape[0], 1 if sink else 0, _p(sinks),
                                               float(softcap or 0.0), _p(error_flag), _stream()),
                "attention_prefill_tc")
 
@@ -750,6 +771,18 @@ def embedding_positions(tokens, positions, table, position_table, out, scale: fl
                                              dtype_code(table.dtype), _p(out), _p(copy), n, hidden, table.shape[0],
                                              position_table.shape[0], scale, _p(error_flag), _stream()),
                "embedding_positions")
+
+
+def stream_sum(x, x0=None, bias=None):
+    """x[t] += x0[t] + bias, in place (32-bit rows; either may be absent); see csrc/residual_ops.cu."""
+    _cuda(x, x0, bias)
+    _f32(x, x0)
+    n, hidden = x.shape
+    if (x0 is not None and x0.shape != x.shape) or (bias is not None and bias.numel() != hidden):
+        raise KernelError("stream_sum: rows of one shape, a bias of their width")
+    with _timed("stream_sum", nbytes=n * hidden * (12 if x0 is not None else 8)):
+        _check(lib().lia_stream_sum(_p(x), _p(x0), _p(bias), dtype_code(bias.dtype) if bias is not None else F32, n, hidden,
+                                    _stream()), "stream_sum")
 
 
 def reinject_input(x, x0, bias, side_by_side):
@@ -975,13 +1008,15 @@ def activation_rows(source, out, act: int = ACT_NONE, gated: bool = False, const
 
 def attention_general(q1, q1_strides, q2, q2_strides, k1_pages, k2_pages, v_pages, v_stride, dv, positions, slots,
                       block_table, out, out_strides, n_tokens, nq, nkv, window, scale, sink=False, rows=None,
-                      error_flag=None, label=None, work_bytes=0, softcap=None):
+                      error_flag=None, label=None, work_bytes=0, softcap=None, sinks=None):
     """Softmax attention whose keys come in up to two parts (k1 [pages, page, nkv, dk1] with q1, k2 [.., dk2] with q2; k2
     and q2 may be None) and whose values are the first `dv` of every `v_stride` elements of `v_pages`; q1, q2 and out
-    are addressed by (token stride, head stride) in elements; `sink` adds one to the denominator; `softcap`: the scores
+    are addressed by (token stride, head stride) in elements; `sink` adds one to the denominator, `sinks`
+    (32-bit [nq]) exp(sinks[h]) to head h's; `softcap`: the scores
     pass cap * tanh(score / cap) ahead of the softmax; see
     csrc/attention_generic.cu.  For every token of the batch, or for the batch indices `rows`."""
-    _cuda(k1_pages, k2_pages, v_pages, positions, slots, block_table, rows, error_flag)
+    _cuda(k1_pages, k2_pages, v_pages, positions, slots, block_table, rows, error_flag, sinks)
+    _check_sinks(sinks, nq)
     for t in (q1, q2, out):
         if t is not None and not t.is_cuda:
             raise KernelError("kernels need CUDA tensors")
@@ -997,13 +1032,15 @@ def attention_general(q1, q1_strides, q2, q2_strides, k1_pages, k2_pages, v_page
                                            _p(k2_pages), dk2, _p(v_pages), int(v_stride), int(dv), dtype_code(q1.dtype),
                                            _p(positions), _p(slots), _p(block_table), block_table.shape[1], _p(rows),
                                            _p(out), out_strides[0], out_strides[1], n, nq, nkv, k1_pages.shape[1],
-                                           int(window or 0), scale, float(softcap or 0.0), 1 if sink else 0, k1_pages.shape[0], _p(error_flag),
+                                           int(window or 0), scale, float(softcap or 0.0), 1 if sink else 0, _p(sinks), k1_pages.shape[0], _p(error_flag),
                                            _stream()), "attention_general")
 
 
 def qkv_prepare(rows, bias, q_norm, k_norm, eps, freq, rot_dims, vmix_mode, vmix_lambda, v_first, positions, slots,
-                block_table, q_out, k_pages, v_pages, nq, nkv, d, dv, write_kv=True, error_flag=None, norm_whole=False):
-    """Bias, per-head RMS norm of q and k, rotate-half encoding, value mixing and the append to the pages for the
+                block_table, q_out, k_pages, v_pages, nq, nkv, d, dv, write_kv=True, error_flag=None, norm_whole=False,
+                pairs=False, norm_behind=False):
+    """Bias, per-head RMS norm of q and k, rotary encoding (rotate-half, or `pairs`: element 2i with 2i + 1), with
+    `norm_behind` an RMS norm per head without a weight behind it, value mixing and the append to the pages for the
     32-bit rows [q | k | v] of a product; see csrc/qk_prepare.cu.  `norm_whole`: one RMS norm over all of q's elements and
     one over all of k's instead (weights [nq d] and [nkv d])."""
     _cuda(bias, q_norm, k_norm, freq, v_first, positions, slots, block_table, q_out, k_pages, v_pages, error_flag)
@@ -1018,7 +1055,8 @@ def qkv_prepare(rows, bias, q_norm, k_norm, eps, freq, rot_dims, vmix_mode, vmix
                                      int(rot_dims), int(vmix_mode), float(vmix_lambda), _p(v_first), _p(positions),
                                      _p(slots), _p(block_table), block_table.shape[1], _p(q_out), _p(k_pages), _p(v_pages),
                                      dtype_code(q_out.dtype), rows.shape[0], nq, nkv, d, dv, k_pages.shape[1],
-                                     k_pages.shape[0], 1 if write_kv else 0, 1 if norm_whole else 0, _p(error_flag), _stream()),
+                                     k_pages.shape[0], 1 if write_kv else 0, 1 if norm_whole else 0, 1 if pairs else 0,
+                                     1 if norm_behind else 0, _p(error_flag), _stream()),
                "qkv_prepare")
 
 
@@ -1286,11 +1324,12 @@ def moe_grouped_accepts(x, w_gate_up, w_down) -> bool:
 
 
 def moe_route(x, router, top: int, scale: float, ids, weights, shared_gate=None, correction=None, groups: int = 0,
-              keep: int = 0, renormalise: bool = False):
+              keep: int = 0, renormalise: bool = False, sigmoid: bool = False, two_best: bool = False):
     """Router scores in 32-bit, the `top` largest chosen: ids, weights [n, top]; with one more row in `router` than
     outputs, shared_gate [n] = the logistic function of that row's product.  `correction` [outputs] is added to the
     scores for the choice only; `groups`/`keep`: only outputs of the best `keep` of `groups` equal groups can be chosen;
-    `renormalise`: the weights are divided by their sum."""
+    `renormalise`: the weights are divided by their sum; `sigmoid`: scores are the logistic function of each product (else
+    the softmax over all); `two_best`: a group's score is the sum of its two largest (else its largest)."""
     _cuda(x, router, ids, weights, shared_gate, correction)
     _f32(router, weights, shared_gate, correction)
     n, hidden = x.shape
@@ -1301,7 +1340,7 @@ def moe_route(x, router, top: int, scale: float, ids, weights, shared_gate=None,
     with _timed("moe_route"):
         _check(lib().lia_moe_route(_p(x), dtype_code(x.dtype), x.stride(0), _p(router), n, hidden, experts, int(top),
                                    float(scale), extra, _p(correction), int(groups), int(keep), 1 if renormalise else 0,
-                                   _p(ids), _p(weights), _p(shared_gate), _stream()), "moe_route")
+                                   1 if sigmoid else 0, 1 if two_best else 0, _p(ids), _p(weights), _p(shared_gate), _stream()), "moe_route")
 
 
 def moe_plan(ids, experts: int, offsets, order, inverse, tiles, n_tiles, tile_rows: int = 0, pad: bool = False):
@@ -1368,7 +1407,7 @@ def gemm_tc_grouped(mode, a, w, out, tile_rows: int, tiles, n_tiles, max_tiles: 
 
 
 def moe_combine(residual, y, inverse, weights, shared_y, shared_gate, top: int, alpha: float, store: bool, x=None):
-    """residual (+)= alpha * (sum_c weights[t, c] y[inverse[t, c]] + shared_gate[t] shared_y[t]); a choice without a row
+    """residual (+)= alpha * (sum_c weights[t, c] y[inverse[t, c]] + shared_gate[t] shared_y[t]), shared_gate None: ones; a choice without a row
     (inverse < 0: an identity output) adds weights[t, c] x[t], x the tokens' inputs [n, hidden]."""
     _cuda(residual, y, inverse, weights, shared_y, shared_gate, x)
     _f32(residual, y, weights, shared_y, shared_gate)
@@ -1683,3 +1722,70 @@ def gated_group_norm(y, z, weight, slots, out, groups: int, eps: float):
     with _timed("gated_group_norm", nbytes=n * width * (8 + out.element_size())):
         _check(lib().lia_gated_group_norm(_p(y), _p(z), z.stride(0), _p(weight), _p(slots), _p(out), dtype_code(out.dtype), n,
                                           int(groups), width // groups, float(eps), _stream()), "gated_group_norm")
+
+
+# ---- a matrix memory with exponential gates per head (mLSTM): csrc/mlstm.cu, csrc/mlstm_tc.cu ----
+MLSTM_MAX_HEAD = 512
+
+
+def mlstm_scratch_floats(chunks: int, heads: int, d: int, dv: int) -> int:
+    return chunks * heads * (d * dv + d + 3)
+
+
+def mlstm_tc_pieces(d: int, dv: int) -> int:
+    """How many pieces the tensor-core kernels cut a head's values into (bfloat16 q, k and v); 0: they do not take the sizes."""
+    return int(lib().lia_mlstm_tc_pieces(int(d), int(dv)))
+
+
+def mlstm_chunks(portion_tokens: int, n_segments: int, tensor_cores: bool) -> int:
+    """Most chunks that a step's portions are cut into."""
+    fn = lib().lia_mlstm_tc_chunks if tensor_cores else lib().lia_retention_chunks
+    return int(fn(int(portion_tokens), int(n_segments)))
+
+
+def _check_mlstm(qkv, gates, i_bias, f_bias, state, norm_weight, out, heads, d, dv):
+    n = out.shape[0]
+    if qkv.stride(1) != 1 or gates.stride(1) != 1 or qkv.shape[0] != n or gates.shape[0] != n or \
+            qkv.shape[1] != heads * (2 * d + dv) or gates.shape[1] < heads * (dv + 2) or out.shape[1] != heads * dv or \
+            i_bias.numel() != heads or f_bias.numel() != heads or norm_weight.numel() != heads * dv or \
+            state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < heads * (d * dv + d + 1):
+        raise KernelError("mlstm: shapes do not agree")
+    _cuda(i_bias, f_bias, norm_weight, out)
+    _f32(gates, i_bias, f_bias, state, norm_weight)
+
+
+def mlstm(qkv, gates, i_bias, f_bias, cap: float, state, segments, n_segments: int, max_chunks: int, slots, norm_weight, eps: float,
+          out, heads: int, d: int, dv: int, scratch, y=None):
+    """The matrix memory along the step's portions: qkv [n, heads (2 d + dv)] = [q | k | v], 32-bit (on the 32-bit pipes,
+    csrc/mlstm.cu) or bfloat16 (on the tensor cores where `mlstm_tc_pieces`, csrc/mlstm_tc.cu; `y` [n, heads dv] 32-bit where
+    that is more than one); gates [n, >= heads (dv + 2)] = [output gate | i | f] 32-bit; state [slots, >= heads (d dv + d + 1)]
+    32-bit; out [n, heads dv] = the normed and gated heads."""
+    _check_mlstm(qkv, gates, i_bias, f_bias, state, norm_weight, out, heads, d, dv)
+    _cuda(segments, slots, scratch, y)
+    _f32(scratch, y)
+    n = out.shape[0]
+    tensor_cores = qkv.dtype == torch.bfloat16
+    if (tensor_cores and out.dtype != torch.bfloat16) or (y is not None and tuple(y.shape) != tuple(out.shape)):
+        raise KernelError("mlstm: bfloat16 rows give bfloat16 rows; y has the output's shape")
+    nbytes = n * heads * ((2 * d + dv) * qkv.element_size() + dv * (4 + out.element_size()))
+    args = (_p(qkv), qkv.stride(0), _p(gates), gates.stride(0), _p(i_bias), _p(f_bias), float(cap), _p(state), state.stride(0),
+            _p(segments), int(n_segments), int(max_chunks), _p(slots), _p(norm_weight), float(eps), _p(out))
+    with _timed("mlstm_tc" if tensor_cores else "mlstm", nbytes=nbytes, flops=4 * n * heads * d * dv):
+        if tensor_cores:
+            _check(lib().lia_mlstm_tc(*args, _p(y), heads, d, dv, _p(scratch), scratch.numel(), _stream()), "mlstm_tc")
+        else:
+            _check(lib().lia_mlstm(*args, dtype_code(out.dtype), heads, d, dv, _p(scratch), scratch.numel(), _stream()), "mlstm")
+
+
+def mlstm_single(qkv, gates, i_bias, f_bias, cap: float, state, single_rows, slots, norm_weight, eps: float, out, heads: int, d: int,
+                 dv: int, round16: bool = False, wanted_ctas: int = 0):
+    """The same for the step's single tokens, state in place; `round16`: 32-bit q, k and v are rounded to bfloat16 as they are
+    read (what the portions' kernels are given); `wanted_ctas`: how many CTAs the device should have before heads stay whole."""
+    _check_mlstm(qkv, gates, i_bias, f_bias, state, norm_weight, out, heads, d, dv)
+    _cuda(single_rows, slots)
+    n_single = single_rows.numel()
+    with _timed("mlstm_single", nbytes=n_single * heads * 8 * (d * dv + d)):
+        _check(lib().lia_mlstm_single(_p(qkv), dtype_code(qkv.dtype), qkv.stride(0), 1 if round16 else 0, _p(gates), gates.stride(0),
+                                      _p(i_bias), _p(f_bias), float(cap), _p(state), state.stride(0), _p(single_rows), n_single,
+                                      _p(slots), _p(norm_weight), float(eps), _p(out), dtype_code(out.dtype), heads, d, dv,
+                                      int(wanted_ctas), _stream()), "mlstm_single")

@@ -23,6 +23,10 @@ Options (each absent by default):
     use the scores without it);
   * `groups` {"count", "keep"}: the router's outputs form `count` equal groups of neighbours, a group's score is its
     largest choice score, and only outputs of the `keep` best groups can be chosen;
+  * `scores` "sigmoid": s = sigmoid(z), each output's own (default "softmax");
+  * `group_score` "two_best": a group's score is the sum of its two largest choice scores (of its one, where a group is one
+    output);
+  * `shared_gated` False: the shared expert has no gate, shared(x) is added as it is;
   * `renormalise`: weight_e = s_e / (sum of the chosen s + 1e-20) * router_scale.
 
 Parameters: hidden, experts, top, intermediate, router_scale, shared ({"intermediate": n} or None), and optionally
@@ -66,6 +70,8 @@ class ExpertMixture(FeedForward):
         if int(params.get("identity") or 0) < 0 or outputs > ops.MOE_MAX_EXPERTS or top > outputs:
             raise ValueError(f"expert mixture: identity outputs are not negative, the router has at most {ops.MOE_MAX_EXPERTS} "
                              "outputs and no more are chosen than there are")
+        if params.get("scores", "softmax") not in ("softmax", "sigmoid") or params.get("group_score", "best") not in ("best", "two_best"):
+            raise ValueError("expert mixture: scores is 'softmax' or 'sigmoid', group_score 'best' or 'two_best'")
         groups = params.get("groups")
         if groups:
             count, keep = int(groups["count"]), int(groups["keep"])
@@ -90,7 +96,9 @@ class ExpertMixture(FeedForward):
         if params.get("shared"):
             ffs, p = int(params["shared"]["intermediate"]), prefix + n["shared"]
             specs += ([TensorSpec(p + n["gate"], (ffs, h))] if gated else []) + \
-                [TensorSpec(p + n["up"], (ffs, h)), TensorSpec(p + n["down"], (h, ffs)), TensorSpec(prefix + n["shared_gate"], (1, h))]
+                [TensorSpec(p + n["up"], (ffs, h)), TensorSpec(p + n["down"], (h, ffs))]
+            if params.get("shared_gated", True):
+                specs.append(TensorSpec(prefix + n["shared_gate"], (1, h)))
         return specs
 
     def __init__(self, params, tensors, prefix, runtime):
@@ -101,6 +109,7 @@ class ExpertMixture(FeedForward):
         self.gated = params.get("expert_form", "gated_silu") == "gated_silu"
         self.identity = int(params.get("identity") or 0)
         self.renormalise = bool(params.get("renormalise"))
+        self.sigmoid, self.two_best = params.get("scores") == "sigmoid", params.get("group_score") == "two_best"
         groups = params.get("groups")
         self.groups, self.keep = (int(groups["count"]), int(groups["keep"])) if groups else (0, 0)
         n = self._names(params, prefix)
@@ -110,9 +119,11 @@ class ExpertMixture(FeedForward):
         self.w_down = prepare_weight(torch.stack([expert(e, "down") for e in range(self.experts)]), runtime)   # [E, hidden, ff]
         router = [tensors[prefix + n["router"]]]
         self.shared = bool(params.get("shared"))
+        self.shared_gated = bool(params.get("shared_gated", True))
         if self.shared:
             self.ffs, p = int(params["shared"]["intermediate"]), prefix + n["shared"]
-            router.append(tensors[prefix + n["shared_gate"]].view(1, self.hidden))        # the gate's row rides on the router's product
+            if self.shared_gated:
+                router.append(tensors[prefix + n["shared_gate"]].view(1, self.hidden))    # the gate's row rides on the router's product
             first = torch.cat([tensors[p + n["gate"]], tensors[p + n["up"]]], dim=0) if self.gated else tensors[p + n["up"]]
             self.w_shared_gate_up = prepare_weight(first, runtime)
             self.w_shared_down = prepare_weight(tensors[p + n["down"]], runtime)
@@ -127,9 +138,9 @@ class ExpertMixture(FeedForward):
         scratch = ctx.runtime.scratch
         ids = scratch("moe.ids", pairs, torch.int32).view(n, top)
         weights = scratch("moe.weights", pairs, torch.float32).view(n, top)
-        shared_gate = scratch("moe.shared_gate", n, torch.float32) if self.shared else None
+        shared_gate = scratch("moe.shared_gate", n, torch.float32) if self.shared and self.shared_gated else None
         ops.moe_route(x, self.router, top, self.router_scale, ids, weights, shared_gate, correction=self.correction,
-                      groups=self.groups, keep=self.keep, renormalise=self.renormalise)
+                      groups=self.groups, keep=self.keep, renormalise=self.renormalise, sigmoid=self.sigmoid, two_best=self.two_best)
         if self.grouped is None:
             self.grouped = ops.moe_grouped_accepts(x, self.w_gate_up, self.w_down)
         if self.grouped:

@@ -3,15 +3,16 @@
 `sink_attention`: grouped-query attention, q = Wq x + bq, k = Wk x + bk, v = Wv x + bv (biases optional), with
   * an RMS norm of every q head and every k head over the head's elements, with one weight of the head's size for all
     q heads and one for all k heads (optional; `qk_norm` "whole": one RMS norm over all of q's elements at once and one
-    over all of k's, with weights of those sizes), ahead of the rotation;
-  * rotate-half encoding over the first `rot.dims` elements of a head, frequencies plain or scaled by wavelength bands
-    (`rotary.band_scaled_frequencies`);
+    over all of k's, with weights of those sizes), ahead of the rotation; `qk_norm` "behind": each head over its root mean
+    square without a weight, behind the rotation;
+  * rotary encoding over the first `rot.dims` elements of a head, in halves or (`rot_pairs`) element 2i with 2i + 1,
+    frequencies plain or scaled by wavelength bands (`rotary.band_scaled_frequencies`);
   * values of a head size of their own;
   * value mixing (optional): the first such layer of a model leaves its values of the step's tokens in a step buffer
     (`value_mix` "source"), later ones ("mixed") use v <- (1 - lambda) v + lambda v_first, lambda a stored scalar; the
     mixed values are what the pages hold;
   * a sink (optional): one is added to the softmax's denominator, p_j = exp(s_j) / (1 + sum exp(s_j)), the weight of
-    a key of score 0 that has no value;
+    a key of score 0 that has no value; `sink` "learned": exp of a stored number a query head in place of the one;
   * a cap on the scores (optional, `softcap`): s <- cap * tanh(s / cap) ahead of the softmax;
   * all keys j <= i, or the last `window` of them;
   * an output gate (optional, `gate` "sigmoid"): the heads side by side are multiplied by sigmoid(W_g x) ahead of the output
@@ -75,7 +76,7 @@ class SinkAttention(Mixer):
     can_store = True
     projects_input = True
     NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "o_bias": "o.b",
-             "q_norm": "q.norm", "k_norm": "k.norm", "mix": "vmix", "gate": "g"}
+             "q_norm": "q.norm", "k_norm": "k.norm", "mix": "vmix", "gate": "g", "sink": "sink"}
 
     @staticmethod
     def _names(params, prefix):
@@ -95,12 +96,13 @@ class SinkAttention(Mixer):
             raise ValueError("attention: window must be positive or None")
         if params.get("softcap") is not None and not float(params["softcap"]) > 0:
             raise ValueError("attention: softcap must be positive or None")
-        if params.get("biases") not in (None, False, True, "qkv") or params.get("qk_norm") not in (None, False, True, "whole"):
-            raise ValueError("attention: biases is absent, True or 'qkv'; qk_norm is absent, True or 'whole'")
+        if params.get("biases") not in (None, False, True, "qkv") or params.get("qk_norm") not in (None, False, True, "whole",
+                                                                                                            "behind"):
+            raise ValueError("attention: biases is absent, True or 'qkv'; qk_norm is absent, True, 'whole' or 'behind'")
+        if params.get("sink") not in (None, False, True, "learned"):
+            raise ValueError("attention: sink is absent, True or 'learned'")
         if params.get("gate") not in (None, "sigmoid"):
             raise ValueError("attention: gate is None or 'sigmoid'")
-        if params.get("softcap") is not None and params.get("sink"):
-            raise ValueError("attention: a sink and a cap on the scores together are not built")
 
     @staticmethod
     def tensor_specs(params, prefix):
@@ -117,8 +119,10 @@ class SinkAttention(Mixer):
                 specs.append(TensorSpec(n["o_bias"], (h,)))
         if params.get("qk_norm") == "whole":
             specs += [TensorSpec(n["q_norm"], (nq * d,), kind="norm"), TensorSpec(n["k_norm"], (nkv * d,), kind="norm")]
-        elif params.get("qk_norm"):
+        elif params.get("qk_norm") and params["qk_norm"] != "behind":
             specs += [TensorSpec(n["q_norm"], (d,), kind="norm"), TensorSpec(n["k_norm"], (d,), kind="norm")]
+        if params.get("sink") == "learned":
+            specs.append(TensorSpec(n["sink"], (nq,)))
         if params.get("value_mix"):
             specs.append(TensorSpec(n["mix"], ()))          # the first such layer stores one too and does not use it
         return specs
@@ -160,18 +164,21 @@ class SinkAttention(Mixer):
             self.output_bias = f32(tensors[n["o_bias"]]) if params["biases"] != "qkv" else None
         self.norm_whole = params.get("qk_norm") == "whole"
         self.softcap = None if params.get("softcap") is None else float(params["softcap"])
-        self.q_norm = f32(tensors[n["q_norm"]]) if params.get("qk_norm") else None
-        self.k_norm = f32(tensors[n["k_norm"]]) if params.get("qk_norm") else None
+        self.norm_behind = params.get("qk_norm") == "behind"
+        weighted = params.get("qk_norm") and not self.norm_behind
+        self.q_norm = f32(tensors[n["q_norm"]]) if weighted else None
+        self.k_norm = f32(tensors[n["k_norm"]]) if weighted else None
+        self.sinks = f32(tensors[n["sink"]]) if params.get("sink") == "learned" else None
+        self.pairs = bool(params.get("rot_pairs"))
         self.rot_dims, self.freq = _frequencies(params.get("rot"), device)
         self.mix_mode = {None: 0, "source": 1, "mixed": 2}[params.get("value_mix")]
         self.mix_lambda = float(tensors[n["mix"]].to(torch.float32)) if self.mix_mode == 2 else 0.0
         # bfloat16 with keys and values of head sizes that the tensor-core kernels take: those kernels; else the kernel
         # for every size
         self.paged = None
-        if runtime.compute_dtype == torch.bfloat16 and PagedAttention.takes(self.d, self.dv, self.nq // self.nkv) and \
-                not (self.softcap and self.d != self.dv):
+        if runtime.compute_dtype == torch.bfloat16 and PagedAttention.takes(self.d, self.dv, self.nq // self.nkv):
             self.paged = PagedAttention(runtime.compute_dtype, self.nq, self.nkv, self.d, self.window, self.scale, sink=self.sink,
-                                        softcap=self.softcap, v_head_dim=self.dv)
+                                        softcap=self.softcap, v_head_dim=self.dv, sinks=self.sinks)
 
     def graph_key(self, ctx) -> tuple:
         return self.paged.graph_key(ctx) if self.paged is not None else ()
@@ -187,14 +194,15 @@ class SinkAttention(Mixer):
         v_first = ctx.buffer("sinkattn.v_first", (n, nkv * dv), torch.float32) if self.mix_mode else None
         ops.qkv_prepare(projected, self.bias_in, self.q_norm, self.k_norm, self.eps, self.freq, self.rot_dims,
                         self.mix_mode, self.mix_lambda, v_first, ctx.positions, ctx.slots, kv.block_table, q, kv.k_pages,
-                        kv.v_pages, nq, nkv, d, dv, write_kv=kv.writes, error_flag=flag, norm_whole=self.norm_whole)
+                        kv.v_pages, nq, nkv, d, dv, write_kv=kv.writes, error_flag=flag, norm_whole=self.norm_whole,
+                        pairs=self.pairs, norm_behind=self.norm_behind)
         o = ctx.buffer("sinkattn.o", (n, nq * dv), rt.compute_dtype)
         if self.paged is not None:
             self.paged.forward(ctx, q, kv, o)
         else:
             ops.attention_general(q, (nq * d, d), None, None, kv.k_pages, None, kv.v_pages, dv, dv, ctx.positions, ctx.slots,
                                   kv.block_table, o, (nq * dv, dv), n, nq, nkv, self.window, self.scale, sink=self.sink,
-                                  error_flag=flag, softcap=self.softcap)
+                                  error_flag=flag, softcap=self.softcap, sinks=self.sinks)
         if self.gate_at is not None:
             ops.gate_rows(o, projected[:, self.gate_at:self.gate_at + nq * dv], ops.GATE_SIGMOID)
         linear(rt, STORE if store else ACCUM, o, self.w_o, residual, scale, error_flag=flag, name="o")
