@@ -624,6 +624,34 @@ def foduzen_workload(steps, warmup) -> int:
                          FODUZEN_SIZES, foduzen_pair, steps, warmup)
 
 
+# The Botuvik decoder beside the Pilutar, Foduzen, Vatunex and Llama decoders at equal sizes (--workload botuvik): four layer runs
+# each.  Botuvik: the matrix memory with a dense squared-ReLU feed-forward (first and last), between them one layer that runs
+# twice, capped attention over all keys with a learned sink a head and a mixture of eight gated experts in four groups of
+# which three stay (two chosen, one shared expert); a token's active expert weights equal the dense layer's.  Pilutar (capped
+# attention, a linear recurrence, grouped experts), Foduzen (a recurrence on the tensor cores) and Vatunex (norms on both sides
+# of a sublayer, a sink) are the closest models, each in its own workload's form.
+def botuvik_pair(size: dict):
+    from lia_rs_b200.config import BotuvikConfig
+    dense = {"kind": "dense", "ff": size["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": size["expert_ff"]}, "shared": {"ff": size["shared_ff"]},
+           "router": {"experts": size["experts"], "top": size["top"], "groups": {"count": 4, "keep": 3}}}
+    memory = {"type": "mlstm", "mlp": dense, "mixer": {"heads": size["heads"], "dim": size["dim"] // 2, "vdim": size["dim"],
+                                                       "gate_cap": 15.0}}
+    attention = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": size["heads"], "kv_heads": size["kv_heads"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5,
+        "softcap": 25.0, "rot": {"base": 50000.0, "dims": size["dim"]}}}
+    botuvik = BotuvikConfig.from_dict({
+        "architecture": "Botuvik", "vocab": 8192, "width": size["width"], "norm": {"eps": 1e-5},
+        "layers": [memory, attention, memory], "loop": {"start": 1, "stop": 2, "times": 2}})
+    others = foduzen_pair(size)
+    return {"botuvik": botuvik, **{name: others[name] for name in ("pilutar", "foduzen", "vatunex", "llama")}}
+
+
+def botuvik_workload(steps, warmup) -> int:
+    return pair_workload("botuvik", "Botuvik beside the Pilutar, Foduzen, Vatunex and Llama decoders at equal sizes, four layers, bf16",
+                         FODUZEN_SIZES, botuvik_pair, steps, warmup)
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -634,7 +662,7 @@ def main() -> int:
                         help="run fewer layers than the configuration's 40 (both numbers are reported)")
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--no-points", action="store_true", help="skip batch 1 and batch 64")
-    parser.add_argument("--workload", default=None, choices=["8b-decode", "8b-prefill", "0.5b-mixed", "nafevik", "vatunex", "zipelix", "pilutar", "foduzen"],
+    parser.add_argument("--workload", default=None, choices=["8b-decode", "8b-prefill", "0.5b-mixed", "nafevik", "vatunex", "zipelix", "pilutar", "foduzen", "botuvik"],
                         help="one of the family's other sizes on the workload it is quoted on (prints its own line)")
     parser.add_argument("--device-trace", action="store_true",
                         help="with --workload 0.5b-mixed: one more pass under a trace of the device's kernels; adds "
@@ -663,6 +691,8 @@ def main() -> int:
         return pilutar_workload(args.steps, args.warmup)
     if args.workload == "foduzen":
         return foduzen_workload(args.steps, args.warmup)
+    if args.workload == "botuvik":
+        return botuvik_workload(args.steps, args.warmup)
     if args.workload:
         return other_workload(args.workload, args.steps, args.warmup, trace=args.device_trace)
 

@@ -67,16 +67,14 @@ __device__ __forceinline__ int range_length(const Params& p, int span) {
     return (per + TILE_KEYS - 1) / TILE_KEYS * TILE_KEYS;
 }
 
-// tanh by the hardware's approximation (relative error about 2^-11, below the rounding of the 16-bit probabilities)
-__device__ __forceinline__ float tanh_approx(float x) {
-    float y;
-    asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 __device__ __forceinline__ float ex2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+// tanh as 1 - 2 / (1 + exp(2x)): absolute error about 2^-22
+__device__ __forceinline__ float tanh_by_exponential(float x) {
+    return 1.0f - __fdividef(2.0f, 1.0f + ex2_approx(x * 2.8853900817779268f));
 }
 // 2^n for a whole number n <= 0 (or -infinity), exactly.
 __device__ __forceinline__ float exp2_whole(float n) {
@@ -464,7 +462,7 @@ attention_decode_kernel(Params p) {
                 for (int i = 0; i < 4; ++i) st[h][i] += st_odd[h][i];
                 if (CAP) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) st[h][i] = tanh_approx(st[h][i] * p.cap_in);
+                    for (int i = 0; i < 4; ++i) st[h][i] = tanh_by_exponential(st[h][i] * p.cap_in);
                 }
                 if (low_hidden) st[h][0] = st[h][1] = -INFINITY;       // (only the range's last keys can be)
                 if (high_hidden) st[h][2] = st[h][3] = -INFINITY;

@@ -5,12 +5,6 @@
 #include "tcgen05.cuh"
 
 namespace tc5 {
-// tanh by the hardware's approximation (relative error about 2^-11, below the rounding of the 16-bit probabilities)
-__device__ __forceinline__ float tanh_approx(float x) {
-    float y;
-    asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 __device__ __forceinline__ float ex2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -34,6 +28,27 @@ __device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
     uint64_t d;
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
     return d;
+}
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+// tanh as 1 - 2 / (1 + exp(2x)): absolute error about 2^-22, any x
+__device__ __forceinline__ float tanh_by_exponential(float x) {
+    return 1.0f - __fdividef(2.0f, 1.0f + ex2_approx(x * 2.8853900817779268f));
+}
+// tanh of two numbers within [-1, 1]: x P(x^2), P the polynomial of degree 5 that agrees with tanh(sqrt(u)) / sqrt(u) at the six
+// Chebyshev nodes of [0, 1] (absolute error below 2^-20).  It runs on the multiply-add pipes, beside the exponentials.
+__device__ __forceinline__ uint64_t tanh_within_one(uint64_t x) {
+    const uint64_t u = mul_f32x2(x, x);
+    uint64_t r = pack_f32x2(-0.00305822904f, -0.00305822904f);
+    r = fma_f32x2(r, u, pack_f32x2(0.0167208552f, 0.0167208552f));
+    r = fma_f32x2(r, u, pack_f32x2(-0.0515859884f, -0.0515859884f));
+    r = fma_f32x2(r, u, pack_f32x2(0.132807206f, 0.132807206f));
+    r = fma_f32x2(r, u, pack_f32x2(-0.333289514f, -0.333289514f));
+    r = fma_f32x2(r, u, pack_f32x2(0.999999395f, 0.999999395f));
+    return mul_f32x2(r, x);
 }
 __device__ __forceinline__ float exp2_whole(float n) {       // 2^n for a whole number n <= 0 (or -infinity), exactly
     return n < -126.f ? 0.f : __int_as_float(((int)n + 127) << 23);

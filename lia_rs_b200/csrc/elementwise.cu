@@ -7,7 +7,7 @@
 // A token id outside [0, vocab) writes zeros and raises the error flag (no read out of range).
 template <typename TW>
 __global__ void embedding_kernel(const int* __restrict__ tokens, const TW* __restrict__ table,
-                                 float* __restrict__ out, int n_tokens, int hidden, int vocab,
+                                 float* __restrict__ out, float* __restrict__ copy, int n_tokens, int hidden, int vocab,
                                  float scale, int* __restrict__ error_flag) {
     pdl_launch_dependents();
     pdl_wait();
@@ -18,11 +18,15 @@ __global__ void embedding_kernel(const int* __restrict__ tokens, const TW* __res
     if (!ok && threadIdx.x == 0 && error_flag) atomicExch(error_flag, 1);
     const TW* row = table + (size_t)(ok ? token : 0) * hidden;
     float* dst = out + (size_t)t * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-        dst[i] = ok ? to_float(row[i]) * scale : 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = ok ? to_float(row[i]) * scale : 0.f;
+        dst[i] = v;
+        if (copy) copy[(size_t)t * hidden + i] = v;
+    }
 }
 
-LIA_EXPORT int lia_embedding(const int* tokens, const void* table, int table_dtype, float* out,
+// `copy` (or null): the same rows once more.
+LIA_EXPORT int lia_embedding(const int* tokens, const void* table, int table_dtype, float* out, float* copy,
                              int n_tokens, int hidden, int vocab, float scale, int* error_flag,
                              cudaStream_t stream) {
     if (n_tokens <= 0) return LIA_OK;
@@ -30,10 +34,10 @@ LIA_EXPORT int lia_embedding(const int* tokens, const void* table, int table_dty
     const int threads = hidden >= 1024 ? 256 : 128;
     if (table_dtype == LIA_BF16)
         return lia_launch(embedding_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, tokens,
-                          (const __nv_bfloat16*)table, out, n_tokens, hidden, vocab, scale, error_flag);
+                          (const __nv_bfloat16*)table, out, copy, n_tokens, hidden, vocab, scale, error_flag);
     if (table_dtype == LIA_F32)
         return lia_launch(embedding_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, tokens, (const float*)table,
-                          out, n_tokens, hidden, vocab, scale, error_flag);
+                          out, copy, n_tokens, hidden, vocab, scale, error_flag);
     return LIA_ERR_DTYPE;
 }
 

@@ -28,102 +28,147 @@ namespace {
 constexpr int TILE_M = 32, TILE_N = 64, TILE_K = 32;
 constexpr int MOE_MAX_EXPERTS = 1024, MOE_MAX_TOP = 32;
 
-template <typename T>
-__global__ void moe_route_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ router, int hidden,
+// TOKENS tokens a CTA: a router row is read once for all of them.  A score's additions have the same order whatever TOKENS is.
+template <typename T, int TOKENS>
+__global__ void moe_route_kernel(const T* __restrict__ x, long long ld, const float* __restrict__ router, int n, int hidden,
                                  int experts, int top, float scale, int extra, const float* __restrict__ correction,
                                  int groups, int keep, int renormalise, int sigmoid, int two_best, int* __restrict__ ids,
                                  float* __restrict__ weights, float* __restrict__ shared_gate) {
-    extern __shared__ __align__(16) float route_shared[];  // x [hidden], z [experts + extra], choice scores [experts], groups' scores [groups]
-    __shared__ int picked[MOE_MAX_TOP];
+    // x [TOKENS][padded], z [TOKENS][experts + extra], choice scores [TOKENS][experts], groups' scores [TOKENS][groups]
+    extern __shared__ __align__(16) float route_shared[];
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x;
+    const int first = blockIdx.x * TOKENS, count = min(TOKENS, n - first);
+    const int padded = (hidden + 3) & ~3, outputs = experts + extra;
     float* xs = route_shared;
-    float* z = xs + hidden;
-    float* choice = z + experts + extra;
-    const T* row = x + (size_t)t * ld;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) xs[i] = to_float(row[i]);
+    float* z_all = xs + TOKENS * padded;
+    float* choice_all = z_all + TOKENS * outputs;
+    float* judged_all = choice_all + TOKENS * experts;
+    if (sizeof(T) == 2 && (hidden & 7) == 0 && (ld & 7) == 0 && ((uintptr_t)x & 15u) == 0) {
+        const int eighths = hidden / 8;
+        for (int e = threadIdx.x; e < TOKENS * eighths; e += blockDim.x) {
+            const int t = e / eighths, i = (e - t * eighths) * 8;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (t < count) v = *reinterpret_cast<const uint4*>(x + (size_t)(first + t) * ld + i);
+            const uint32_t words[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                *reinterpret_cast<float2*>(xs + t * padded + i + 2 * k) = make_float2(__uint_as_float(words[k] << 16), __uint_as_float(words[k] & 0xffff0000u));
+        }
+    } else {
+        for (int t = 0; t < TOKENS; ++t)
+            for (int i = threadIdx.x; i < hidden; i += blockDim.x) xs[t * padded + i] = t < count ? to_float(x[(size_t)(first + t) * ld + i]) : 0.f;
+    }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     // (four elements a lane and step where the rows allow it; the order of a score's additions depends on `hidden` alone)
     const bool by_fours = (hidden & 3) == 0 && ((uintptr_t)router & 15u) == 0;
-    for (int e = warp; e < experts + extra; e += warps) {
+    for (int e = warp; e < outputs; e += warps) {
         const float* w = router + (size_t)e * hidden;
-        float acc = 0.f;
+        float acc[TOKENS];
+#pragma unroll
+        for (int t = 0; t < TOKENS; ++t) acc[t] = 0.f;
         if (by_fours) {
             const float4* w4 = reinterpret_cast<const float4*>(w);
             const float4* x4 = reinterpret_cast<const float4*>(xs);
 #pragma unroll 4
             for (int i = lane; i < hidden / 4; i += 32) {
-                const float4 a = x4[i], b = __ldg(w4 + i);
-                acc = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+                const float4 b = __ldg(w4 + i);
+#pragma unroll
+                for (int t = 0; t < TOKENS; ++t) {
+                    const float4 a = x4[t * (padded / 4) + i];
+                    acc[t] = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc[t]))));
+                }
             }
         } else {
-            for (int i = lane; i < hidden; i += 32) acc = fmaf(xs[i], w[i], acc);
+            for (int i = lane; i < hidden; i += 32) {
+                const float b = w[i];
+#pragma unroll
+                for (int t = 0; t < TOKENS; ++t) acc[t] = fmaf(xs[t * padded + i], b, acc[t]);
+            }
         }
-        acc = warp_sum(acc);
-        if (lane == 0) z[e] = acc;
+#pragma unroll
+        for (int t = 0; t < TOKENS; ++t) {
+            const float sum = warp_sum(acc[t]);
+            if (lane == 0) z_all[t * outputs + e] = sum;
+        }
     }
     __syncthreads();
-    if (threadIdx.x != 0) return;
-    if (sigmoid) {
-        for (int e = 0; e < experts; ++e) z[e] = 1.0f / (1.0f + expf(-z[e]));
-    } else {
-        float largest = -INFINITY;
-        for (int e = 0; e < experts; ++e) largest = fmaxf(largest, z[e]);
-        float total = 0.f;
-        for (int e = 0; e < experts; ++e) {
-            z[e] = expf(z[e] - largest);
-            total += z[e];
+    // scores and choice: a warp a token
+    for (int t = warp; t < count; t += warps) {
+        float* z = z_all + t * outputs;
+        float* choice = choice_all + t * experts;
+        if (sigmoid) {
+            for (int e = lane; e < experts; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
+        } else {
+            float largest = -INFINITY;
+            for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, z[e]);
+            largest = warp_max(largest);
+            float total = 0.f;
+            for (int e = lane; e < experts; e += 32) {
+                z[e] = expf(z[e] - largest);
+                total += z[e];
+            }
+            const float inv = 1.0f / warp_sum(total);
+            for (int e = lane; e < experts; e += 32) z[e] *= inv;
         }
-        const float inv = 1.0f / total;
-        for (int e = 0; e < experts; ++e) z[e] *= inv;
-    }
-    for (int e = 0; e < experts; ++e) choice[e] = z[e] + (correction ? correction[e] : 0.f);      // z: the scores s_e
-    if (groups > 1) {
-        // the `keep` groups with the largest group score stay (the lower group wins a tie); the others' outputs cannot
-        // be chosen
-        const int size = experts / groups;
-        float* judged = choice + experts;
-        for (int g = 0; g < groups; ++g) {
-            float best = -INFINITY, second = -INFINITY;
-            for (int e = g * size; e < (g + 1) * size; ++e) {
+        for (int e = lane; e < experts; e += 32) choice[e] = z[e] + (correction ? correction[e] : 0.f);      // z: the scores s_e
+        __syncwarp();
+        if (groups > 1) {
+            // the `keep` groups with the largest group score stay (the lower group wins a tie); the others' outputs cannot
+            // be chosen
+            const int size = experts / groups;
+            float* judged = judged_all + t * groups;
+            for (int g = lane; g < groups; g += 32) {
+                float best = -INFINITY, second = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float v = choice[e];
+                    if (v > best) second = best, best = v;
+                    else second = fmaxf(second, v);
+                }
+                judged[g] = two_best && size > 1 ? best + second : best;
+            }
+            __syncwarp();
+            for (int g = lane; g < groups; g += 32) {
+                int ahead = 0;
+                for (int o = 0; o < groups; ++o)
+                    if (o != g && (judged[o] > judged[g] || (judged[o] == judged[g] && o < g))) ++ahead;
+                if (ahead >= keep) {
+                    // NaN marks an output that is out of the choice (a choice score may be any number, minus infinity too)
+                    for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = __int_as_float(0x7fc00000);
+                }
+            }
+            __syncwarp();
+        }
+        float chosen_sum = 0.f;
+        int mine = 0;                                          // lane c keeps the c-th choice
+        for (int c = 0; c < top; ++c) {
+            int best = experts;                                // (none)
+            float value = 0.f;
+            for (int e = lane; e < experts; e += 32) {
                 const float v = choice[e];
-                if (v > best) second = best, best = v;
-                else second = fmaxf(second, v);
+                if (v != v) continue;                          // taken, or of a group that is out
+                if (best == experts || v > value) value = v, best = e;
             }
-            judged[g] = two_best && size > 1 ? best + second : best;
-        }
-        for (int g = 0; g < groups; ++g) {
-            int ahead = 0;
-            for (int o = 0; o < groups; ++o)
-                if (o != g && (judged[o] > judged[g] || (judged[o] == judged[g] && o < g))) ++ahead;
-            if (ahead >= keep) {
-                // NaN marks an output that is out of the choice (a choice score may be any number, minus infinity too)
-                for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = __int_as_float(0x7fc00000);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const int other = __shfl_xor_sync(0xffffffffu, best, o);
+                const float v = __shfl_xor_sync(0xffffffffu, value, o);
+                if (other != experts && (best == experts || v > value || (v == value && other < best))) value = v, best = other;
             }
+            if (best == experts) best = 0;                     // (fewer outputs left than `top`: the launcher refuses that)
+            if (lane == c) mine = best;
+            chosen_sum += z[best];
+            if (lane == 0) choice[best] = __int_as_float(0x7fc00000);
+            __syncwarp();
         }
-    }
-    float chosen_sum = 0.f;
-    for (int c = 0; c < top; ++c) {
-        int best = -1;
-        float value = 0.f;
-        for (int e = 0; e < experts; ++e) {
-            const float v = choice[e];
-            if (v != v) continue;                          // taken, or of a group that is out
-            if (best < 0 || v > value) value = v, best = e;
+        const float factor = renormalise ? scale / (chosen_sum + 1e-20f) : scale;
+        if (lane < top) {
+            ids[(size_t)(first + t) * top + lane] = mine;
+            weights[(size_t)(first + t) * top + lane] = z[mine] * factor;
         }
-        if (best < 0) best = 0;                            // (fewer outputs left than `top`: the launcher refuses that)
-        picked[c] = best;
-        chosen_sum += z[best];
-        choice[best] = __int_as_float(0x7fc00000);
+        if (extra && lane == 0) shared_gate[first + t] = 1.0f / (1.0f + expf(-z[experts]));
     }
-    const float factor = renormalise ? scale / (chosen_sum + 1e-20f) : scale;
-    for (int c = 0; c < top; ++c) {
-        ids[(size_t)t * top + c] = picked[c];
-        weights[(size_t)t * top + c] = z[picked[c]] * factor;
-    }
-    if (extra) shared_gate[t] = 1.0f / (1.0f + expf(-z[experts]));
 }
 
 __global__ void moe_plan_kernel(const int* __restrict__ ids, int pairs, int experts, int tile_rows, int pad, int rows_cap,
@@ -307,25 +352,33 @@ LIA_EXPORT int lia_moe_route(const void* x, int dtype, long long ld, const float
                              cudaStream_t stream) {
     if (n <= 0) return LIA_OK;
     if (hidden <= 0 || experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts || top > MOE_MAX_TOP ||
-        extra < 0 || extra > 1 || (extra && !shared_gate) || ld < hidden || (size_t)(hidden + 3 * experts + 1) * 4 > 200 * 1024)
+        extra < 0 || extra > 1 || (extra && !shared_gate) || ld < hidden || (size_t)(hidden + 3 + 3 * experts + 1) * 4 > 200 * 1024)
         return LIA_ERR_SIZE;
     if (groups > 1 && (experts % groups || keep < 1 || keep > groups || (long long)keep * (experts / groups) < top))
         return LIA_ERR_SIZE;
-    const size_t bytes = (size_t)(hidden + 2 * experts + extra + (groups > 1 ? groups : 0)) * sizeof(float);
+    const size_t one = (size_t)(((hidden + 3) & ~3) + 2 * experts + extra + (groups > 1 ? groups : 0)) * sizeof(float);
     static bool raised = false;
     if (!raised) {
-        cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<float, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         raised = true;
     }
-    if (dtype == LIA_F32)
-        return lia_launch(moe_route_kernel<float>, dim3(n), dim3(256), bytes, stream, (const float*)x, ld, router, hidden,
-                          experts, top, scale, extra, correction, groups, keep, renormalise, sigmoid, two_best, ids,
-                          weights, shared_gate);
-    if (dtype == LIA_BF16)
-        return lia_launch(moe_route_kernel<__nv_bfloat16>, dim3(n), dim3(256), bytes, stream, (const __nv_bfloat16*)x, ld,
-                          router, hidden, experts, top, scale, extra, correction, groups, keep, renormalise, sigmoid, two_best, ids,
-                          weights, shared_gate);
+    const bool eight = n >= 8 * 148 && 8 * one <= 200 * 1024;
+#define LIA_ROUTE(T, TOKENS)                                                                                             \
+    return lia_launch(moe_route_kernel<T, TOKENS>, dim3((n + TOKENS - 1) / TOKENS), dim3(256), TOKENS * one, stream,     \
+                      (const T*)x, ld, router, n, hidden, experts, top, scale, extra, correction, groups, keep,          \
+                      renormalise, sigmoid, two_best, ids, weights, shared_gate)
+    if (dtype == LIA_F32) {
+        if (eight) LIA_ROUTE(float, 8);
+        LIA_ROUTE(float, 1);
+    }
+    if (dtype == LIA_BF16) {
+        if (eight) LIA_ROUTE(__nv_bfloat16, 8);
+        LIA_ROUTE(__nv_bfloat16, 1);
+    }
+#undef LIA_ROUTE
     return LIA_ERR_DTYPE;
 }
 

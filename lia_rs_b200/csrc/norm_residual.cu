@@ -42,13 +42,79 @@ __global__ void norm_residual_kernel(const float* __restrict__ y, const float* _
         nr[i] = from_float<TO>(xr[i] * inv2 * next_weight[i]);
 }
 
+template <typename TO> __device__ __forceinline__ void store_four(TO* dst, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void store_four<float>(float* dst, float a, float b, float c, float d) {
+    *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
+}
+template <> __device__ __forceinline__ void store_four<__nv_bfloat16>(__nv_bfloat16* dst, float a, float b, float c, float d) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    uint2 v;
+    v.x = *reinterpret_cast<uint32_t*>(&lo);
+    v.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = v;
+}
+
+// The same with a row in registers: PER quads a thread (width a multiple of 4, rows 16-byte aligned), the row read once and
+// the weights, which no kernel writes, on their way before the kernel ahead is awaited.
+template <typename TO, int PER>
+__global__ void norm_residual_quads_kernel(const float* __restrict__ y, const float* __restrict__ bias,
+                                           const float* __restrict__ weight, float* __restrict__ residual,
+                                           const float* __restrict__ next_weight, TO* __restrict__ next, int hidden, float eps,
+                                           float next_eps) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    const int r = blockIdx.x, quads = hidden / 4;
+    float4 w[PER], w2[PER], b[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + i * blockDim.x;
+        const bool in = q < quads;
+        w[i] = in ? reinterpret_cast<const float4*>(weight)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+        w2[i] = in && next ? reinterpret_cast<const float4*>(next_weight)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+        b[i] = in && bias ? reinterpret_cast<const float4*>(bias)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    float4 v[PER], x[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + i * blockDim.x;
+        v[i] = q < quads ? reinterpret_cast<const float4*>(y + (size_t)r * hidden)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+        x[i] = q < quads ? reinterpret_cast<const float4*>(residual + (size_t)r * hidden)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        v[i].x += b[i].x, v[i].y += b[i].y, v[i].z += b[i].z, v[i].w += b[i].w;
+        sum = fmaf(v[i].x, v[i].x, sum), sum = fmaf(v[i].y, v[i].y, sum);
+        sum = fmaf(v[i].z, v[i].z, sum), sum = fmaf(v[i].w, v[i].w, sum);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)hidden + eps);
+    float sum2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + i * blockDim.x;
+        x[i].x += v[i].x * inv * w[i].x, x[i].y += v[i].y * inv * w[i].y;
+        x[i].z += v[i].z * inv * w[i].z, x[i].w += v[i].w * inv * w[i].w;
+        if (q < quads) reinterpret_cast<float4*>(residual + (size_t)r * hidden)[q] = x[i];
+        sum2 = fmaf(x[i].x, x[i].x, sum2), sum2 = fmaf(x[i].y, x[i].y, sum2);
+        sum2 = fmaf(x[i].z, x[i].z, sum2), sum2 = fmaf(x[i].w, x[i].w, sum2);
+    }
+    if (!next) return;
+    const float inv2 = 1.0f / sqrtf(block_sum(sum2, scratch) / (float)hidden + next_eps);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int q = threadIdx.x + i * blockDim.x;
+        if (q < quads)
+            store_four<TO>(next + (size_t)r * hidden + 4 * q, x[i].x * inv2 * w2[i].x, x[i].y * inv2 * w2[i].y, x[i].z * inv2 * w2[i].z,
+                           x[i].w * inv2 * w2[i].w);
+    }
+}
+
 // residual[r] += rms(v) * weight with v = sum_i scale_i * (w_i ? rms_i(y_i + b_i) * w_i : y_i + b_i) over one or two terms, and
 // `next` (optional) the new stream in the compute element type: what follows a sublayer whose output is normed and whose
 // successor reads the stream itself, in one pass.  A thread keeps PER quads of the row in registers (width a multiple of
 // 4, rows 16-byte aligned); PER 0: any width, the row read again for every pass.
 struct NormTerm { const float* y; const float* bias; const float* weight; float scale, eps; };
-
-template <typename TO> __device__ __forceinline__ void store_four(TO* dst, float a, float b, float c, float d);
 
 template <typename TO, int TERMS, int PER>
 __global__ void norm_terms_residual_kernel(NormTerm t0, NormTerm t1, const float* __restrict__ weight,
@@ -176,17 +242,6 @@ __device__ __forceinline__ float activate(int act, float z, float p0 = 0.f, floa
     return z;
 }
 
-template <> __device__ __forceinline__ void store_four<float>(float* dst, float a, float b, float c, float d) {
-    *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
-}
-template <> __device__ __forceinline__ void store_four<__nv_bfloat16>(__nv_bfloat16* dst, float a, float b, float c, float d) {
-    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
-    uint2 v;
-    v.x = *reinterpret_cast<uint32_t*>(&lo);
-    v.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(dst) = v;
-}
-
 // four elements a thread: rows whose width and strides are multiples of 4 from 16-byte aligned bases.  `gated`: the
 // row holds `width` gate elements and then `width` more, out = act(gate) * the other.
 template <typename TO>
@@ -228,14 +283,31 @@ LIA_EXPORT int lia_norm_residual(const float* y, const float* bias, const float*
                                  float next_eps, cudaStream_t stream) {
     if (rows <= 0) return LIA_OK;
     if (hidden <= 0 || (next && !next_weight)) return LIA_ERR_SIZE;
-    const int threads = hidden >= 2048 ? 512 : hidden >= 512 ? 256 : 128;
+    int threads = hidden >= 2048 ? 512 : hidden >= 512 ? 256 : 128;
+    if (next && next_dtype != LIA_F32 && next_dtype != LIA_BF16) return LIA_ERR_DTYPE;
+    const uintptr_t bits = (uintptr_t)y | (uintptr_t)bias | (uintptr_t)weight | (uintptr_t)residual | (uintptr_t)next_weight | (uintptr_t)next;
+    if (hidden % 4 == 0 && (bits & 15u) == 0 && hidden <= 8192) {
+        const int quads = hidden / 4;
+        threads = quads <= 64 ? 64 : quads <= 128 ? 128 : quads <= 256 ? 256 : 512;
+        const int per = (quads + threads - 1) / threads;
+#define LIA_QUADS(TO, PER)                                                                                                  \
+    return lia_launch(norm_residual_quads_kernel<TO, PER>, dim3(rows), dim3(threads), 0, stream, y, bias, weight, residual, \
+                      next_weight, (TO*)next, hidden, eps, next_eps)
+        if (next && next_dtype == LIA_BF16) {
+            if (per == 1) LIA_QUADS(__nv_bfloat16, 1);
+            if (per == 2) LIA_QUADS(__nv_bfloat16, 2);
+            LIA_QUADS(__nv_bfloat16, 4);
+        }
+        if (per == 1) LIA_QUADS(float, 1);
+        if (per == 2) LIA_QUADS(float, 2);
+        LIA_QUADS(float, 4);
+#undef LIA_QUADS
+    }
     if (!next || next_dtype == LIA_F32)
         return lia_launch(norm_residual_kernel<float>, dim3(rows), dim3(threads), 0, stream, y, bias, weight, residual,
                           next_weight, (float*)next, rows, hidden, eps, next_eps);
-    if (next_dtype == LIA_BF16)
-        return lia_launch(norm_residual_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, y, bias, weight,
-                          residual, next_weight, (__nv_bfloat16*)next, rows, hidden, eps, next_eps);
-    return LIA_ERR_DTYPE;
+    return lia_launch(norm_residual_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, y, bias, weight, residual,
+                      next_weight, (__nv_bfloat16*)next, rows, hidden, eps, next_eps);
 }
 
 // One or two terms (y1 null: one) of rows [rows, hidden], each with an optional bias [hidden] and an optional norm (weight

@@ -38,7 +38,7 @@ def lib():
 
 
 class _Signatures:
-    lia_embedding = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p]
+    lia_embedding = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p]
     lia_rmsnorm = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]
     lia_layernorm = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p]
     lia_rope_kv_write = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
@@ -314,11 +314,14 @@ def _gemm_work(a, w, out):
             2 * a.shape[0] * w.shape[0] * a.shape[1])
 
 
-def embedding(tokens, table, out, scale: float, error_flag=None):
-    _cuda(tokens, table, out, error_flag)
+def embedding(tokens, table, out, scale: float, error_flag=None, copy=None):
+    """out[t] = table[token_t] * scale, 32-bit; `copy`: the same rows once more."""
+    _cuda(tokens, table, out, error_flag, copy)
     n, hidden = out.shape
+    if copy is not None and (copy.shape != out.shape or copy.dtype != torch.float32):
+        raise KernelError("embedding: the copy is 32-bit rows of the output's shape")
     with _timed("embedding"):
-        _check(lib().lia_embedding(_p(tokens), _p(table), dtype_code(table.dtype), _p(out), n, hidden,
+        _check(lib().lia_embedding(_p(tokens), _p(table), dtype_code(table.dtype), _p(out), _p(copy), n, hidden,
                                    table.shape[0], scale, _p(error_flag), _stream()), "embedding")
 
 

@@ -219,9 +219,7 @@ class DecoderModel:
             rt.ops.embedding_positions(ctx.tokens, ctx.positions, self.embedding, self.position_table, h,
                                        spec.embedding_scale, copy=first, error_flag=ctx.error_flag)
         else:
-            rt.ops.embedding(ctx.tokens, self.embedding, h, spec.embedding_scale, ctx.error_flag)
-            if first is not None:
-                first.copy_(h)
+            rt.ops.embedding(ctx.tokens, self.embedding, h, spec.embedding_scale, ctx.error_flag, copy=first)
         ctx.rounded_stream = rounded
         picked = None
         last = len(spec.schedule) - 1

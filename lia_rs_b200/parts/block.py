@@ -118,6 +118,7 @@ class SandwichBlock(Arrangement):
     `output_bias` is added ahead of post1.  `residual_scale` has no meaning here (a norm follows the sublayer) and must
     be 1.  Checkpoint names: `names["norm1"]`, `["norm1b"]`, `["mixer"]`, `["norm2"]`, `["norm2b"]`, `["feed_forward"]`."""
 
+    supports_rows = True
     PLACES = ("norm1", "norm1b", "norm2", "norm2b")
 
     @staticmethod
@@ -171,7 +172,7 @@ class SandwichBlock(Arrangement):
             key += part.graph_key(ctx)
         return key
 
-    def forward(self, ctx, residual, kv=None, state=None):
+    def forward(self, ctx, residual, kv=None, state=None, rows=None, n_rows=None):
         ops = self.runtime.ops
         deferred = DeferredNorm(ctx, self.pre1, residual)
         x = deferred if self.mixer.takes_deferred_norm else deferred.tensor()
@@ -181,10 +182,21 @@ class SandwichBlock(Arrangement):
         else:
             y.zero_()
             self.mixer.forward(ctx, x, y, 1.0, kv=kv, state=state)
+        picked = None
+        if rows is not None:
+            # only `rows` matter after this layer: cache and state are up to date for every token, the rest runs on the
+            # picked rows alone
+            picked = ctx.buffer("block.picked", (n_rows, residual.shape[1]), residual.dtype)
+            if not n_rows:
+                return picked
+            chosen = ctx.buffer("block.picked_term0", tuple(picked.shape), torch.float32)
+            ops.gather_rows(residual, rows, picked)
+            ops.gather_rows(y, rows, chosen)
+            residual, y = picked, chosen
         weight, eps = self.post["norm1b"]
         if self.feed_forward is None:
             ops.norm_residual(y, weight, residual, eps, bias=self.mixer.output_bias)
-            return None
+            return picked
         if self.feed_forward.takes_deferred_norm and residual.shape[0] <= ops.STREAM_MAX_TOKENS:
             ops.norm_residual(y, weight, residual, eps, bias=self.mixer.output_bias)
             x = DeferredNorm(ctx, self.pre2, residual, buffer_name="block.x2")
@@ -200,7 +212,7 @@ class SandwichBlock(Arrangement):
             self.feed_forward.forward(ctx, x, y, 1.0)
         weight, eps = self.post["norm2b"]
         ops.norm_residual(y, weight, residual, eps)
-        return None
+        return picked
 
 
 @register_arrangement("postnorm")

@@ -62,7 +62,7 @@ def attention(h, positions, w, m, eps):
     """q, k, v = W h + b; q and k turned in interleaved pairs over their first rot.dims elements, then each head of q and
     of k over its root mean square (no weight); `attend`; the heads side by side through W_o."""
     T, H, d = h.shape[0], m["heads"], m["dim"]
-    G, dv = m["kv_heads"], m["vdim"]
+    G, dv = m.get("kv_heads", H), m.get("vdim", d)
     q = (h @ w["q"].to(F64).T + w["q.b"].to(F64)).view(T, H, d)
     k = (h @ w["k"].to(F64).T + w["k.b"].to(F64)).view(T, G, d)
     v = (h @ w["v"].to(F64).T + w["v.b"].to(F64)).view(T, G, dv)
@@ -73,10 +73,12 @@ def attention(h, positions, w, m, eps):
     return o.reshape(T, H * dv) @ w["o"].to(F64).T
 
 
-def mlstm_recurrence(q, k, v, i, f, state=None):
+def mlstm_recurrence(q, k, v, i, f, state=None, fragile=None):
     """q, k [T, H, d], v [T, H, dv], log gates i, f [T, H].  With S [H, d, dv], n [H, d] and m [H] (all zero at the start, or
     `state`): m_t = max(f_t + m_(t-1), i_t), S_t = exp(f_t + m_(t-1) - m_t) S_(t-1) + exp(i_t - m_t) k_t v_t^T, n_t the same
-    with k_t alone, o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6).  Returns (o [T, H, dv], (S, n, m))."""
+    with k_t alone, o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6).  Returns (o [T, H, dv], (S, n, m)).  `fragile` [T]:
+    marked where a head's query lies almost across everything its memory holds, so that S_t^T q_t is what rounding leaves of it
+    (the norm behind it raises that to full size)."""
     T, H, d = q.shape
     S, n, m = (torch.zeros(H, d, v.shape[2], dtype=F64), torch.zeros(H, d, dtype=F64), torch.zeros(H, dtype=F64)) \
         if state is None else tuple(t.clone() for t in state)
@@ -88,11 +90,15 @@ def mlstm_recurrence(q, k, v, i, f, state=None):
         n = keep[:, None] * n + put[:, None] * k[t]
         m = new
         below = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
-        out[t] = torch.einsum("hdv,hd->hv", S, q[t]) / below[:, None]
+        read = torch.einsum("hdv,hd->hv", S, q[t])
+        if fragile is not None:
+            most = S.flatten(1).norm(dim=1) * q[t].norm(dim=1)
+            fragile[t] |= bool((read.norm(dim=1) < 3e-2 * most).any())
+        out[t] = read / below[:, None]
     return out, (S, n, m)
 
 
-def mlstm(h, w, m, eps, state=None):
+def mlstm(h, w, m, eps, state=None, fragile=None):
     """q = W_q h dim^(-1/2), k = W_k h, v = W_v h; log gates i = cap tanh((W_i h + b_i) / cap) and
     f = log sigmoid(cap tanh((W_f h + b_f) / cap)); `mlstm_recurrence`; each head's o over its root mean square; heads side
     by side times a weight, times sigmoid(W_g h), through W_o.  Returns (output, the state behind the last token)."""
@@ -102,7 +108,7 @@ def mlstm(h, w, m, eps, state=None):
     v = (h @ w["v"].to(F64).T).view(T, H, dv)
     i = cap * torch.tanh((h @ w["i"].to(F64).T + w["i.b"].to(F64)) / cap)
     f = torch.nn.functional.logsigmoid(cap * torch.tanh((h @ w["f"].to(F64).T + w["f.b"].to(F64)) / cap))
-    o, state = mlstm_recurrence(q, k, v, i, f, state)
+    o, state = mlstm_recurrence(q, k, v, i, f, state, fragile)
     y = rms(o, eps).reshape(T, H * dv) * w["norm"].to(F64) * torch.sigmoid(h @ w["g"].to(F64).T)
     return y @ w["o"].to(F64).T, state
 
@@ -135,11 +141,11 @@ def route(h, w, router, fragile=None):
         c = c.masked_fill(~allowed.repeat_interleave(size, dim=1), -math.inf)
         if fragile is not None and keep < count:
             ranked = torch.sort(judged, dim=-1, descending=True).values
-            fragile |= (ranked[:, keep - 1] - ranked[:, keep]) < 2e-2
+            fragile |= (ranked[:, keep - 1] - ranked[:, keep]) < 2.5e-2
     chosen = torch.topk(c, top, dim=-1).indices
     if fragile is not None and top < total:
         ranked = torch.sort(c, dim=-1, descending=True).values
-        fragile |= (ranked[:, top - 1] - ranked[:, top]) < 1e-2
+        fragile |= (ranked[:, top - 1] - ranked[:, top]) < 1.5e-2
     picked = torch.gather(s, 1, chosen)
     return chosen, picked / (picked.sum(dim=-1, keepdim=True) + 1e-20)
 
@@ -176,7 +182,7 @@ def layer_order(config):
 def forward(config: dict, tensors: dict, tokens, layer_outputs=None, fragile=None):
     """Logits [T, vocab] (64-bit) of one sequence from position 0.  `layer_outputs`: a list that receives the residual
     stream after every layer run.  `fragile`: a boolean tensor [T] in which the rows are marked whose result rests on a
-    router's close call that 16-bit rounding may turn."""
+    router's close call that 16-bit rounding may turn, or on what rounding leaves of a memory's answer."""
     eps = float(config["norm"]["eps"])
     positions = torch.arange(len(tokens))
     norm = lambda x, name: rms(x, eps) * tensors[name].to(F64)
@@ -190,7 +196,10 @@ def forward(config: dict, tensors: dict, tokens, layer_outputs=None, fragile=Non
         layer, p = config["layers"][i], f"l{i}."
         w = {k[len(p) + 4:]: v for k, v in tensors.items() if k.startswith(p + "mix.")}
         h = norm(x, p + "norm1")
-        y = attention(h, positions, w, layer["mixer"], eps) if layer["type"] == "attention" else mlstm(h, w, layer["mixer"], eps)[0]
+        if layer["type"] == "attention":
+            y = attention(h, positions, w, layer["mixer"], eps)
+        else:
+            y = mlstm(h, w, layer["mixer"], eps, fragile=fragile)[0]
         x = x + norm(y, p + "norm1b")
         mlp = layer.get("mlp")
         if mlp:
