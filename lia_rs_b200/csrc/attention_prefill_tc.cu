@@ -293,12 +293,22 @@ attention_prefill_tc_kernel(Params p) {
             tmem_load64_nowait(tmem_s + (uint32_t)((j & 1) * KT + half * HALF) + lane_base, raw);
             tmem_load_wait();
             if (CAP) {
-                // the cap's tanh: a polynomial while no score of the warp's tile passes the cap itself, else by exponentials
+                // the cap's tanh: a polynomial while no score of the warp's tile passes the cap, a shorter one while none passes
+                // half of it, else by exponentials
                 float far[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int c = 0; c < HALF; ++c) far[c & 3] = fmaxf(far[c & 3], fabsf(__uint_as_float(raw[c])));
                 const float farthest = fmaxf(fmaxf(far[0], far[1]), fmaxf(far[2], far[3])) * fabsf(p.cap_in);
-                if (!__any_sync(0xffffffffu, !(farthest <= 1.0f))) {
+                if (!__any_sync(0xffffffffu, !(farthest <= 0.5f))) {
+                    const uint64_t in2 = pack_f32x2(p.cap_in, p.cap_in);
+#pragma unroll
+                    for (int c = 0; c < HALF; c += 2) {
+                        float t0, t1;
+                        unpack_f32x2(tanh_within_half(mul_f32x2(pack_f32x2(__uint_as_float(raw[c]), __uint_as_float(raw[c + 1])), in2)), t0, t1);
+                        raw[c] = __float_as_uint(t0);
+                        raw[c + 1] = __float_as_uint(t1);
+                    }
+                } else if (!__any_sync(0xffffffffu, !(farthest <= 1.0f))) {
                     const uint64_t in2 = pack_f32x2(p.cap_in, p.cap_in);
 #pragma unroll
                     for (int c = 0; c < HALF; c += 2) {

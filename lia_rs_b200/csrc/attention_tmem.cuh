@@ -38,8 +38,9 @@ __device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
 __device__ __forceinline__ float tanh_by_exponential(float x) {
     return 1.0f - __fdividef(2.0f, 1.0f + ex2_approx(x * 2.8853900817779268f));
 }
-// tanh of two numbers within [-1, 1]: x P(x^2), P the polynomial of degree 5 that agrees with tanh(sqrt(u)) / sqrt(u) at the six
-// Chebyshev nodes of [0, 1] (absolute error below 2^-20).  It runs on the multiply-add pipes, beside the exponentials.
+// tanh of two numbers within [-1, 1] or [-1/2, 1/2]: x P(x^2), P the polynomial of degree 5 (3) that agrees with
+// tanh(sqrt(u)) / sqrt(u) at the six (four) Chebyshev nodes of [0, 1] ([0, 1/4]); absolute error below 2^-20 in both.  They run
+// on the multiply-add pipes, beside the exponentials.
 __device__ __forceinline__ uint64_t tanh_within_one(uint64_t x) {
     const uint64_t u = mul_f32x2(x, x);
     uint64_t r = pack_f32x2(-0.00305822904f, -0.00305822904f);
@@ -48,6 +49,14 @@ __device__ __forceinline__ uint64_t tanh_within_one(uint64_t x) {
     r = fma_f32x2(r, u, pack_f32x2(0.132807206f, 0.132807206f));
     r = fma_f32x2(r, u, pack_f32x2(-0.333289514f, -0.333289514f));
     r = fma_f32x2(r, u, pack_f32x2(0.999999395f, 0.999999395f));
+    return mul_f32x2(r, x);
+}
+__device__ __forceinline__ uint64_t tanh_within_half(uint64_t x) {
+    const uint64_t u = mul_f32x2(x, x);
+    uint64_t r = pack_f32x2(-0.0443927384f, -0.0443927384f);
+    r = fma_f32x2(r, u, pack_f32x2(0.131899394f, 0.131899394f));
+    r = fma_f32x2(r, u, pack_f32x2(-0.333262842f, -0.333262842f));
+    r = fma_f32x2(r, u, pack_f32x2(0.999999451f, 0.999999451f));
     return mul_f32x2(r, x);
 }
 __device__ __forceinline__ float exp2_whole(float n) {       // 2^n for a whole number n <= 0 (or -infinity), exactly

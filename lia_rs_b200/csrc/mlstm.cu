@@ -423,7 +423,7 @@ LIA_EXPORT int lia_mlstm(const float* qkv, long long ld, const float* gates, lon
 
 // The single tokens alone (batch indices `single_rows`): qkv of qkv_dtype (round16: 32-bit rows are rounded to bfloat16 as
 // they are read), the other arguments as for lia_mlstm.  `wanted_ctas`: a head's columns are shared by up to 8 CTAs while there
-// are fewer CTAs than this.
+// are fewer CTAs than this and a CTA's share of the memory is 128 KB or more (a cluster costs about 2 us: smaller heads stay whole).
 LIA_EXPORT int lia_mlstm_single(const void* qkv, int qkv_dtype, long long ld, int round16, const float* gates, long long ld_g,
                                 const float* i_bias, const float* f_bias, float cap, float* state, long long slot_stride,
                                 const int* single_rows, int n_single, const int* slots, const float* norm_weight, float eps,
@@ -441,7 +441,8 @@ LIA_EXPORT int lia_mlstm_single(const void* qkv, int qkv_dtype, long long ld, in
     p.q_scale = 1.0f / sqrtf((float)d);
     const bool four = dv % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15u) == 0;
     int share = 1;
-    while (four && share < 8 && dv % (share * 2 * 32) == 0 && (long long)n_single * heads * share < wanted_ctas) share *= 2;
+    while (four && share < 8 && dv % (share * 2 * 32) == 0 && (long long)d * dv >= 32768LL * share && (long long)n_single * heads * share < wanted_ctas)
+        share *= 2;
     if (out_dtype == LIA_F32)
         return four ? launch_single<float, 4>(p, n_single, share, round16, stream) : launch_single<float, 1>(p, n_single, 1, round16, stream);
     return four ? launch_single<__nv_bfloat16, 4>(p, n_single, share, round16, stream)

@@ -35,6 +35,8 @@ __device__ __forceinline__ float pow2(float x) {             // x <= 0; relative
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// the logistic function by the hardware's exponential and division (relative error about 2^-21; the result is rounded to 16 bits)
+__device__ __forceinline__ float fast_sigmoid(float v) { return __fdividef(1.0f, 1.0f + __expf(-v)); }
 // two numbers as bfloat16 pairs: the nearest, and the nearest to what that misses
 __device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
@@ -57,7 +59,8 @@ __device__ __forceinline__ void bring_rows(__nv_bfloat16* dst, const __nv_bfloat
 }
 __device__ __forceinline__ void rows_there() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
-template <int TILES>                                     // TILES: most 16-wide tiles of a piece of the values
+// TILES: most 16-wide tiles of a piece of the values; FULL: every piece has that many (nothing then depends on the width)
+template <int TILES, bool FULL>
 __global__ void __launch_bounds__(MLSTM_THREADS)
 mlstm_sums_tc_kernel(MlstmArgs p, int piece) {
     extern __shared__ __align__(16) uint8_t sums_raw[];  // k [TOKENS][d + 8], v [TOKENS][w + 8] (then v' near), v' rest [TOKENS][w + 8]
@@ -68,7 +71,7 @@ mlstm_sums_tc_kernel(MlstmArgs p, int piece) {
     int first, len;
     bool last;
     if (!mlstm_find_chunk<TOKENS>(p, blockIdx.x, &first, &len, &last)) return;
-    const int h = blockIdx.y, d = p.d, dv = p.dv, c0 = blockIdx.z * piece, w = min(piece, dv - c0), ks = d + 8, vs = w + 8;
+    const int h = blockIdx.y, d = p.d, dv = p.dv, c0 = blockIdx.z * piece, w = FULL ? TILES * 16 : min(piece, dv - c0), ks = d + 8, vs = w + 8;
     __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(sums_raw);
     __nv_bfloat16* hi = k_s + TOKENS * ks;
     __nv_bfloat16* lo = hi + TOKENS * vs;
@@ -159,8 +162,8 @@ mlstm_sums_tc_kernel(MlstmArgs p, int piece) {
     }
 }
 
-template <int TILES>
-__global__ void __launch_bounds__(MLSTM_THREADS)
+template <int TILES, bool FULL>
+__global__ void __launch_bounds__(MLSTM_THREADS, 2)
 mlstm_output_tc_kernel(MlstmArgs p, int piece) {
     // q [TOKENS][d + 8], v [TOKENS][w + 8], then k [TOKENS][d + 8] and, in the same room once the chunk's own tokens are done
     // with, the incoming memory near and rest [d][w + 8] each
@@ -175,7 +178,7 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
     if (!mlstm_find_chunk<TOKENS>(p, blockIdx.x, &first, &len, &last)) return;
     const int slot = p.slots[first];
     if (slot < 0) return;
-    const int h = blockIdx.y, d = p.d, dv = p.dv, c0 = blockIdx.z * piece, w = min(piece, dv - c0), ds = d + 8, ws = w + 8;
+    const int h = blockIdx.y, d = p.d, dv = p.dv, c0 = blockIdx.z * piece, w = FULL ? TILES * 16 : min(piece, dv - c0), ds = d + 8, ws = w + 8;
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(out_raw);
     __nv_bfloat16* v_s = q_s + TOKENS * ds;
     __nv_bfloat16* k_s = v_s + TOKENS * ws;
@@ -261,7 +264,7 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
             }
 #pragma unroll
             for (int c = 0; c < TILES; ++c) {
-                if (c >= col_tiles) break;
+                if (!FULL && c >= col_tiles) break;
                 uint32_t b[4];
                 ldsm4_trans(shared_address(v_s + (j0 + half * 16 + (lane & 15)) * ws + c * 16 + (lane >> 4) * 8), b);
                 mma(acc[2 * c], near, b[0], b[1]);
@@ -288,7 +291,7 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
     const float w_low = start_s[t_low], w_high = start_s[t_high];
 #pragma unroll
     for (int c = 0; c < TILES; ++c) {
-        if (c >= col_tiles) break;
+        if (!FULL && c >= col_tiles) break;
         float in[2][4] = {};
         for (int k = 0; k < k_tiles; ++k) {
             uint32_t a[4], b[4], r[4];
@@ -318,7 +321,7 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
     float sq_low = 0.f, sq_high = 0.f;
 #pragma unroll
     for (int j = 0; j < 2 * TILES; ++j) {
-        if (j >= 2 * col_tiles) break;
+        if (!FULL && j >= 2 * col_tiles) break;
         acc[j][0] *= inv_low, acc[j][1] *= inv_low, acc[j][2] *= inv_high, acc[j][3] *= inv_high;
         sq_low = fmaf(acc[j][0], acc[j][0], fmaf(acc[j][1], acc[j][1], sq_low));
         sq_high = fmaf(acc[j][2], acc[j][2], fmaf(acc[j][3], acc[j][3], sq_high));
@@ -328,7 +331,7 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
         const size_t down = (size_t)p.heads * dv;
 #pragma unroll
         for (int j = 0; j < 2 * TILES; ++j) {
-            if (j >= 2 * col_tiles) break;
+            if (!FULL && j >= 2 * col_tiles) break;
             const int col = j * 8 + tq * 2;
             if (t_low < len) *reinterpret_cast<float2*>(y + gr * down + col) = make_float2(acc[j][0], acc[j][1]);
             if (t_high < len) *reinterpret_cast<float2*>(y + (gr + 8) * down + col) = make_float2(acc[j][2], acc[j][3]);
@@ -340,23 +343,34 @@ mlstm_output_tc_kernel(MlstmArgs p, int piece) {
     sq_low += __shfl_xor_sync(0xffffffffu, sq_low, 2);
     sq_high += __shfl_xor_sync(0xffffffffu, sq_high, 2);
     const float norm_low = 1.0f / sqrtf(sq_low / (float)dv + p.eps), norm_high = 1.0f / sqrtf(sq_high / (float)dv + p.eps);
-    const float* weights = p.norm_weight + (size_t)h * dv;
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)h * dv;
-    const float* gates = p.gates + (size_t)h * dv;
+    const float* weights = p.norm_weight + (size_t)h * dv + tq * 2;
+    // (rows behind the chunk's end read the gate of the chunk's first token and write nothing)
+    const float* g_low = p.gates + (size_t)(first + (t_low < len ? t_low : 0)) * p.ld_g + (size_t)h * dv + tq * 2;
+    const float* g_high = p.gates + (size_t)(first + (t_high < len ? t_high : 0)) * p.ld_g + (size_t)h * dv + tq * 2;
+    __nv_bfloat16* out_low = reinterpret_cast<__nv_bfloat16*>(p.out) + ((size_t)(first + t_low) * p.heads + h) * dv + tq * 2;
+    __nv_bfloat16* out_high = out_low + (size_t)8 * p.heads * dv;
+    constexpr int BATCH = 4;                             // (the loads of four columns' tiles are in flight together)
 #pragma unroll
-    for (int j = 0; j < 2 * TILES; ++j) {
-        if (j >= 2 * col_tiles) break;
-        const int col = j * 8 + tq * 2;
-        const float f0 = weights[col], f1 = weights[col + 1];
-        if (t_low < len) {
-            const float* g = gates + (size_t)(first + t_low) * p.ld_g + col;
-            *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(first + t_low) * p.heads * dv + col) =
-                __floats2bfloat162_rn(acc[j][0] * norm_low * f0 * mlstm_sigmoid(g[0]), acc[j][1] * norm_low * f1 * mlstm_sigmoid(g[1]));
+    for (int j0 = 0; j0 < 2 * TILES; j0 += BATCH) {
+        if (!FULL && j0 >= 2 * col_tiles) break;
+        float2 f[BATCH], low[BATCH], high[BATCH];
+#pragma unroll
+        for (int k = 0; k < BATCH; ++k) {
+            if (!FULL && j0 + k >= 2 * col_tiles) break;
+            f[k] = *reinterpret_cast<const float2*>(weights + (j0 + k) * 8);
+            low[k] = *reinterpret_cast<const float2*>(g_low + (j0 + k) * 8);
+            high[k] = *reinterpret_cast<const float2*>(g_high + (j0 + k) * 8);
         }
-        if (t_high < len) {
-            const float* g = gates + (size_t)(first + t_high) * p.ld_g + col;
-            *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(first + t_high) * p.heads * dv + col) =
-                __floats2bfloat162_rn(acc[j][2] * norm_high * f0 * mlstm_sigmoid(g[0]), acc[j][3] * norm_high * f1 * mlstm_sigmoid(g[1]));
+#pragma unroll
+        for (int k = 0; k < BATCH; ++k) {
+            const int j = j0 + k;
+            if (!FULL && j >= 2 * col_tiles) break;
+            if (t_low < len)
+                *reinterpret_cast<__nv_bfloat162*>(out_low + j * 8) = __floats2bfloat162_rn(
+                    acc[j][0] * norm_low * f[k].x * fast_sigmoid(low[k].x), acc[j][1] * norm_low * f[k].y * fast_sigmoid(low[k].y));
+            if (t_high < len)
+                *reinterpret_cast<__nv_bfloat162*>(out_high + j * 8) = __floats2bfloat162_rn(
+                    acc[j][2] * norm_high * f[k].x * fast_sigmoid(high[k].x), acc[j][3] * norm_high * f[k].y * fast_sigmoid(high[k].y));
         }
     }
 }
@@ -398,21 +412,21 @@ int piece_of(int d, int dv) {
     return 0;
 }
 
-template <int TILES>
+template <int TILES, bool FULL>
 int launch_portions(const MlstmArgs& p, int piece, int max_chunks, bool four, cudaStream_t stream) {
     static bool raised = false;
     if (!raised) {
-        if (cudaFuncSetAttribute(mlstm_sums_tc_kernel<TILES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(mlstm_output_tc_kernel<TILES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST_BYTES) != cudaSuccess)
+        if (cudaFuncSetAttribute(mlstm_sums_tc_kernel<TILES, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(mlstm_output_tc_kernel<TILES, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST_BYTES) != cudaSuccess)
             return LIA_ERR_LAUNCH;
         raised = true;
     }
     const dim3 grid(max_chunks, p.heads, (p.dv + piece - 1) / piece);
-    int code = lia_launch(mlstm_sums_tc_kernel<TILES>, grid, dim3(MLSTM_THREADS), sums_bytes(p.d, piece), stream, p, piece);
+    int code = lia_launch(mlstm_sums_tc_kernel<TILES, FULL>, grid, dim3(MLSTM_THREADS), sums_bytes(p.d, piece), stream, p, piece);
     if (code != LIA_OK) return code;
     code = mlstm_launch_carry(p, TOKENS, four, stream);
     if (code != LIA_OK) return code;
-    code = lia_launch(mlstm_output_tc_kernel<TILES>, grid, dim3(MLSTM_THREADS), output_bytes(p.d, piece), stream, p, piece);
+    code = lia_launch(mlstm_output_tc_kernel<TILES, FULL>, grid, dim3(MLSTM_THREADS), output_bytes(p.d, piece), stream, p, piece);
     if (code != LIA_OK || grid.z == 1) return code;
     return lia_launch(mlstm_norm_kernel, dim3(max_chunks, p.heads, TOKENS / (MLSTM_THREADS / 32)), dim3(MLSTM_THREADS), 0, stream, p);
 }
@@ -443,7 +457,8 @@ LIA_EXPORT int lia_mlstm_tc(const void* qkv, long long ld, const float* gates, l
         ld_g < (long long)heads * (dv + 2) || slot_stride < (long long)heads * ((long long)d * dv + d + 1) || max_chunks <= 0 ||
         !scratch || scratch_floats < mlstm_scratch_words(max_chunks, heads, d, dv) || (pieces > 1 && !y))
         return LIA_ERR_SIZE;
-    if (((uintptr_t)qkv | (uintptr_t)scratch | (uintptr_t)y | (uintptr_t)out) & 15u) return LIA_ERR_ALIGN;
+    if ((((uintptr_t)qkv | (uintptr_t)scratch | (uintptr_t)y | (uintptr_t)out) & 15u) || (((uintptr_t)gates | (uintptr_t)norm_weight) & 7u) || ld_g % 2)
+        return LIA_ERR_ALIGN;
     MlstmArgs p = {};
     p.qkv = qkv; p.ld = ld; p.qkv_bf16 = 1; p.gates = gates; p.ld_g = ld_g; p.i_bias = i_bias; p.f_bias = f_bias; p.cap = cap;
     p.state = state; p.slot_stride = slot_stride; p.segments = segments; p.n_segments = n_segments; p.slots = slots;
@@ -452,7 +467,11 @@ LIA_EXPORT int lia_mlstm_tc(const void* qkv, long long ld, const float* gates, l
     mlstm_place_scratch(p, scratch, max_chunks);
     const bool four = slot_stride % 4 == 0 && ((uintptr_t)state & 15u) == 0;
     const int piece = piece_of(d, dv);
-    if (piece <= 32) return launch_portions<2>(p, piece, max_chunks, four, stream);
-    if (piece <= 64) return launch_portions<4>(p, piece, max_chunks, four, stream);
-    return launch_portions<8>(p, piece, max_chunks, four, stream);
+#define LIA_PORTIONS(TILES)                                                                                            \
+    return piece == 16 * TILES && dv % piece == 0 ? launch_portions<TILES, true>(p, piece, max_chunks, four, stream)  \
+                                                  : launch_portions<TILES, false>(p, piece, max_chunks, four, stream)
+    if (piece <= 32) LIA_PORTIONS(2);
+    if (piece <= 64) LIA_PORTIONS(4);
+    LIA_PORTIONS(8);
+#undef LIA_PORTIONS
 }

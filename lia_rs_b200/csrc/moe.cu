@@ -361,21 +361,22 @@ LIA_EXPORT int lia_moe_route(const void* x, int dtype, long long ld, const float
     if (!raised) {
         cudaFuncSetAttribute(moe_route_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        cudaFuncSetAttribute(moe_route_kernel<float, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<float, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         raised = true;
     }
-    const bool eight = n >= 8 * 148 && 8 * one <= 200 * 1024;
+    const bool many = n >= 4 * 148 && 4 * one <= 200 * 1024;
+    const int threads = many || experts + extra <= 8 ? 256 : experts + extra <= 16 ? 512 : 1024;      // (few tokens: a warp an output)
 #define LIA_ROUTE(T, TOKENS)                                                                                             \
-    return lia_launch(moe_route_kernel<T, TOKENS>, dim3((n + TOKENS - 1) / TOKENS), dim3(256), TOKENS * one, stream,     \
+    return lia_launch(moe_route_kernel<T, TOKENS>, dim3((n + TOKENS - 1) / TOKENS), dim3(threads), TOKENS * one, stream,     \
                       (const T*)x, ld, router, n, hidden, experts, top, scale, extra, correction, groups, keep,          \
                       renormalise, sigmoid, two_best, ids, weights, shared_gate)
     if (dtype == LIA_F32) {
-        if (eight) LIA_ROUTE(float, 8);
+        if (many) LIA_ROUTE(float, 4);
         LIA_ROUTE(float, 1);
     }
     if (dtype == LIA_BF16) {
-        if (eight) LIA_ROUTE(__nv_bfloat16, 8);
+        if (many) LIA_ROUTE(__nv_bfloat16, 4);
         LIA_ROUTE(__nv_bfloat16, 1);
     }
 #undef LIA_ROUTE
