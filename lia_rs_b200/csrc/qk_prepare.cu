@@ -19,7 +19,7 @@
 #include "common.cuh"
 
 namespace {
-constexpr int PREP_WARPS = 4;
+constexpr int PREP_WARPS = 4, PREP_MOST_WARPS = 16;
 
 // page row (in units of cache rows) of `pos` for `slot`, or -1 with the flag raised
 __device__ __forceinline__ long long page_row(const int* __restrict__ block_table, int table_stride, int slot, int pos,
@@ -58,7 +58,7 @@ __device__ __forceinline__ void norm_and_rotate(float* h, int d, const float* __
 }
 
 template <typename T>
-__global__ void __launch_bounds__(PREP_WARPS * 32)
+__global__ void __launch_bounds__(PREP_MOST_WARPS * 32)
 qkv_prepare_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ bias,
                    const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
                    const float* __restrict__ freq, int rot_dims, int vmix_mode, float lambda,
@@ -67,7 +67,7 @@ qkv_prepare_kernel(const float* __restrict__ rows, long long ld, const float* __
                    T* __restrict__ k_pages, T* __restrict__ v_pages, int n_tokens, int nq, int nkv, int d, int dv,
                    int page_size, int num_pages, int write_kv, int norm_whole, int pairs, int norm_behind,
                    int* __restrict__ error_flag) {
-    extern __shared__ float prep_shared[];                 // [rot_dims] cosines then sines, then [PREP_WARPS][d]
+    extern __shared__ float prep_shared[];                 // [rot_dims] cosines then sines, then [warps][d]
     __shared__ float whole_scratch[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -99,7 +99,7 @@ qkv_prepare_kernel(const float* __restrict__ rows, long long ld, const float* __
             whole_inv[part] = 1.0f / sqrtf(sum / (float)width + eps);
         }
     }
-    for (int head = warp; head < nq + nkv; head += PREP_WARPS) {
+    for (int head = warp; head < nq + nkv; head += blockDim.x >> 5) {
         const bool is_q = head < nq;
         for (int i = lane; i < d; i += 32) h[i] = row[head * d + i] + (bias ? bias[head * d + i] : 0.f);
         if (norm_whole) {
@@ -212,9 +212,12 @@ LIA_EXPORT int lia_qkv_prepare(const float* rows, long long ld, const float* bia
         (rot_dims > 0 && !freq) || ld < (long long)(nq + nkv) * d + (long long)nkv * dv || vmix_mode < 0 || vmix_mode > 2 ||
         (vmix_mode && !v_first) || d > 4096)
         return LIA_ERR_SIZE;
-    const size_t smem = ((size_t)rot_dims + (size_t)PREP_WARPS * d) * sizeof(float);
+    // few tokens: up to a warp a head (a norm over whole projections keeps four: its sum follows the number of threads)
+    int warps = PREP_WARPS;
+    while (!norm_whole && n_tokens <= 256 && warps < PREP_MOST_WARPS && warps < nq + nkv && d <= 512) warps *= 2;
+    const size_t smem = ((size_t)rot_dims + (size_t)warps * d) * sizeof(float);
 #define LIA_PREP(T)                                                                                                   \
-    return lia_launch(qkv_prepare_kernel<T>, dim3(n_tokens), dim3(PREP_WARPS * 32), smem, stream, rows, ld, bias,     \
+    return lia_launch(qkv_prepare_kernel<T>, dim3(n_tokens), dim3(warps * 32), smem, stream, rows, ld, bias,     \
                       q_norm, k_norm, eps, freq, rot_dims, vmix_mode, lambda, v_first, positions, slots, block_table, \
                       table_stride, (T*)q_out, (T*)k_pages, (T*)v_pages, n_tokens, nq, nkv, d, dv, page_size,         \
                       num_pages, write_kv, norm_whole, pairs, norm_behind, error_flag)

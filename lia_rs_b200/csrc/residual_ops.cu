@@ -58,6 +58,26 @@ __global__ void stream_sum_kernel(float* __restrict__ x, const float* __restrict
         x[e] = v;
     }
 }
+
+// the same four elements a thread (hidden a multiple of 4, 16-byte aligned rows)
+template <typename TB>
+__global__ void stream_sum4_kernel(float* __restrict__ x, const float* __restrict__ x0, const TB* __restrict__ bias,
+                                   long long quads, int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < quads; e += (long long)gridDim.x * blockDim.x) {
+        float4 v = reinterpret_cast<const float4*>(x)[e];
+        if (x0) {
+            const float4 u = reinterpret_cast<const float4*>(x0)[e];
+            v.x += u.x, v.y += u.y, v.z += u.z, v.w += u.w;
+        }
+        if (bias) {
+            const TB* b = bias + (4 * e) % hidden;
+            v.x += to_float(b[0]), v.y += to_float(b[1]), v.z += to_float(b[2]), v.w += to_float(b[3]);
+        }
+        reinterpret_cast<float4*>(x)[e] = v;
+    }
+}
 }  // namespace
 
 // out[t, :] = table[token_t, :] * scale + position_table[position_t, :], 32-bit; `copy` (optional) receives the same.
@@ -102,6 +122,15 @@ LIA_EXPORT int lia_stream_sum(float* x, const float* x0, const void* bias, int b
                               cudaStream_t stream) {
     if (n_tokens <= 0 || (!x0 && !bias)) return LIA_OK;
     if (hidden <= 0) return LIA_ERR_SIZE;
+    if (hidden % 4 == 0 && (((uintptr_t)x | (uintptr_t)x0) & 15u) == 0) {
+        const long long quads = (long long)n_tokens * (hidden / 4);
+        const dim3 grid((unsigned)((quads + 255) / 256 < 148 * 16 ? (quads + 255) / 256 : 148 * 16));
+        if (bias_dtype == LIA_BF16)
+            return lia_launch(stream_sum4_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, x, x0, (const __nv_bfloat16*)bias, quads, hidden);
+        if (bias_dtype == LIA_F32)
+            return lia_launch(stream_sum4_kernel<float>, grid, dim3(256), 0, stream, x, x0, (const float*)bias, quads, hidden);
+        return LIA_ERR_DTYPE;
+    }
     const long long blocks = ((long long)n_tokens * hidden + 255) / 256;
     const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
     if (bias_dtype == LIA_BF16)
