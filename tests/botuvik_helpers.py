@@ -80,7 +80,7 @@ BOTUVIK = {
     "bot-F": dict(          # tensor-core sizes without a router (no row rests on a close call); the run is the first two layers
         config={"architecture": "Botuvik", "vocab": 160, "width": 96, "norm": {"eps": 1e-5}, "initializer_range": 0.06,
                 "layers": [
-                    _mlstm(4, 32, 64, 18.0, _dense(128)),
+                    _mlstm(3, 32, 64, 18.0, _dense(128)),
                     _attention(8, 2, 128, 128, 0.1, softcap=30.0, rot=(2e4, 64), mlp=None),
                     _mlstm(1, 16, 256, 7.0, _dense(64))],
                 "loop": {"start": 0, "stop": 2, "times": 2}},

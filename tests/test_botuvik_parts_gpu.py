@@ -370,7 +370,7 @@ def test_single_tokens_by_several_ctas_a_head(share, qkv_dtype):
 
 # ---- router, mixture, the stream's step ----
 
-@pytest.mark.parametrize("experts,top,groups", [(8, 3, (4, 3)), (6, 2, (3, 2)), (4, 1, (4, 2)), (12, 5, (2, 1)), (7, 7, None), (1, 1, None),
+@pytest.mark.parametrize("experts,top,groups", [(10, 3, (5, 4)), (6, 2, (3, 2)), (4, 1, (4, 2)), (12, 5, (2, 1)), (7, 7, None), (1, 1, None),
                                                 (64, 8, (8, 4)), (9, 3, (1, 1))])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_router(experts, top, groups, dtype):
@@ -412,7 +412,7 @@ def test_groups_are_judged_by_their_two_largest():
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("hidden,ff,experts,top,groups,shared,n", [
-    (72, 40, 6, 2, (3, 2), 24, 5), (64, 48, 8, 3, (4, 3), 96, 130), (128, 64, 8, 8, None, None, 33), (50, 30, 4, 1, (4, 1), 18, 17),
+    (72, 40, 6, 2, (3, 2), 24, 5), (64, 48, 10, 3, (5, 3), 96, 130), (128, 64, 8, 8, None, None, 33), (50, 30, 4, 1, (4, 1), 18, 17),
     (96, 32, 1, 1, None, 40, 9)])
 def test_mixture_with_an_ungated_shared_expert(hidden, ff, experts, top, groups, shared, n, dtype):
     from lia_rs_b200.cache import CacheManager
